@@ -573,3 +573,119 @@ class TevanexConfig:
         if cfg.vocab < 1 or cfg.width < 1 or not cfg.norm_eps > 0:
             raise ConfigError("config.json: vocab and width must be positive and norm.eps above zero")
         return cfg
+
+
+@dataclass(frozen=True)
+class ZatusunLayerConfig:
+    """One entry of ``layers``: the mixer's kind (``latent_attention``, ``attention`` or ``hgrn2``) and sizes, and the
+    feed-forward (None: the layer has only its mixer)."""
+    type: str
+    mixer: Mapping[str, Any]
+    mlp: Optional[Mapping[str, Any]]
+
+
+_ZATUSUN_MIXER_KEYS = {
+    "latent_attention": ("heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "scale"),
+    "attention": ("heads", "kv_heads", "dim", "vdim", "scale", "diff"),
+    "hgrn2": ("heads", "dim", "vdim"),
+}
+_ZATUSUN_ROT_SCALING_KEYS = {
+    "latent_attention": ("factor", "original", "fast", "slow"),
+    "attention": ("factor", "original", "low", "high"),
+}
+
+
+@dataclass(frozen=True)
+class ZatusunConfig:
+    """The keys of a Zatusun config.json: ``vocab``, ``width``, ``max_positions``, ``norm.eps``, ``embedding.scale``,
+    ``logit_softcap``, ``layers`` (each with ``type``, ``mixer`` and ``mlp``) and ``loop`` (layers start .. stop - 1 run
+    ``times`` times in a row).  A ``latent_attention`` names ``heads``, ``dim``, ``rot_dim``, ``vdim``, ``q_rank``,
+    ``kv_rank``, ``scale`` and ``rot`` (``base``, ``dims`` and optionally ``scaling`` with ``factor``, ``original``,
+    ``fast``, ``slow``); an ``attention`` ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale``, ``diff`` and optionally
+    ``mask.size`` and ``rot`` (``scaling`` with ``factor``, ``original``, ``low``, ``high``); an ``hgrn2`` ``heads``,
+    ``dim``, ``vdim``.  A feed-forward is of ``kind`` ``moe``: ``expert`` (``ff``, ``limit``) and ``router`` (``experts``,
+    ``top``)."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    embedding_scale: float
+    logit_softcap: float
+    layers: Tuple[ZatusunLayerConfig, ...]
+    loop: Optional[Tuple[int, int, int]]
+    max_positions: int          # rows of the learned position table; 0: left to the tensor's shape
+    eos_token_ids: Tuple[int, ...] = field(default_factory=tuple)
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "ZatusunConfig":
+        norm = d.get("norm") or {}
+        layers = []
+        for i, entry in enumerate(d.get("layers") or []):
+            kind = entry.get("type")
+            if kind not in _ZATUSUN_MIXER_KEYS:
+                raise ConfigError(f"config.json: layer {i} has a mixer of type {kind!r}; known: "
+                                  + ", ".join(sorted(_ZATUSUN_MIXER_KEYS)))
+            mixer = entry.get("mixer") or {}
+            for key in _ZATUSUN_MIXER_KEYS[kind]:
+                if mixer.get(key) is None:
+                    raise ConfigError(f"config.json: layer {i} ({kind}): mixer key {key!r} is missing")
+            if kind != "hgrn2":
+                rot, room = mixer.get("rot"), "rot_dim" if kind == "latent_attention" else "dim"
+                if rot:
+                    for key in ("base", "dims"):
+                        if rot.get(key) is None:
+                            raise ConfigError(f"config.json: layer {i}: mixer.rot.{key} is missing")
+                    if int(rot["dims"]) % 2 or int(rot["dims"]) > int(mixer[room]):
+                        raise ConfigError(f"config.json: layer {i}: mixer.rot.dims must be even and at most mixer.{room}")
+                    for key in _ZATUSUN_ROT_SCALING_KEYS[kind] if rot.get("scaling") else ():
+                        if rot["scaling"].get(key) is None:
+                            raise ConfigError(f"config.json: layer {i}: mixer.rot.scaling.{key} is missing")
+            if kind == "attention":
+                if int(mixer["kv_heads"]) < 1 or int(mixer["heads"]) % int(mixer["kv_heads"]):
+                    raise ConfigError(f"config.json: layer {i}: {mixer['heads']} query heads cannot be grouped over "
+                                      f"{mixer['kv_heads']} key/value heads")
+                if mixer.get("mask") and int(mixer["mask"].get("size") or 0) < 1:
+                    raise ConfigError(f"config.json: layer {i}: mixer.mask.size must be a positive number of positions")
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if mlp.get("kind") != "moe":
+                    raise ConfigError(f"config.json: layer {i}: a feed-forward of kind {mlp.get('kind')!r} is not known "
+                                      "(known: 'moe')")
+                for group, keys in (("expert", ("ff", "limit")), ("router", ("experts", "top"))):
+                    for key in keys:
+                        if (mlp.get(group) or {}).get(key) is None:
+                            raise ConfigError(f"config.json: layer {i}: mlp.{group}.{key} is missing")
+                if not 1 <= int(mlp["router"]["top"]) <= int(mlp["router"]["experts"]):
+                    raise ConfigError(f"config.json: layer {i}: mlp.router.top must lie between 1 and mlp.router.experts")
+            layers.append(ZatusunLayerConfig(str(kind), dict(mixer), dict(mlp) if mlp is not None else None))
+        if not layers:
+            raise ConfigError("config.json: 'layers' is missing or empty")
+        loop, loop_t = d.get("loop"), None
+        if loop:
+            loop_t = (_need(loop, "start", int), _need(loop, "stop", int), _need(loop, "times", int))
+            a, b, n = loop_t
+            if not (0 <= a < b <= len(layers)) or n < 1:
+                raise ConfigError(f"config.json: loop {dict(loop)} does not fit {len(layers)} layers")
+        eos = d.get("eos_token_id")
+        eos_ids = () if eos is None else (tuple(int(e) for e in eos) if isinstance(eos, (list, tuple)) else (int(eos),))
+        emb = d.get("embedding") or {}
+        cfg = cls(architecture=str(d.get("architecture") or (d.get("architectures") or ["Zatusun"])[0]),
+                  vocab=_need(d, "vocab", int), width=_need(d, "width", int), norm_eps=_need(norm, "eps", float),
+                  embedding_scale=float(emb["scale"]) if emb.get("scale") is not None else 1.0,
+                  logit_softcap=float(d["logit_softcap"]) if d.get("logit_softcap") else 0.0,
+                  layers=tuple(layers), loop=loop_t,
+                  max_positions=int(d.get("max_positions") or d.get("max_position_embeddings") or 0), eos_token_ids=eos_ids)
+        if cfg.vocab < 1 or cfg.width < 1 or not cfg.norm_eps > 0:
+            raise ConfigError("config.json: vocab and width must be positive and norm.eps above zero")
+        return cfg
+
+    def passes(self):
+        """(layer index, number of the pass that this run of the layer opens or None) in the order the layers run."""
+        n = len(self.layers)
+        if self.loop is None:
+            return [(i, None) for i in range(n)]
+        a, b, times = self.loop
+        order = [(i, None) for i in range(a)]
+        for t in range(times):
+            order += [(i, t if i == a else None) for i in range(a, b)]
+        return order + [(i, None) for i in range(b, n)]

@@ -7,13 +7,15 @@
 // ---------------------------------------------------------------- embedding
 // residual[t, :] = table[ids[t], :] * scale, the factor applied in float32   (upstream, without a factor:
 // base/src/kernels.cu:279-287)
+// With a position table: + pos_table[positions[t], :], which the factor leaves alone.
 // An id below zero names a token that the sampling kernel of the step before left on the
 // device: -(1 + r) stands for sampled[r] (n_sampled entries), so that a step can be
 // launched before the host has seen the tokens it starts from.
 template <typename T>
 __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __restrict__ ids,
                                     const int* __restrict__ sampled, int n_sampled,
-                                    float* __restrict__ resid, int H, int V, float scale, int* status) {
+                                    float* __restrict__ resid, int H, int V, float scale, const T* __restrict__ pos_table,
+                                    const int* __restrict__ positions, int n_positions, int* status) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
@@ -25,15 +27,28 @@ __global__ void embed_gather_kernel(const T* __restrict__ table, const int* __re
     return;
   }
   const T* row = table + (size_t)id * H;
-  for (int i = threadIdx.x; i < H; i += blockDim.x) resid[(size_t)t * H + i] = to_f32(row[i]) * scale;
+  const T* prow = nullptr;
+  if (pos_table != nullptr) {
+    const int pos = positions[t];
+    if (pos >= 0 && pos < n_positions) prow = pos_table + (size_t)pos * H;
+    else if (threadIdx.x == 0) atomicCAS(status, 0, KVB_STATUS_BAD_POSITION);
+  }
+  for (int i = threadIdx.x; i < H; i += blockDim.x) {
+    float v = to_f32(row[i]) * scale;
+    if (prow != nullptr) v += to_f32(prow[i]);
+    resid[(size_t)t * H + i] = v;
+  }
 }
 
 KVB_EXPORT int kvb_embed_gather(const void* table, int dtype, const int* ids, const int* sampled, int n_sampled,
-                                float* resid, int T_, int H, int V, float scale, int* status, cudaStream_t stream) {
+                                float* resid, int T_, int H, int V, float scale, const void* pos_table,
+                                const int* positions, int n_positions, int* status, cudaStream_t stream) {
   if (T_ <= 0) return 0;
+  if (pos_table != nullptr && positions == nullptr) return KVB_ERR_BAD_SIZE;
   const int threads = H >= 1024 ? 256 : 128;
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(embed_gather_kernel<T>, dim3(T_), dim3(threads), 0, stream,
-                                            (const T*)table, ids, sampled, n_sampled, resid, H, V, scale, status)));
+                                            (const T*)table, ids, sampled, n_sampled, resid, H, V, scale, (const T*)pos_table, positions, n_positions,
+                                            status)));
   return kvb_launch_result();
 }
 

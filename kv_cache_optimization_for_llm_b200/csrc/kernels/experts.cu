@@ -266,11 +266,13 @@ KVB_EXPORT int kvb_expert_act(const void* p, const float* gate, int ld_gate, voi
 // behind the E routed experts one that every token uses: S gate features, then S up features, with a limit of its own
 // and w = 1, whose result is multiplied by sigmoid(shared_logit[t * ld_s]) (float32; null: by 1), which for a last
 // matrix without bias is the same as multiplying its output.  gate [T, ld_gate] float32: the weights, 0 for an expert
-// that was not chosen.  out [T, E F + S + pad] dense, the padding columns zero.
+// that was not chosen.  weigh_output: the weight multiplies a(g) (u + 1) instead, behind the limits.
+// out [T, E F + S + pad] dense, the padding columns zero.
 template <typename T>
 __global__ void limited_act_kernel(const T* __restrict__ p, int ld_p, const float* __restrict__ gate, int ld_gate,
                                    const float* __restrict__ shared_logit, int ld_s, T* __restrict__ out, int E, int F,
-                                   int S, int width, float limit, float shared_limit, float alpha, size_t total) {
+                                   int S, int width, float limit, float shared_limit, float alpha, int weigh_output,
+                                   size_t total) {
   pdl_trigger();
   pdl_wait();
   const int EF = E * F;
@@ -283,9 +285,11 @@ __global__ void limited_act_kernel(const T* __restrict__ p, int ld_p, const floa
       const int e = j / F, i = j - e * F;
       const float w = gate[t * ld_gate + e];
       if (w != 0.f) {
-        const float g = fminf(w * to_f32(p[t * ld_p + 2 * e * F + i]), limit);
-        const float u = fminf(fmaxf(w * to_f32(p[t * ld_p + 2 * e * F + F + i]), -limit), limit);
+        const float w_in = weigh_output ? 1.0f : w;
+        const float g = fminf(w_in * to_f32(p[t * ld_p + 2 * e * F + i]), limit);
+        const float u = fminf(fmaxf(w_in * to_f32(p[t * ld_p + 2 * e * F + F + i]), -limit), limit);
         a = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+        if (weigh_output) a *= w;
       }
     } else if (j < EF + S) {
       const int i = j - EF;
@@ -309,7 +313,7 @@ __device__ __forceinline__ float limited_one(float g, float u, float w, float li
 __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, int ld_p, const float* __restrict__ gate,
                                           int ld_gate, const float* __restrict__ shared_logit, int ld_s,
                                           __nv_bfloat16* __restrict__ out, int E, int F, int S, int width, float limit,
-                                          float shared_limit, float alpha, size_t groups) {
+                                          float shared_limit, float alpha, int weigh_output, size_t groups) {
   pdl_trigger();
   pdl_wait();
   const int EF = E * F, gpr = width >> 3;
@@ -326,6 +330,7 @@ __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, i
       w = gate[t * ld_gate + e];
       gp = p + t * ld_p + 2 * e * F + i;
       up = gp + F;
+      if (weigh_output && w != 0.f) { post = w; w = 1.f; }
     } else if (j < EF + S) {
       w = 1.f;
       lim = shared_limit;
@@ -354,7 +359,7 @@ __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, i
 
 KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int ld_gate, const float* shared_logit,
                                int ld_s, void* out, int T_, int E, int F, int S, int pad, float limit, float shared_limit,
-                               float alpha, int dtype, cudaStream_t stream) {
+                               float alpha, int weigh_output, int dtype, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   const int width = E * F + S + pad;
   if (E < 0 || F < 1 || S < 0 || pad < 0 || E * F + S < 1 || ld_p < 2 * (E * F + S)) return KVB_ERR_BAD_SIZE;
@@ -364,7 +369,8 @@ KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int l
     const size_t want8 = (groups + 255) / 256;
     const int blocks8 = (int)(want8 < (size_t)kvb_sm_count() * 16 ? want8 : (size_t)kvb_sm_count() * 16);
     kvb_launch(limited_act_bf16x8_kernel, dim3(blocks8), dim3(256), 0, stream, (const __nv_bfloat16*)p, ld_p, gate, ld_gate,
-               shared_logit, ld_s, (__nv_bfloat16*)out, E, F, S, width, limit, shared_limit, alpha, groups);
+               shared_logit, ld_s, (__nv_bfloat16*)out, E, F, S, width, limit, shared_limit, alpha, weigh_output,
+               groups);
     return kvb_launch_result();
   }
   const size_t total = (size_t)T_ * width;
@@ -372,7 +378,7 @@ KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int l
   const int blocks = (int)(want < (size_t)kvb_sm_count() * 16 ? want : (size_t)kvb_sm_count() * 16);
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(limited_act_kernel<T>, dim3(blocks), dim3(256), 0, stream, (const T*)p, ld_p,
                                             gate, ld_gate, shared_logit, ld_s, (T*)out, E, F, S, width, limit,
-                                            shared_limit, alpha, total)));
+                                            shared_limit, alpha, weigh_output, total)));
   return kvb_launch_result();
 }
 

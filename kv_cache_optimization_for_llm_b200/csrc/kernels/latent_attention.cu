@@ -5,12 +5,15 @@
 // The up-projections are moved to the query side: with k_h = U_h c the score q.k_h equals
 // (U_h^T q).c, so every head attends with an "absorbed" query [U_h^T q_plain | q_rot] over the
 // same cached rows, the weighted sum of the latents comes out [rank] wide per head and the
-// value up-projection is applied to it afterwards.  Three kernels:
+// value up-projection is applied to it afterwards.  The kernels:
 //   latent_prep       per token: RMS norm of the query latent, RMS norm of the key/value latent,
 //                     interleaved rotary encoding of the shared key part, cache write
 //   head_gemm         a product per head, out[t, h, :] = W[h] . in[t, h, :]  (absorbs the queries,
-//                     and up-projects the attended latents)
-//   latent_attention  causal softmax attention of all heads over the cached rows, with a sink:
+//                     and up-projects the attended latents; with a gate its result is multiplied by
+//                     the gate's sigmoid)
+//   head_rows         for steps whose per-head products the library made: [heads, tokens, N] back to one
+//                     row per token, with the same optional gate
+//   latent_attention  causal softmax attention of all heads over the cached rows, optionally with a sink:
 //                     the denominator also holds exp(sink_h), a key without a value
 // Scores, softmax weights, sums and angles are float32.  Keys are walked in chunks of 32 by
 // absolute position, so a token's result does not depend on how its request was cut into steps,
@@ -93,10 +96,11 @@ KVB_EXPORT int kvb_latent_prep(const void* d_in, int ld, int q_rank, int kv_off,
 // Plain FMA in ascending k with float32 sums: an output does not depend on the number of rows.
 constexpr int HG_BM = 64, HG_BN = 64, HG_BK = 16;
 
+// With `gate` (row stride ld_gate, the layout of out): times sigmoid(gate[t, h * hs_out + n]).
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_gemm_kernel(const T* __restrict__ in, int ld_in, int hs_in, const T* __restrict__ W, T* __restrict__ out,
-                 int ld_out, int hs_out, int M, int N, int K) {
+                 int ld_out, int hs_out, int M, int N, int K, const T* __restrict__ gate, int ld_gate) {
   __shared__ float As[HG_BK][HG_BM + 4];
   __shared__ float Ws[HG_BK][HG_BN + 4];
   pdl_trigger();
@@ -143,19 +147,82 @@ head_gemm_kernel(const T* __restrict__ in, int ld_in, int hs_in, const T* __rest
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) out[(size_t)m * ld_out + (size_t)h * hs_out + n] = from_f32<T>(acc[i][j]);
+      if (n < N) {
+        float v = acc[i][j];
+        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-to_f32(gate[(size_t)m * ld_gate + (size_t)h * hs_out + n])));
+        out[(size_t)m * ld_out + (size_t)h * hs_out + n] = from_f32<T>(v);
+      }
     }
   }
 }
 
 KVB_EXPORT int kvb_head_gemm(const void* in, int ld_in, int hs_in, const void* W, void* out, int ld_out, int hs_out,
-                             int M, int N, int K, int H, int dtype, cudaStream_t stream) {
+                             int M, int N, int K, int H, const void* gate, int ld_gate, int dtype, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || H <= 0) return 0;
   if (K <= 0 || H > 65535) return KVB_ERR_BAD_SIZE;
   dim3 grid((N + HG_BN - 1) / HG_BN, (M + HG_BM - 1) / HG_BM, H);
   if (grid.y > 65535) return KVB_ERR_BAD_SIZE;
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(head_gemm_kernel<T>, grid, dim3(256), 0, stream, (const T*)in, ld_in, hs_in,
-                                            (const T*)W, (T*)out, ld_out, hs_out, M, N, K)));
+                                            (const T*)W, (T*)out, ld_out, hs_out, M, N, K, (const T*)gate, ld_gate)));
+  return kvb_launch_result();
+}
+
+// in [H, T, N] dense (a batched product's result) -> out[t, h * N + n], times sigmoid(gate[t, h * N + n]) when there is a
+// gate.  VEC elements per thread (N a multiple of VEC; 16-byte accesses with VEC 8).
+template <int VEC>
+__global__ void __launch_bounds__(256)
+head_rows_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, int ld_out,
+                 const __nv_bfloat16* __restrict__ gate, int ld_gate, int T_, int H, int N, size_t total) {
+  pdl_trigger();
+  pdl_wait();
+  const int per_head = N / VEC;
+  for (size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (size_t)gridDim.x * blockDim.x) {
+    const size_t th = idx / per_head;
+    const int n = (int)(idx - th * per_head) * VEC;
+    const size_t t = th / H;
+    const int h = (int)(th - t * H);
+    const __nv_bfloat16* src = in + ((size_t)h * T_ + t) * N + n;
+    const __nv_bfloat16* g = gate != nullptr ? gate + t * ld_gate + (size_t)h * N + n : nullptr;
+    __nv_bfloat16* dst = out + t * ld_out + (size_t)h * N + n;
+    alignas(16) __nv_bfloat16 x[VEC];
+    alignas(16) __nv_bfloat16 gv[VEC];
+    if (VEC == 8) {
+      *reinterpret_cast<uint4*>(x) = *reinterpret_cast<const uint4*>(src);
+      if (g != nullptr) *reinterpret_cast<uint4*>(gv) = *reinterpret_cast<const uint4*>(g);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { x[i] = src[i]; if (g != nullptr) gv[i] = g[i]; }
+    }
+    if (g != nullptr) {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i)
+        x[i] = __float2bfloat16_rn(__bfloat162float(x[i]) / (1.0f + expf(-__bfloat162float(gv[i]))));
+    }
+    if (VEC == 8) {
+      *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(x);
+    } else {
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) dst[i] = x[i];
+    }
+  }
+}
+
+KVB_EXPORT int kvb_head_rows(const void* in, void* out, int ld_out, const void* gate, int ld_gate, int T_, int H, int N,
+                             cudaStream_t stream) {
+  if (T_ <= 0 || H <= 0) return 0;
+  if (N < 1) return KVB_ERR_BAD_SIZE;
+  const bool vec = N % 8 == 0 && ld_out % 8 == 0 && ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
+                   (gate == nullptr || (ld_gate % 8 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0));
+  const size_t total = (size_t)T_ * H * (vec ? N / 8 : N);
+  const size_t want = (total + 255) / 256;
+  const int blocks = (int)(want < (size_t)kvb_sm_count() * 16 ? want : (size_t)kvb_sm_count() * 16);
+  using B = __nv_bfloat16;
+  if (vec)
+    kvb_launch(head_rows_kernel<8>, dim3(blocks), dim3(256), 0, stream, (const B*)in, (B*)out, ld_out, (const B*)gate, ld_gate,
+               T_, H, N, total);
+  else
+    kvb_launch(head_rows_kernel<1>, dim3(blocks), dim3(256), 0, stream, (const B*)in, (B*)out, ld_out, (const B*)gate, ld_gate,
+               T_, H, N, total);
   return kvb_launch_result();
 }
 
@@ -163,7 +230,7 @@ KVB_EXPORT int kvb_head_gemm(const void* in, int ld_in, int hs_in, const void* W
 // A block takes one query token and up to kLatWarps heads, one head per warp.  The block loads a
 // chunk of 32 cached rows into shared memory once for all its heads; a lane scores one key
 // (dot over Dc), the warp keeps a running maximum and sum that start from the sink
-// (m = sink_h, l = 1: the sink counts once and has no value), and lanes then own value dims.
+// (m = sink_h, l = 1: the sink counts once and has no value; without one m = -inf, l = 0), and lanes then own value dims.
 constexpr int kLatWarps = 8;
 
 template <typename T> struct Word;     // a 4-byte word of shared memory: 1 float or 2 bfloat16
@@ -221,7 +288,7 @@ latent_attention_kernel(const T* __restrict__ q_abs, int ld_qa, int hs_qa,     /
     }
     for (int i = rdims + lane; i < rot; i += 32) q[rank + i] = to_f32(qr[i]);
   }
-  float m = live ? sink[h] : 0.f, l = 1.f;
+  float m = sink == nullptr ? -CUDART_INF_F : (live ? sink[h] : 0.f), l = sink == nullptr ? 0.f : 1.f;
   float acc[NR];
 #pragma unroll
   for (int r = 0; r < NR; ++r) acc[r] = 0.f;
@@ -257,6 +324,7 @@ latent_attention_kernel(const T* __restrict__ q_abs, int ld_qa, int hs_qa,     /
       s = dot * scale;
     }
     const float m_new = fmaxf(m, warp_max(s));
+    if (m_new == -CUDART_INF_F) continue;              // no readable key yet, and no sink
     const float corr = expf(m - m_new);
     const float p = s == -CUDART_INF_F ? 0.f : expf(s - m_new);
     l = l * corr + warp_sum(p);
@@ -279,7 +347,7 @@ latent_attention_kernel(const T* __restrict__ q_abs, int ld_qa, int hs_qa,     /
 #pragma unroll
   for (int r = 0; r < NR; ++r) {
     const int i = r * 32 + lane;
-    if (i < rank) o[i] = from_f32<T>(acc[r] / l);
+    if (i < rank) o[i] = from_f32<T>(l > 0.f ? acc[r] / l : 0.f);
   }
 }
 
@@ -423,7 +491,11 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     }
     for (int i = rdims + lane; i < rot; i += 32) q[rank + i] = qr[i];
     for (int i = Dc + lane; i < DcP; i += 32) q[i] = __float2bfloat16_rn(0.f);
-    if (lane == 0) { pos_s[r] = pos; m_s[r] = sink[hh]; l_s[r] = 1.f; }
+    if (lane == 0) {
+      pos_s[r] = pos;
+      m_s[r] = sink == nullptr ? -CUDART_INF_F : sink[hh];
+      l_s[r] = sink == nullptr ? 0.f : 1.f;
+    }
   }
   const int max_pos = ntok > 0 ? positions[first + ntok - 1] : -1;
 
@@ -535,7 +607,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
       psum += __shfl_xor_sync(0xffffffffu, psum, 1);
       psum += __shfl_xor_sync(0xffffffffu, psum, 2);
       if ((tid & 3) == 0) {
-        const float corr = expf(m_old - m_new);
+        const float corr = m_old == m_new ? 1.f : expf(m_old - m_new);     // also where neither a key nor a sink was met yet
         m_s[row] = m_new;
         l_s[row] = l_s[row] * corr + psum;
         corr_s[row] = corr;
@@ -571,7 +643,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     const int r = mrow + g + 8 * hrow;
     if (r >= rows_used) continue;
     const int tl = r / HB, hh = h0 + r - tl * HB;
-    const float inv = 1.0f / l_s[r];
+    const float inv = l_s[r] > 0.f ? 1.0f / l_s[r] : 0.f;
     __nv_bfloat16* o = out + (size_t)(first + tl) * ld_out + (size_t)hh * hs_out + ncol0 + 2 * t4;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {

@@ -234,7 +234,7 @@ KVB_EXPORT int kvb_tanh_slice(const void* in, int ld, void* out, int T_, int n, 
 
 // ---------------------------------------------------------------- several summands join the residual, then a norm
 // For output row b (token row t = rows ? rows[b] : b):
-//   v = resid[t] + d1[t] + d2[t] + e[t] + vec        every summand optional: two branch outputs (a layer whose
+//   v = (base ? base[t] : resid[t]) + d1[t] + d2[t] + e[t] + vec       base: float32 rows that take the stream's place; every summand optional: two branch outputs (a layer whose
 //                                                     sublayers read the same normed input), float32 rows (the
 //                                                     embedding's output re-entering), one float32 vector for all rows
 //   resid[t] = v                                      (only when every row is produced: rows == null)
@@ -242,20 +242,20 @@ KVB_EXPORT int kvb_tanh_slice(const void* in, int ld, void* out, int T_, int n, 
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
 join_norm_kernel(float* __restrict__ resid, const T* __restrict__ d1, const T* __restrict__ d2,
-                 const float* __restrict__ e, const float* __restrict__ vec, const float* __restrict__ w, int kind,
-                 float eps, void* __restrict__ out, int out_f32, const int* __restrict__ rows, int H) {
+                 const float* __restrict__ e, const float* __restrict__ vec, const float* __restrict__ base,
+                 const float* __restrict__ w, int kind, float eps, void* __restrict__ out, int out_f32, const int* __restrict__ rows, int H) {
   extern __shared__ float row[];
   __shared__ float part[32];
   pdl_trigger();
   pdl_wait();
   const int b = blockIdx.x;
   const size_t src = (size_t)(rows ? rows[b] : b) * H;
-  const bool any = d1 != nullptr || d2 != nullptr || e != nullptr || vec != nullptr;
+  const bool any = d1 != nullptr || d2 != nullptr || e != nullptr || vec != nullptr || base != nullptr;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
     float branches = 0.f;                          // the branches are summed first, then joined to the stream
     if (d1) branches = to_f32(d1[src + i]);
     if (d2) branches += to_f32(d2[src + i]);
-    float v = resid[src + i] + branches;
+    float v = (base ? base[src + i] : resid[src + i]) + branches;
     if (e) v += e[src + i];
     if (vec) v += vec[i];
     row[i] = v;
@@ -276,7 +276,7 @@ join_norm_kernel(float* __restrict__ resid, const T* __restrict__ d1, const T* _
 
 // dtype: the type of d1 and d2 (and of out unless out_f32).  Refuses rows wider than 51200.
 KVB_EXPORT int kvb_join_norm(float* resid, const void* d1, const void* d2, const float* e, const float* vec,
-                             const float* w, int kind, float eps, void* out, int out_f32, const int* rows,
+                             const float* base, const float* w, int kind, float eps, void* out, int out_f32, const int* rows,
                              int n_out_rows, int H, int dtype, cudaStream_t stream) {
   if (n_out_rows <= 0) return 0;
   if (kind < 0 || kind > 2) return KVB_ERR_BAD_SIZE;
@@ -288,7 +288,7 @@ KVB_EXPORT int kvb_join_norm(float* resid, const void* d1, const void* d2, const
       if (err != cudaSuccess) return (int)err;
     }
     kvb_launch(join_norm_kernel<T>, dim3(n_out_rows), dim3(kRowThreads), smem, stream, resid, (const T*)d1,
-               (const T*)d2, e, vec, w, kind, eps, out, out_f32, rows, H);
+               (const T*)d2, e, vec, base, w, kind, eps, out, out_f32, rows, H);
   });
   return kvb_launch_result();
 }

@@ -9,7 +9,11 @@
 // joins the softmax's denominator once and has no value (exp(sink_h) beside the keys' exp(s)); `chunk`, a mask by
 // blocks of positions counted from the sequence's start (query i sees key j <= i only when i / chunk == j / chunk);
 // and `gate`, rows in the activations' type by whose sigmoid the result is multiplied element by element
-// (gate[t * gate_ld + head * Dv + i]).  Members left out of an initialiser are null or 0: absent.
+// (gate[t * gate_ld + head * Dv + i]).  And `pair`: two attention maps per head over the same values (differential
+// attention).  A query head then holds two queries of Dk, [map 1 | map 2], a key/value head two keys in front of its
+// value, [k1 | k2 | v]; each map has a softmax of its own, and the head's result a1 - pair_weight * a2 is divided by its
+// root mean square over the Dv channels (pair_eps inside the root) before out_scale multiplies it.
+// Members left out of an initialiser are null or 0: absent.
 struct ScoreShape {
   const float* head_scale;   // [heads] or null
   const float* slopes;       // [heads] or null
@@ -19,6 +23,8 @@ struct ScoreShape {
   int chunk;                 // 0: none
   const void* gate;          // [T, >= heads * Dv] or null
   int gate_ld;
+  int pair;                  // 1: two maps per head
+  float pair_weight, pair_eps;
 };
 
 // The first key that position `pos` sees: the window's and the block's lower ends, whichever is later.

@@ -96,33 +96,50 @@ __device__ __forceinline__ float key_dot<__nv_bfloat16>(const float* q_s, const 
   return dot;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kWarps * 32)
+// From the partial softmax states of NW warps (their maxima and sums, STRIDE floats apart): each warp's factor on its
+// partial results, and one over the merged sum (0 without any key).
+template <int NW, int STRIDE>
+__device__ __forceinline__ float merge_factors(const float* m, const float* l, float* f) {
+  float M = -CUDART_INF_F, L = 0.f;
+  for (int w = 0; w < NW; ++w) M = fmaxf(M, m[w * STRIDE]);
+  for (int w = 0; w < NW; ++w) {
+    f[w] = (m[w * STRIDE] == -CUDART_INF_F) ? 0.f : expf(m[w * STRIDE] - M);
+    L += l[w * STRIDE] * f[w];
+  }
+  return L > 0.f ? 1.0f / L : 0.f;
+}
+
+// PAIR: two maps per head (see ScoreShape): four warps for each, over the same chunks.
+template <typename T, bool PAIR>
+__global__ void __launch_bounds__(kWarps * 32 * (PAIR ? 2 : 1))
 window_attention_kernel(const T* __restrict__ q_base, int q_row_stride, const T* __restrict__ pages,
                         const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
                         const int* __restrict__ positions, const int* __restrict__ token_req, T* __restrict__ out,
                         int nq, int nkv, int Dk, int Dv, float scale, int window, int keep_first, int one_more,
                         int vec, ScoreShape shape, int* status) {
-  __shared__ float q_s[kMaxDim];
-  __shared__ float acc_s[kWarps][kMaxDim];
-  __shared__ float m_s[kWarps], l_s[kWarps];
+  constexpr int kMaps = PAIR ? 2 : 1;
+  __shared__ float q_all[kMaps * kMaxDim];
+  __shared__ float acc_s[kMaps * kWarps][kMaxDim];
+  __shared__ float m_s[kMaps * kWarps], l_s[kMaps * kWarps];
 
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
   const int hk = h / (nq / nkv);
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int slot = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int map = PAIR ? slot / kWarps : 0, warp = PAIR ? slot % kWarps : slot;
   const int pos = positions[t];
   const int* table = block_table + (size_t)token_req[t] * max_pages;
-  const int row_len = Dk + Dv;
+  const int v_at = kMaps * Dk, row_len = v_at + Dv;
   const int lo = first_seen_key(pos, window, shape.chunk);       // first key of the window or of the position's block
   const int keep = window > 0 ? keep_first : 0;                  // keys below it are seen whatever the window
   const int keep_chunks = (keep + 31) / 32;
   const int lo_chunk = lo / 32;
 
-  const T* q = q_base + (size_t)t * q_row_stride + (size_t)h * Dk;
-  for (int i = threadIdx.x; i < Dk; i += blockDim.x) q_s[i] = to_f32(q[i]);
+  const T* q = q_base + (size_t)t * q_row_stride + (size_t)h * v_at;
+  for (int i = threadIdx.x; i < v_at; i += blockDim.x) q_all[i] = to_f32(q[i]);
   __syncthreads();
+  const float* q_s = q_all + map * Dk;
 
   float m = -CUDART_INF_F, l = 0.f;
   float acc[kMaxDim / 32];
@@ -146,7 +163,7 @@ window_attention_kernel(const T* __restrict__ q_base, int q_row_stride, const T*
         atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE);
       } else {
         off = (((long long)page * nkv + hk) * page_size + (j % page_size)) * row_len;
-        s = shape_score(key_dot<T>(q_s, pages + off, Dk, vec != 0) * scale, shape, h, pos - j);
+        s = shape_score(key_dot<T>(q_s, pages + off + map * Dk, Dk, vec != 0) * scale, shape, h, pos - j);
       }
     }
     const float cm = warp_max(s);
@@ -162,7 +179,7 @@ window_attention_kernel(const T* __restrict__ q_base, int q_row_stride, const T*
       const long long oj = __shfl_sync(0xffffffffu, off, jj);
       const float pj = __shfl_sync(0xffffffffu, p, jj);
       if (oj < 0) continue;
-      const T* v = pages + oj + Dk;
+      const T* v = pages + oj + v_at;
 #pragma unroll
       for (int r = 0; r < kMaxDim / 32; ++r) {
         const int i = r * 32 + lane;
@@ -172,13 +189,38 @@ window_attention_kernel(const T* __restrict__ q_base, int q_row_stride, const T*
     m = m_new;
   }
 
-  if (lane == 0) { m_s[warp] = m; l_s[warp] = l; }
+  if (lane == 0) { m_s[slot] = m; l_s[slot] = l; }
 #pragma unroll
   for (int r = 0; r < kMaxDim / 32; ++r) {
     const int i = r * 32 + lane;
-    if (i < Dv) acc_s[warp][i] = acc[r];
+    if (i < Dv) acc_s[slot][i] = acc[r];
   }
   __syncthreads();
+  if (PAIR) {
+    if (slot == 0) {
+      T* o = out + ((size_t)t * nq + h) * Dv;
+      float inv[2], f[2][kWarps];
+      for (int a = 0; a < 2; ++a) inv[a] = merge_factors<kWarps, 1>(m_s + a * kWarps, l_s + a * kWarps, f[a]);
+      float d[kMaxDim / 32], ss = 0.f;
+#pragma unroll
+      for (int r = 0; r < kMaxDim / 32; ++r) {
+        const int i = r * 32 + lane;
+        float a1 = 0.f, a2 = 0.f;
+        if (i < Dv) {
+          for (int w = 0; w < kWarps; ++w) { a1 += acc_s[w][i] * f[0][w]; a2 += acc_s[kWarps + w][i] * f[1][w]; }
+        }
+        d[r] = a1 * inv[0] - shape.pair_weight * (a2 * inv[1]);
+        ss = fmaf(d[r], d[r], ss);
+      }
+      const float g = shape.out_scale / sqrtf(warp_sum(ss) / (float)Dv + shape.pair_eps);
+#pragma unroll
+      for (int r = 0; r < kMaxDim / 32; ++r) {
+        const int i = r * 32 + lane;
+        if (i < Dv) o[i] = from_f32<T>(d[r] * g);
+      }
+    }
+    return;
+  }
   if (warp == 0) {
     // what joins the denominator without a value: a key of score 0, or the head's learned score
     const float extra = one_more ? 0.f : (shape.sinks != nullptr ? shape.sinks[h] : -CUDART_INF_F);
@@ -244,7 +286,8 @@ __device__ __forceinline__ void load_16_bytes(const __nv_bfloat16* p, float* x) 
 
 // Small groups and values keep to 64 registers, so that four blocks share an SM (a decode step of 64 requests and
 // 8 key/value heads is then one round of blocks, not one and a seventh).
-template <typename T, int VPL, int GP>
+// PAIR: the GP rows of queries are the group's heads times two maps, row g being map g % 2 of head g / 2.
+template <typename T, int VPL, int GP, bool PAIR>
 __global__ void __launch_bounds__(kGroupWarps * 32, (GP * VPL <= 8) ? 4 : 1)
 window_attention_group_kernel(const T* __restrict__ q_base, int q_row_stride, const T* __restrict__ pages,
                               const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
@@ -261,11 +304,12 @@ window_attention_group_kernel(const T* __restrict__ q_base, int q_row_stride, co
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x, hk = blockIdx.y;
-  const int G = nq / nkv;
+  constexpr int kMaps = PAIR ? 2 : 1;
+  const int G = nq / nkv * kMaps;                    // rows of queries of this key/value head
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = positions[t];
   const int* table = block_table + (size_t)token_req[t] * max_pages;
-  const int row_len = Dk + Dv;
+  const int v_at = kMaps * Dk, row_len = v_at + Dv;
   const int lo = first_seen_key(pos, window, shape.chunk);
   const int keep = window > 0 ? keep_first : 0;
   const int keep_chunks = (keep + 31) / 32;
@@ -307,29 +351,34 @@ window_attention_group_kernel(const T* __restrict__ q_base, int q_row_stride, co
         for (int g = 0; g < GP; ++g) dot[g] = 0.f;
         if (vec) {
           constexpr int PER = 16 / (int)sizeof(T);
+#pragma unroll
+          for (int a = 0; a < kMaps; ++a) {
 #pragma unroll 4
-          for (int i = 0; i < Dk; i += PER) {     // unrolled: the row's loads are all requested before the first is used
-            float x[PER];
-            load_16_bytes(k + i, x);
+            for (int i = 0; i < Dk; i += PER) {     // unrolled: the row's loads are all requested before the first is used
+              float x[PER];
+              load_16_bytes(k + a * Dk + i, x);
 #pragma unroll
-            for (int e4 = 0; e4 < PER; e4 += 4) {
+              for (int e4 = 0; e4 < PER; e4 += 4) {
 #pragma unroll
-              for (int g = 0; g < GP; ++g) {
-                const float4 qv = *reinterpret_cast<const float4*>(q_s + g * Dk + i + e4);
-                dot[g] = fmaf(qv.x, x[e4], dot[g]); dot[g] = fmaf(qv.y, x[e4 + 1], dot[g]);
-                dot[g] = fmaf(qv.z, x[e4 + 2], dot[g]); dot[g] = fmaf(qv.w, x[e4 + 3], dot[g]);
+                for (int g = a; g < GP; g += kMaps) {
+                  const float4 qv = *reinterpret_cast<const float4*>(q_s + g * Dk + i + e4);
+                  dot[g] = fmaf(qv.x, x[e4], dot[g]); dot[g] = fmaf(qv.y, x[e4 + 1], dot[g]);
+                  dot[g] = fmaf(qv.z, x[e4 + 2], dot[g]); dot[g] = fmaf(qv.w, x[e4 + 3], dot[g]);
+                }
               }
             }
           }
         } else {
-          for (int i = 0; i < Dk; ++i) {
-            const float x = to_f32(k[i]);
 #pragma unroll
-            for (int g = 0; g < GP; ++g) dot[g] = fmaf(q_s[g * Dk + i], x, dot[g]);
-          }
+          for (int a = 0; a < kMaps; ++a)
+            for (int i = 0; i < Dk; ++i) {
+              const float x = to_f32(k[a * Dk + i]);
+#pragma unroll
+              for (int g = a; g < GP; g += kMaps) dot[g] = fmaf(q_s[g * Dk + i], x, dot[g]);
+            }
         }
 #pragma unroll
-        for (int g = 0; g < GP; ++g) s[g] = g < G ? shape_score(dot[g] * scale, shape, hk * G + g, pos - j) : 0.f;
+        for (int g = 0; g < GP; ++g) s[g] = g < G ? shape_score(dot[g] * scale, shape, (hk * G + g) / kMaps, pos - j) : 0.f;
       }
     }
     if (warp_max(off >= 0 ? 1.f : -CUDART_INF_F) == -CUDART_INF_F) continue;   // nothing readable in this chunk
@@ -352,7 +401,7 @@ window_attention_group_kernel(const T* __restrict__ q_base, int q_row_stride, co
       for (int u = 0; u < 8; ++u) {
         const long long oj = __shfl_sync(0xffffffffu, off, (jj0 + u) & 31);
         if (oj >= 0 && jj0 + u < n_in_chunk) {
-          load_values<T, VPL>(pages + oj + Dk + lane * VPL, x[u]);
+          load_values<T, VPL>(pages + oj + v_at + lane * VPL, x[u]);
         } else {
 #pragma unroll
           for (int r = 0; r < VPL; ++r) x[u][r] = 0.f;
@@ -377,56 +426,83 @@ window_attention_group_kernel(const T* __restrict__ q_base, int q_row_stride, co
     for (int r = 0; r < VPL; ++r) acc_s[(warp * GP + g) * Dv + lane * VPL + r] = acc[g][r];
   }
   __syncthreads();
-  // warp g finishes head g: the warps' partial sums are merged in the order of the warps
-  for (int g = warp; g < G; g += kGroupWarps) {
-    const int hq = hk * G + g;
-    const float extra = one_more ? 0.f : (shape.sinks != nullptr ? shape.sinks[hq] : -CUDART_INF_F);
-    float M = extra;
-    for (int w = 0; w < kGroupWarps; ++w) M = fmaxf(M, m_s[w * GP + g]);
-    float L = extra == -CUDART_INF_F ? 0.f : expf(extra - M), f[kGroupWarps];
-    for (int w = 0; w < kGroupWarps; ++w) {
-      const float mw = m_s[w * GP + g];
-      f[w] = (mw == -CUDART_INF_F) ? 0.f : expf(mw - M);
-      L += l_s[w * GP + g] * f[w];
+  if constexpr (PAIR) {      // warp w finishes head w: both maps' merged results, their difference, its norm over the head's channels
+    for (int hh = warp; hh < G / 2; hh += kGroupWarps) {
+      float inv[2], f[2][kGroupWarps];
+#pragma unroll
+      for (int a = 0; a < 2; ++a)
+        inv[a] = merge_factors<kGroupWarps, GP>(m_s + 2 * hh + a, l_s + 2 * hh + a, f[a]);
+      float d[VPL], ss = 0.f;
+#pragma unroll
+      for (int r = 0; r < VPL; ++r) {
+        const int i = r * 32 + lane;
+        float a1 = 0.f, a2 = 0.f;
+        for (int w = 0; w < kGroupWarps; ++w) {
+          a1 += acc_s[(w * GP + 2 * hh) * Dv + i] * f[0][w];
+          a2 += acc_s[(w * GP + 2 * hh + 1) * Dv + i] * f[1][w];
+        }
+        d[r] = a1 * inv[0] - shape.pair_weight * (a2 * inv[1]);
+        ss = fmaf(d[r], d[r], ss);
+      }
+      const float scale_out = shape.out_scale / sqrtf(warp_sum(ss) / (float)Dv + shape.pair_eps);
+      T* o = out + ((size_t)t * nq + hk * (G / 2) + hh) * Dv;
+#pragma unroll
+      for (int r = 0; r < VPL; ++r) o[r * 32 + lane] = from_f32<T>(d[r] * scale_out);
     }
-    T* o = out + ((size_t)t * nq + hq) * Dv;
-    const T* gate = shape.gate ? static_cast<const T*>(shape.gate) + (size_t)t * shape.gate_ld + (size_t)hq * Dv : nullptr;
-    for (int i = lane; i < Dv; i += 32) {
-      float a = 0.f;
-      for (int w = 0; w < kGroupWarps; ++w) a += acc_s[(w * GP + g) * Dv + i] * f[w];
-      a = L > 0.f ? a / L * shape.out_scale : 0.f;
-      if (gate != nullptr) a *= 1.0f / (1.0f + expf(-to_f32(gate[i])));
-      o[i] = from_f32<T>(a);
+  } else {
+    // warp g finishes head g: the warps' partial sums are merged in the order of the warps
+    for (int g = warp; g < G; g += kGroupWarps) {
+      const int hq = hk * G + g;
+      const float extra = one_more ? 0.f : (shape.sinks != nullptr ? shape.sinks[hq] : -CUDART_INF_F);
+      float M = extra;
+      for (int w = 0; w < kGroupWarps; ++w) M = fmaxf(M, m_s[w * GP + g]);
+      float L = extra == -CUDART_INF_F ? 0.f : expf(extra - M), f[kGroupWarps];
+      for (int w = 0; w < kGroupWarps; ++w) {
+        const float mw = m_s[w * GP + g];
+        f[w] = (mw == -CUDART_INF_F) ? 0.f : expf(mw - M);
+        L += l_s[w * GP + g] * f[w];
+      }
+      T* o = out + ((size_t)t * nq + hq) * Dv;
+      const T* gate = shape.gate ? static_cast<const T*>(shape.gate) + (size_t)t * shape.gate_ld + (size_t)hq * Dv : nullptr;
+      for (int i = lane; i < Dv; i += 32) {
+        float a = 0.f;
+        for (int w = 0; w < kGroupWarps; ++w) a += acc_s[(w * GP + g) * Dv + i] * f[w];
+        a = L > 0.f ? a / L * shape.out_scale : 0.f;
+        if (gate != nullptr) a *= 1.0f / (1.0f + expf(-to_f32(gate[i])));
+        o[i] = from_f32<T>(a);
+      }
     }
   }
 }
 
-template <typename T, int VPL, int GP>
+template <typename T, int VPL, int GP, bool PAIR>
 static int launch_group(const void* q, int q_row_stride, const void* pages, const int* block_table, int max_pages,
                         int page_size, int num_pages, const int* positions, const int* token_req, void* out, int T_,
                         int nq, int nkv, int Dk, float scale, int window, int keep_first, int one_more, int vec,
                         ScoreShape shape, int* status, cudaStream_t stream) {
   const size_t smem = ((size_t)GP * Dk + (size_t)kGroupWarps * GP * (VPL * 32 + 2)) * sizeof(float);
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(window_attention_group_kernel<T, VPL, GP>,
+    cudaError_t e = cudaFuncSetAttribute(window_attention_group_kernel<T, VPL, GP, PAIR>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  kvb_launch(window_attention_group_kernel<T, VPL, GP>, dim3(T_, nkv), dim3(kGroupWarps * 32), smem, stream, (const T*)q,
+  kvb_launch(window_attention_group_kernel<T, VPL, GP, PAIR>, dim3(T_, nkv), dim3(kGroupWarps * 32), smem, stream, (const T*)q,
              q_row_stride, (const T*)pages, block_table, max_pages, page_size, num_pages, positions, token_req, (T*)out, nq,
              nkv, Dk, scale, window, keep_first, one_more, vec, shape, status);
   return kvb_launch_result();
 }
 
-template <typename T, int VPL>
+template <typename T, int VPL, bool PAIR>
 static int launch_group_gp(int G, const void* q, int q_row_stride, const void* pages, const int* block_table,
                            int max_pages, int page_size, int num_pages, const int* positions, const int* token_req,
                            void* out, int T_, int nq, int nkv, int Dk, float scale, int window, int keep_first,
                            int one_more, int vec, ScoreShape shape, int* status, cudaStream_t stream) {
-#define KVB_WG(GP) return launch_group<T, VPL, GP>(q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, \
+#define KVB_WG(GP) return launch_group<T, VPL, GP, PAIR>(q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, \
                                                    positions, token_req, out, T_, nq, nkv, Dk, scale, window, keep_first, \
                                                    one_more, vec, shape, status, stream)
-  if (G == 1) KVB_WG(1);
+  if constexpr (!PAIR) {
+    if (G == 1) KVB_WG(1);
+  }
   if (G == 2) KVB_WG(2);
   if (G <= 4) KVB_WG(4);
   KVB_WG(8);
@@ -447,22 +523,34 @@ static int window_attention_any(const void* q, int q_row_stride, const void* pag
   if (shape.chunk < 0 || (shape.chunk > 0 && keep_first > 0) || (one_more && shape.sinks != nullptr)) return KVB_ERR_BAD_SIZE;
   const int esz = dtype == KVB_F32 ? 4 : 2;
   const int per16 = 16 / esz;
-  const int vec = (Dk % per16 == 0 && (Dk + Dv) % per16 == 0 && ((uintptr_t)pages % 16) == 0) ? 1 : 0;
-  // groups of up to 8 heads with values of 32, 64 or 128 channels: a block per key/value head, the rows read once
-  const int G = nq / nkv;
+  const int maps = shape.pair ? 2 : 1;
+  if (shape.pair && (one_more || shape.sinks != nullptr || shape.gate != nullptr)) return KVB_ERR_BAD_SIZE;
+  const int vec = (Dk % per16 == 0 && (maps * Dk + Dv) % per16 == 0 && ((uintptr_t)pages % 16) == 0) ? 1 : 0;
+  // groups of up to 8 heads (4 with two maps) with values of 32, 64 or 128 channels: a block per key/value head, the
+  // rows read once
+  const int G = nq / nkv * maps;
   if (G <= kMaxGroup && (Dv == 32 || Dv == 64 || Dv == 128) && vec) {
-#define KVB_WV(VPL)                                                                                                     \
-  KVB_DISPATCH_DTYPE(dtype, T, return (launch_group_gp<T, VPL>(G, q, q_row_stride, pages, block_table, max_pages,      \
-                                                               page_size, num_pages, positions, token_req, out, T_, nq, \
-                                                               nkv, Dk, scale, window, keep_first, one_more, vec,      \
-                                                               shape, status, stream)))
+#define KVB_WP(VPL, PAIR)                                                                                              \
+  KVB_DISPATCH_DTYPE(dtype, T, return (launch_group_gp<T, VPL, PAIR>(G, q, q_row_stride, pages, block_table, max_pages, \
+                                                                     page_size, num_pages, positions, token_req, out,  \
+                                                                     T_, nq, nkv, Dk, scale, window, keep_first,       \
+                                                                     one_more, vec, shape, status, stream)))
+#define KVB_WV(VPL) { if (shape.pair) { KVB_WP(VPL, true); } else { KVB_WP(VPL, false); } }
     if (Dv == 32) { KVB_WV(1); }
     if (Dv == 64) { KVB_WV(2); }
     if (Dv == 128) { KVB_WV(4); }
 #undef KVB_WV
+#undef KVB_WP
   }
   dim3 grid(T_, nq);
-  KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(window_attention_kernel<T>, grid, dim3(kWarps * 32), 0, stream, (const T*)q,
+  if (shape.pair) {
+    KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(window_attention_kernel<T, true>, grid, dim3(2 * kWarps * 32), 0, stream,
+                                              (const T*)q, q_row_stride, (const T*)pages, block_table, max_pages, page_size,
+                                              num_pages, positions, token_req, (T*)out, nq, nkv, Dk, Dv, scale, window,
+                                              keep_first, one_more, vec, shape, status)));
+    return kvb_launch_result();
+  }
+  KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(window_attention_kernel<T, false>, grid, dim3(kWarps * 32), 0, stream, (const T*)q,
                                             q_row_stride, (const T*)pages, block_table, max_pages, page_size, num_pages,
                                             positions, token_req, (T*)out, nq, nkv, Dk, Dv, scale, window, keep_first,
                                             one_more, vec, shape, status)));
@@ -509,6 +597,18 @@ KVB_EXPORT int kvb_window_attention_masked(const void* q, int q_row_stride, cons
                               out, T_, nq, nkv, Dk, Dv, scale, window, keep_first, one_more, shape, dtype, status, stream);
 }
 
+// Two maps per head over the same values (see ScoreShape): q holds nq heads of two queries of Dk each, a cached row is
+// [k1 | k2 | v] (2 Dk + Dv); out[t, h] = (a1 - pair_weight * a2) / rms * out_scale.
+KVB_EXPORT int kvb_window_attention_pair(const void* q, int q_row_stride, const void* pages, const int* block_table,
+                                         int max_pages, int page_size, int num_pages, const int* positions,
+                                         const int* token_req, void* out, int T_, int nq, int nkv, int Dk, int Dv,
+                                         float scale, int window, int chunk, float pair_weight, float pair_eps,
+                                         float out_scale, int dtype, int* status, cudaStream_t stream) {
+  ScoreShape shape = {nullptr, nullptr, 0.f, out_scale, nullptr, chunk, nullptr, 0, 1, pair_weight, pair_eps};
+  return window_attention_any(q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, positions, token_req,
+                              out, T_, nq, nkv, Dk, Dv, scale, window, 0, 0, shape, dtype, status, stream);
+}
+
 // ---------------------------------------------------------------- biases, norms over the whole projection, rotation, cache write
 // src [T, ld] holds, per token, nq queries of Dk from column 0, nkv keys of Dk from k_off and nkv values of Dv from
 // v_off, as a product left them.  Each gets its bias (float32, may be null).  With qw (float32 [nq * Dk]) all of a
@@ -517,7 +617,8 @@ KVB_EXPORT int kvb_window_attention_masked(const void* q, int q_row_stride, cons
 // head turn by the token's position: channel pair i is (i, i + rot / 2) with layout 0 and (2 i, 2 i + 1) with layout
 // 1, and (u, v) becomes (u c - v s, v c + u s) with c = cos_t[pos][i], s = sin_t[pos][i] (float32 tables of
 // table_len rows, rot / 2 wide; any factor on the rotation is in the tables).  Queries go to q_out [T, nq * Dk];
-// keys and values into the request's pages, a row [key | value] per token and key/value head.  One block per token;
+// keys and values into the request's pages, a row [key | value] per token and key/value head; with maps == 2 a
+// key/value head has two keys, one behind the other in src and in its row (nq then counts queries, two per head).  One block per token;
 // the token's queries and keys wait in shared memory as float32 between the steps.
 struct QkRotArgs {
   const void* src; int ld, k_off, v_off;
@@ -529,6 +630,7 @@ struct QkRotArgs {
   const int* positions; const int* token_req;
   int nq, nkv, Dk, Dv, write;
   int* status;
+  int maps;
 };
 
 __device__ __forceinline__ float turned(const float* x, int d, int rot, int layout, const float* c, const float* s) {
@@ -549,7 +651,8 @@ __global__ void __launch_bounds__(256) qk_rot_append_kernel(QkRotArgs a) {
   pdl_wait();
   const int t = blockIdx.x;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int nQ = a.nq * a.Dk, nK = a.nkv * a.Dk, nV = a.nkv * a.Dv;
+  const int kw = a.maps * a.Dk;               // channels of a key/value head's keys
+  const int nQ = a.nq * a.Dk, nK = a.nkv * kw, nV = a.nkv * a.Dv;
   float* ks = qk_s + nQ;
   const T* row = static_cast<const T*>(a.src) + (size_t)t * a.ld;
   const int pos = a.positions[t];
@@ -604,15 +707,15 @@ __global__ void __launch_bounds__(256) qk_rot_append_kernel(QkRotArgs a) {
     return;
   }
   T* pages = static_cast<T*>(a.pages);
-  const int row_len = a.Dk + a.Dv;
+  const int row_len = kw + a.Dv;
   for (int i = threadIdx.x; i < nK; i += blockDim.x) {
-    const int head = i / a.Dk, d = i - head * a.Dk;
-    pages[(((size_t)page * a.nkv + head) * a.page_size + (pos % a.page_size)) * row_len + d] =
-        from_f32<T>(turned(ks + head * a.Dk, d, rot, a.layout, c, s));
+    const int head = i / kw, at = i - head * kw, first = at / a.Dk * a.Dk;
+    pages[(((size_t)page * a.nkv + head) * a.page_size + (pos % a.page_size)) * row_len + at] =
+        from_f32<T>(turned(ks + head * kw + first, at - first, rot, a.layout, c, s));
   }
   for (int i = threadIdx.x; i < nV; i += blockDim.x) {
     const int head = i / a.Dv, d = i - head * a.Dv;
-    pages[(((size_t)page * a.nkv + head) * a.page_size + (pos % a.page_size)) * row_len + a.Dk + d] =
+    pages[(((size_t)page * a.nkv + head) * a.page_size + (pos % a.page_size)) * row_len + kw + d] =
         from_f32<T>(to_f32(row[a.v_off + i]) + (a.bv ? a.bv[i] : 0.f));
   }
 }
@@ -621,10 +724,11 @@ __global__ void __launch_bounds__(256) qk_rot_append_kernel(QkRotArgs a) {
 KVB_EXPORT int kvb_qk_rot_append(const QkRotArgs* args, int T_, int dtype, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   const QkRotArgs a = *args;
+  if (a.maps < 1 || a.maps > 2) return KVB_ERR_BAD_SIZE;
   if (a.Dk > kMaxDim || a.Dv > kMaxDim || a.Dk < 1 || a.Dv < 1 || a.nkv < 1 || a.nq < 1) return KVB_ERR_BAD_SIZE;
   if (a.rot < 0 || a.rot > a.Dk || (a.rot & 1) || a.layout < 0 || a.layout > 1) return KVB_ERR_BAD_SIZE;
   if (a.rot > 0 && (a.cos_t == nullptr || a.sin_t == nullptr)) return KVB_ERR_BAD_SIZE;
-  const size_t smem = (size_t)(a.nq + a.nkv) * a.Dk * sizeof(float);
+  const size_t smem = (size_t)(a.nq + a.nkv * a.maps) * a.Dk * sizeof(float);
   if (smem > 192 * 1024) return KVB_ERR_BAD_SIZE;
   KVB_DISPATCH_DTYPE(dtype, T, {
     if (smem > 48 * 1024) {

@@ -10,6 +10,9 @@
 // (each step optional), the mask (j <= i and (i - j < window or j < keep_first); or, by blocks of positions counted
 // from the sequence's start, j <= i and i / chunk == j / chunk) and the running max/sum softmax, whose denominator may
 // count a learned score per head once, without a value; the result may be multiplied by the sigmoid of a gate.
+// With two maps per head (ScoreShape::pair) the lower half of a tile's rows are map 1 of its (token, head) pairs and the
+// upper half map 2 of the same ones, so that a warp's sixteen rows all read the same keys; a head's two results meet in
+// shared memory at the end.
 // Key size dk and value size dv are multiples of 8 up to 128; the tiles are padded with zeros to the next of
 // 64 / 128 (keys) and 32 / 64 / 128 (values), which changes no sum.
 #include "common.cuh"
@@ -28,8 +31,8 @@ constexpr float kLog2e = 1.4426950408889634f;
 struct TileDesc { int req, t0, n_tok, pad; };
 
 struct RowsArgs {
-  const __nv_bfloat16* q; int q_row_stride;          // [T, >= nq * dk]
-  const __nv_bfloat16* pages;                        // [num_pages, nkv, page_size, dk + dv]
+  const __nv_bfloat16* q; int q_row_stride;          // [T, >= nq * maps * dk]
+  const __nv_bfloat16* pages;                        // [num_pages, nkv, page_size, maps * dk + dv]
   const int* block_table; int max_pages, page_shift, num_pages;
   const int* positions; const TileDesc* tiles;
   __nv_bfloat16* out;                                // [T, nq * dv]
@@ -41,18 +44,19 @@ struct RowsArgs {
 
 // KS: k-steps of 16 key channels (the padded key size is KS * 16); DP: pairs of 8 value channels (the padded
 // value size is DP * 16); NW: warps, 16 query rows each.
-template <int KS, int DP, int NW>
+template <int KS, int DP, int NW, bool PAIR>
 __global__ void __launch_bounds__(NW * 32)
 window_flash_attention_kernel(RowsArgs p) {
   constexpr int BM = NW * 16;
+  constexpr int MAPS = PAIR ? 2 : 1, MROWS = BM / MAPS;   // rows of one map
   constexpr int kThreads = NW * 32;
   constexpr int KC = KS * 2, VC = DP * 2;                 // 16-byte chunks of a padded key / value row
   constexpr int PK = (KC + 7) / 8 * 128, PV = (VC + 7) / 8 * 128;      // bytes from row to row in shared memory
   constexpr int DT = DP * 2;                              // n-tiles of the output
   extern __shared__ __align__(128) unsigned char smem[];
   unsigned char* q_s = smem;                              // [BM] rows of PK bytes
-  unsigned char* k_s = q_s + BM * PK;                     // [2][BN] rows of PK bytes
-  unsigned char* v_s = k_s + 2 * BN * PK;                 // [2][BN] rows of PV bytes
+  unsigned char* k_s = q_s + BM * PK;                     // [2][MAPS][BN] rows of PK bytes
+  unsigned char* v_s = k_s + 2 * MAPS * BN * PK;          // [2][BN] rows of PV bytes
   int* row_pos = reinterpret_cast<int*>(v_s + 2 * BN * PV);            // [BM] position of each row's token, -1 if none
 
   pdl_trigger();
@@ -64,10 +68,11 @@ window_flash_attention_kernel(RowsArgs p) {
   const int G = p.G, gp_shift = p.gp_shift, gp = 1 << gp_shift;
   const int page_mask = (1 << p.page_shift) - 1;
   const int* table = p.block_table + (size_t)tile.req * p.max_pages;
-  const int dk = p.dk, dv = p.dv, row_len = dk + dv, window = p.window;
+  const int dk = p.dk, dv = p.dv, v_at = MAPS * dk, row_len = v_at + dv, window = p.window;
 
   if (tid < BM) {
-    const int ti = tid >> gp_shift, hi = tid & (gp - 1);
+    const int mr = tid % MROWS;
+    const int ti = mr >> gp_shift, hi = mr & (gp - 1);
     row_pos[tid] = (ti < tile.n_tok && hi < G) ? p.positions[tile.t0 + ti] : -1;
   }
   const int pos_first = p.positions[tile.t0];
@@ -84,17 +89,18 @@ window_flash_attention_kernel(RowsArgs p) {
   auto load_q = [&]() {
     for (int c = tid; c < BM * KC; c += kThreads) {
       const int row = c / KC, part = c - row * KC;
-      const int ti = row >> gp_shift, hi = row & (gp - 1);
+      const int mr = row % MROWS, map = row / MROWS;
+      const int ti = mr >> gp_shift, hi = mr & (gp - 1);
       const bool ok = ti < tile.n_tok && hi < G && part * 8 < dk;
       const __nv_bfloat16* src = p.q + (size_t)(tile.t0 + (ok ? ti : 0)) * p.q_row_stride +
-                                 (size_t)(hk * G + (ok ? hi : 0)) * dk + (ok ? part * 8 : 0);
+                                 (size_t)((hk * G + (ok ? hi : 0)) * MAPS + map) * dk + (ok ? part * 8 : 0);
       cp_async_16_zfill(q_s + swz_pitch<PK>(row, part), src, ok);
     }
   };
   // A key's row [key | value] is copied by kThreads / BN threads, so that its page is looked up once per thread and tile.
   auto load_kv = [&](int t, int buf) {
     constexpr int TPK = kThreads / BN;
-    unsigned char* kd = k_s + buf * BN * PK;
+    unsigned char* kd = k_s + buf * MAPS * BN * PK;
     unsigned char* vd = v_s + buf * BN * PV;
     const int key = tid / TPK, sub = tid % TPK;
     const int j = t * BN + key;
@@ -111,14 +117,17 @@ window_flash_attention_kernel(RowsArgs p) {
       }
     }
 #pragma unroll
-    for (int c = sub; c < KC; c += TPK) {
-      const bool have = ok && c * 8 < dk;
-      cp_async_16_zfill(kd + swz_pitch<PK>(key, c), p.pages + off + (have ? c * 8 : 0), have);
+    for (int map = 0; map < MAPS; ++map) {
+#pragma unroll
+      for (int c = sub; c < KC; c += TPK) {
+        const bool have = ok && c * 8 < dk;
+        cp_async_16_zfill(kd + map * BN * PK + swz_pitch<PK>(key, c), p.pages + off + (have ? map * dk + c * 8 : 0), have);
+      }
     }
 #pragma unroll
     for (int c = sub; c < VC; c += TPK) {
       const bool have = ok && c * 8 < dv;
-      cp_async_16_zfill(vd + swz_pitch<PV>(key, c), p.pages + off + (have ? dk + c * 8 : 0), have);
+      cp_async_16_zfill(vd + swz_pitch<PV>(key, c), p.pages + off + (have ? v_at + c * 8 : 0), have);
     }
   };
 
@@ -165,7 +174,7 @@ window_flash_attention_kernel(RowsArgs p) {
       lo_r[0] = first_seen_key(pos_r[0], window, p.shape.chunk);
       lo_r[1] = first_seen_key(pos_r[1], window, p.shape.chunk);
     }
-    const unsigned char* kt = k_s + buf * BN * PK;
+    const unsigned char* kt = k_s + (buf * MAPS + (PAIR ? warp / (NW / 2) : 0)) * BN * PK;
     const unsigned char* vt = v_s + buf * BN * PV;
 
     // S = Q K^T : 16 rows x 64 keys per warp
@@ -251,6 +260,41 @@ window_flash_attention_kernel(RowsArgs p) {
     l_run[rr] += __shfl_xor_sync(0xffffffffu, l_run[rr], 1);
     l_run[rr] += __shfl_xor_sync(0xffffffffu, l_run[rr], 2);
   }
+  if constexpr (PAIR) {
+    // every row's result goes to shared memory (the tiles are used up); then four threads per (token, head) take the
+    // difference of its two rows, the sum of its squares and the norm
+    constexpr int OP = DP * 16 + 4;                       // floats from row to row
+    float* o_s = reinterpret_cast<float*>(smem);
+#pragma unroll
+    for (int rr = 0; rr < 2; ++rr) {
+      const float inv = l_run[rr] > 0.f ? 1.0f / l_run[rr] : 0.f;
+      float* dst = o_s + (r0 + rr * 8) * OP + ((lane & 3) << 1);
+#pragma unroll
+      for (int n = 0; n < DT; ++n)
+        *reinterpret_cast<float2*>(dst + n * 8) = make_float2(o[n][rr * 2] * inv, o[n][rr * 2 + 1] * inv);
+    }
+    __syncthreads();
+    constexpr int TPR = kThreads / MROWS;                 // 4
+    const int mr = tid / TPR, sub = tid % TPR;
+    const int ti = mr >> gp_shift, hi = mr & (gp - 1);
+    const float* a1 = o_s + mr * OP;
+    const float* a2 = a1 + MROWS * OP;
+    float ss = 0.f;
+    for (int i = sub * 2; i < dv; i += TPR * 2) {
+      const float x = a1[i] - p.shape.pair_weight * a2[i], y = a1[i + 1] - p.shape.pair_weight * a2[i + 1];
+      ss = fmaf(x, x, ss);
+      ss = fmaf(y, y, ss);
+    }
+    ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+    ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+    if (ti >= tile.n_tok || hi >= G) return;
+    const float f = p.shape.out_scale / sqrtf(ss / (float)dv + p.shape.pair_eps);
+    __nv_bfloat16* dst = p.out + ((size_t)(tile.t0 + ti) * p.nq + hk * G + hi) * dv;
+    for (int i = sub * 2; i < dv; i += TPR * 2)
+      *reinterpret_cast<unsigned*>(dst + i) = pack_bf16((a1[i] - p.shape.pair_weight * a2[i]) * f,
+                                                        (a1[i + 1] - p.shape.pair_weight * a2[i + 1]) * f);
+    return;
+  }
 #pragma unroll
   for (int rr = 0; rr < 2; ++rr) {
     const int row = r0 + rr * 8;
@@ -286,25 +330,32 @@ window_flash_attention_kernel(RowsArgs p) {
   }
 }
 
-template <int KS, int DP, int NW>
+template <int KS, int DP, int NW, bool PAIR>
 int launch(const RowsArgs& a, int num_tiles, cudaStream_t stream) {
   constexpr int BM = NW * 16;
   constexpr int PK = (KS * 2 + 7) / 8 * 128, PV = (DP * 2 + 7) / 8 * 128;
-  const size_t smem = (size_t)BM * PK + 2 * (size_t)BN * (PK + PV) + BM * sizeof(int);
+  const size_t smem = (size_t)BM * PK + 2 * (size_t)BN * (PK * (PAIR ? 2 : 1) + PV) + BM * sizeof(int);
+  static_assert(!PAIR || BM * (DP * 16 + 4) * 4 <= BM * PK + 2 * BN * (2 * PK + PV), "the rows' results fit the used-up tiles");
   if (smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(window_flash_attention_kernel<KS, DP, NW>,
+    cudaError_t e = cudaFuncSetAttribute(window_flash_attention_kernel<KS, DP, NW, PAIR>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  kvb_launch(window_flash_attention_kernel<KS, DP, NW>, dim3(num_tiles, a.nkv), dim3(NW * 32), smem, stream, a);
+  kvb_launch(window_flash_attention_kernel<KS, DP, NW, PAIR>, dim3(num_tiles, a.nkv), dim3(NW * 32), smem, stream, a);
   return kvb_launch_result();
 }
 
-template <int KS, int NW>
+template <int KS, int NW, bool PAIR>
 int launch_dv(const RowsArgs& a, int num_tiles, cudaStream_t stream) {
-  if (a.dv <= 32) return launch<KS, 2, NW>(a, num_tiles, stream);
-  if (a.dv <= 64) return launch<KS, 4, NW>(a, num_tiles, stream);
-  return launch<KS, 8, NW>(a, num_tiles, stream);
+  if (a.dv <= 32) return launch<KS, 2, NW, PAIR>(a, num_tiles, stream);
+  if (a.dv <= 64) return launch<KS, 4, NW, PAIR>(a, num_tiles, stream);
+  return launch<KS, 8, NW, PAIR>(a, num_tiles, stream);
+}
+
+template <bool PAIR>
+int launch_any(const RowsArgs& a, int num_tiles, int wide, cudaStream_t stream) {
+  if (a.dk <= 64) return wide ? launch_dv<4, 8, PAIR>(a, num_tiles, stream) : launch_dv<4, 4, PAIR>(a, num_tiles, stream);
+  return wide ? launch_dv<8, 8, PAIR>(a, num_tiles, stream) : launch_dv<8, 4, PAIR>(a, num_tiles, stream);
 }
 
 int log2_exact(int x) {
@@ -321,6 +372,30 @@ KVB_EXPORT int kvb_window_flash_attention_supported(int dk, int dv, int group, i
   return dk >= 8 && dk <= 128 && dk % 8 == 0 && dv >= 8 && dv <= 128 && dv % 8 == 0 && group >= 1 && group <= 64 &&
          log2_exact(page_size) >= 0;
 }
+
+namespace {
+
+int fill_args(RowsArgs& a, const void* q, int q_row_stride, const void* pages, const int* block_table, int max_pages,
+              int page_size, int num_pages, const int* positions, const void* tiles, void* out, int nq, int nkv, int dk,
+              int dv, float scale, int* status) {
+  const int G = nq / nkv;
+  if (!kvb_window_flash_attention_supported(dk, dv, G, page_size)) return KVB_ERR_BAD_SIZE;
+  if ((reinterpret_cast<uintptr_t>(q) & 15) || (q_row_stride & 7) || (reinterpret_cast<uintptr_t>(pages) & 15))
+    return KVB_ERR_ALIGN;
+  a.q = static_cast<const __nv_bfloat16*>(q); a.q_row_stride = q_row_stride;
+  a.pages = static_cast<const __nv_bfloat16*>(pages);
+  a.block_table = block_table; a.max_pages = max_pages; a.page_shift = log2_exact(page_size); a.num_pages = num_pages;
+  a.positions = positions; a.tiles = static_cast<const TileDesc*>(tiles);
+  a.out = static_cast<__nv_bfloat16*>(out);
+  a.nq = nq; a.nkv = nkv; a.G = G; a.dk = dk; a.dv = dv;
+  a.gp_shift = 0;
+  while ((1 << a.gp_shift) < G) ++a.gp_shift;
+  a.scale = scale; a.window = 0; a.keep_first = 0; a.one_more = 0;
+  a.status = status;
+  return 0;
+}
+
+}  // namespace
 
 // tiles: num_tiles x {request row, first token row, tokens, 0}, int32; a tile holds consecutive tokens of one
 // request, positions ascending, at most (wide ? 128 : 64) / (the group padded to a power of two) of them.
@@ -339,24 +414,31 @@ KVB_EXPORT int kvb_window_flash_attention_masked(const void* q, int q_row_stride
   if (num_tiles <= 0) return 0;
   if (nkv < 1 || nkv > 65535 || nq % nkv || window < 0 || keep_first < 0 || softcap < 0.f) return KVB_ERR_BAD_SIZE;
   if (chunk < 0 || (chunk > 0 && keep_first > 0) || (one_more && sinks != nullptr)) return KVB_ERR_BAD_SIZE;
-  const int G = nq / nkv;
-  if (!kvb_window_flash_attention_supported(dk, dv, G, page_size)) return KVB_ERR_BAD_SIZE;
-  if ((reinterpret_cast<uintptr_t>(q) & 15) || (q_row_stride & 7) || (reinterpret_cast<uintptr_t>(pages) & 15))
-    return KVB_ERR_ALIGN;
   RowsArgs a;
-  a.q = static_cast<const __nv_bfloat16*>(q); a.q_row_stride = q_row_stride;
-  a.pages = static_cast<const __nv_bfloat16*>(pages);
-  a.block_table = block_table; a.max_pages = max_pages; a.page_shift = log2_exact(page_size); a.num_pages = num_pages;
-  a.positions = positions; a.tiles = static_cast<const TileDesc*>(tiles);
-  a.out = static_cast<__nv_bfloat16*>(out);
-  a.nq = nq; a.nkv = nkv; a.G = G; a.dk = dk; a.dv = dv;
-  a.gp_shift = 0;
-  while ((1 << a.gp_shift) < G) ++a.gp_shift;
-  a.scale = scale; a.window = window; a.keep_first = keep_first; a.one_more = one_more;
+  const int rc = fill_args(a, q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, positions, tiles, out, nq,
+                           nkv, dk, dv, scale, status);
+  if (rc != 0) return rc;
+  a.window = window; a.keep_first = keep_first; a.one_more = one_more;
   a.shape = ScoreShape{head_scale, slopes, softcap, out_scale, sinks, chunk, gate, gate_ld};
-  a.status = status;
-  if (dk <= 64) return wide ? launch_dv<4, 8>(a, num_tiles, stream) : launch_dv<4, 4>(a, num_tiles, stream);
-  return wide ? launch_dv<8, 8>(a, num_tiles, stream) : launch_dv<8, 4>(a, num_tiles, stream);
+  return launch_any<false>(a, num_tiles, wide, stream);
+}
+
+// Two maps per head over the same values: q [T, >= 2 nq * dk] ([map 1 | map 2] head by head), pages rows [k1 | k2 | v]
+// (2 dk + dv); a tile holds at most (wide ? 64 : 32) / (the group padded to a power of two, at most 32) tokens.
+KVB_EXPORT int kvb_window_flash_attention_pair(const void* q, int q_row_stride, const void* pages, const int* block_table,
+                                               int max_pages, int page_size, int num_pages, const int* positions,
+                                               const void* tiles, int num_tiles, int wide, void* out, int nq, int nkv,
+                                               int dk, int dv, float scale, int window, int chunk, float pair_weight,
+                                               float pair_eps, float out_scale, int* status, cudaStream_t stream) {
+  if (num_tiles <= 0) return 0;
+  if (nkv < 1 || nkv > 65535 || nq % nkv || nq / nkv > 32 || window < 0 || chunk < 0) return KVB_ERR_BAD_SIZE;
+  RowsArgs a;
+  const int rc = fill_args(a, q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, positions, tiles, out, nq,
+                           nkv, dk, dv, scale, status);
+  if (rc != 0) return rc;
+  a.window = window;
+  a.shape = ScoreShape{nullptr, nullptr, 0.f, out_scale, nullptr, chunk, nullptr, 0, 1, pair_weight, pair_eps};
+  return launch_any<true>(a, num_tiles, wide, stream);
 }
 
 KVB_EXPORT int kvb_window_flash_attention(const void* q, int q_row_stride, const void* pages, const int* block_table,

@@ -44,6 +44,8 @@ class DecoderModel:
         # parts that stand in the schedule in front of a layer (the start of a pass through repeated layers)
         self.before = [make("stream", e.before) if e.before is not None else None for e in self.schedule]
         self.keeps_embedding = any(getattr(b, "needs_embedding", False) for b in self.before)
+        # stream parts that make something of the embedding's output once a step, by what they share it under
+        self.from_embedding = {b.embedding_key: b for b in self.before if hasattr(b, "from_embedding")}
 
     def cache_specs(self):
         """Per schedule entry: what its mixer asks of the cache, and whose cache it reads."""
@@ -74,12 +76,14 @@ class DecoderModel:
             # the residual is updated in place from the first layer on: what enters the stream again later is a copy
             embedded = ops.new(tuple(residual.shape), residual.dtype, residual.device)
             embedded.copy_(residual)
+        made = {key: part.from_embedding(residual) for key, part in self.from_embedding.items()}
         delta = None
         for i, entry in enumerate(self.schedule):
             if arena is not None:
                 arena.begin_layer()
             if self.before[i] is not None:
-                delta = self.before[i].forward(residual, delta, embedded)
+                b = self.before[i]
+                delta = b.forward(residual, delta, made[b.embedding_key] if hasattr(b, "from_embedding") else embedded)
             residual, delta = self.layers[entry.layer].forward(residual, delta, batch, cache.binding(i))
         if arena is not None:
             arena.end_layers()
@@ -96,14 +100,16 @@ class DecoderModel:
         width) in the compute precision, plus a fifth."""
         h, v = self.spec.hidden_size, self.spec.vocab_size
         copies = int(getattr(self.embedding, "stream_copies", 1))      # a residual stream kept as several copies
-        step = 4 * max_tokens * h * (copies + (1 if self.keeps_embedding else 0)) + max_logit_rows * 4 * (h + v) + (1 << 16)
+        copies += (1 if self.keeps_embedding else 0) + 2 * len(self.from_embedding)
+        step = 4 * max_tokens * h * copies + max_logit_rows * 4 * (h + v) + (1 << 16)
         per_layer = 0
+        entered = 3 * h if self.from_embedding else 0      # the stream's copy and the float32 product at the start of a pass
         for block in self.layers:
             widths = 0
             for part in getattr(block, "parts", {}).values():
                 declared = getattr(part, "activation_widths", None)
                 widths += sum(declared()) if declared is not None else 8 * h
-            per_layer = max(per_layer, widths or 32 * h)
+            per_layer = max(per_layer, (widths or 32 * h) + entered)
         esize = 4 if self.ctx.dtype == torch.float32 else 2
         layer = int(1.2 * esize * max_tokens * per_layer) + (1 << 16)
         return step, layer

@@ -201,17 +201,23 @@ def _need_cuda(*ts):
 # ------------------------------------------------------------------ elementwise
 
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, status: torch.Tensor,
-                 sampled: Optional[torch.Tensor] = None, scale: float = 1.0) -> torch.Tensor:
-    """float32 residual rows ``table[ids] * scale`` (the factor applied in float32).  With ``sampled`` (int32), an id ``-(1 + r)``
-    stands for ``sampled[r]``: a token that is still on the device."""
+                 sampled: Optional[torch.Tensor] = None, scale: float = 1.0, pos_table: Optional[torch.Tensor] = None,
+                 positions: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """float32 residual rows ``table[ids] * scale`` (the factor applied in float32), with ``pos_table`` (the table's type)
+    plus ``pos_table[positions]``.  With ``sampled`` (int32), an id ``-(1 + r)`` stands for ``sampled[r]``: a token that
+    is still on the device."""
     _need_cuda(table, ids, sampled)
+    assert pos_table is None or (pos_table.dtype == table.dtype and pos_table.is_contiguous()
+                                 and pos_table.shape[1] == table.shape[1] and positions is not None)
     assert sampled is None or (sampled.dtype == torch.int32 and sampled.is_contiguous())
     V, H = table.shape
     T = ids.numel()
     out = new((T, H), torch.float32, table.device)
     rc = lib("elementwise").kvb_embed_gather(_p(table), dtype_code(table.dtype), _p(ids), _p(sampled),
                                              c_int(0 if sampled is None else sampled.numel()), _p(out),
-                                             c_int(T), c_int(H), c_int(V), c_float(scale), _p(status), _stream())
+                                             c_int(T), c_int(H), c_int(V), c_float(scale), _p(pos_table),
+                                             _p(positions if pos_table is not None else None),
+                                             c_int(0 if pos_table is None else pos_table.shape[0]), _p(status), _stream())
     _check(rc, "embed_gather")
     return out
 
@@ -361,17 +367,18 @@ class PendingSum:
     branch outputs ``deltas`` [T, H] of the compute type (a layer whose mixer and feed-forward read
     the same normed input hands on both), float32 ``rows`` [T, H] (the embedding's output entering
     the stream again at the start of a repeated run of layers) and a float32 ``vector`` [H] added to
-    every row.  :func:`join_norm` adds them all and norms the sum in one kernel."""
-    __slots__ = ("deltas", "rows", "vector")
+    every row.  ``base`` (float32 [T, H]): what the stream becomes before anything joins it (a product over the stream
+    that takes its place), None: the stream as it is.  :func:`join_norm` adds them all and norms the sum in one kernel."""
+    __slots__ = ("deltas", "rows", "vector", "base")
 
-    def __init__(self, deltas=(), rows=None, vector=None):
+    def __init__(self, deltas=(), rows=None, vector=None, base=None):
         self.deltas = tuple(d for d in deltas if d is not None)
         assert len(self.deltas) <= 2
-        self.rows, self.vector = rows, vector
+        self.rows, self.vector, self.base = rows, vector, base
 
     def plus(self, rows=None, vector=None) -> "PendingSum":
         assert (rows is None or self.rows is None) and (vector is None or self.vector is None)
-        return PendingSum(self.deltas, self.rows if rows is None else rows, self.vector if vector is None else vector)
+        return PendingSum(self.deltas, self.rows if rows is None else rows, self.vector if vector is None else vector, self.base)
 
 
 def join_norm(resid: torch.Tensor, pending: Optional[PendingSum], kind: Optional[str], weight: Optional[torch.Tensor],
@@ -387,6 +394,8 @@ def join_norm(resid: torch.Tensor, pending: Optional[PendingSum], kind: Optional
     deltas = pending.deltas if pending is not None else ()
     e = pending.rows if pending is not None else None
     vec = pending.vector if pending is not None else None
+    base = pending.base if pending is not None else None
+    assert base is None or (base.dtype == torch.float32 and base.shape == resid.shape and base.is_contiguous())
     dt = deltas[0].dtype if deltas else (compute_dtype or out_dtype)
     for d in deltas:
         assert d.shape == resid.shape and d.is_contiguous() and d.dtype == dt
@@ -396,7 +405,7 @@ def join_norm(resid: torch.Tensor, pending: Optional[PendingSum], kind: Optional
     n = T if rows is None else rows.numel()
     out = new((n, H), out_dtype, resid.device) if kind is not None else None
     rc = lib("rowwise").kvb_join_norm(_p(resid), _p(deltas[0] if deltas else None), _p(deltas[1] if len(deltas) > 1 else None),
-                                      _p(e), _p(vec), _p(weight), c_int(NORM_KINDS[kind]), c_float(eps), _p(out),
+                                      _p(e), _p(vec), _p(base), _p(weight), c_int(NORM_KINDS[kind]), c_float(eps), _p(out),
                                       c_int(1 if out_dtype == torch.float32 else 0), _p(rows), c_int(n), c_int(H),
                                       c_int(dtype_code(dt)), _stream())
     _check(rc, "join_norm")
@@ -546,28 +555,36 @@ def latent_prep(d_in: torch.Tensor, q_rank: int, kv_off: int, rank: int, rot: in
 HEAD_GEMM_LIBRARY_MIN_ROWS = int(os.environ.get('KVB200_HEAD_GEMM_LIBRARY_MIN_ROWS', '128'))
 
 
-def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor) -> torch.Tensor:
+def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, gate=None) -> torch.Tensor:
     """A product per head: ``out[t, h, :] = w[h] @ x[t, first + h * head_stride : ... + K]`` with
-    ``w`` [H, N, K].  float32, and bfloat16 steps of fewer than 128 rows: this package's FMA kernel, float32
+    ``w`` [H, N, K].  ``gate``: (tensor, first column) of rows [T, H * N] by whose sigmoid the result is multiplied.  float32, and bfloat16 steps of fewer than 128 rows: this package's FMA kernel, float32
     sums in ascending k; bfloat16 with more rows: the library's batched product.  Returns [T, H * N]."""
     _need_cuda(x, w)
     H, N, K = w.shape
     assert w.is_contiguous() and w.dtype == x.dtype and x.stride(1) == 1
     out = new((x.shape[0], H * N), x.dtype, x.device)
     T = x.shape[0]
+    gate_at, gate_ld = 0, 0
+    if gate is not None:
+        gt, gcol = gate
+        assert gt.dtype == x.dtype and gt.stride(1) == 1 and gt.shape[0] == T and gt.shape[1] >= gcol + H * N
+        gate_at, gate_ld = _at(gt, gcol), gt.stride(0)
     if x.dtype == torch.bfloat16 and T >= HEAD_GEMM_LIBRARY_MIN_ROWS:
         # many rows: the library's batched product (tensor cores, float32 sums), as the other products of such steps
         xv = torch.as_strided(x, (H, T, K), (head_stride, x.stride(0), 1), x.storage_offset() + first)
         tmp = new((H, T, N), x.dtype, x.device)
         torch.bmm(xv, w.transpose(1, 2), out=tmp)
-        out.view(T, H, N).copy_(tmp.permute(1, 0, 2))
         if _marks is not None:
             _mark("head_gemm_library")
         choices["head_gemm_library"] += 1
+        rc = lib("latent_attention").kvb_head_rows(_p(tmp), _p(out), c_int(out.stride(0)), c_void_p(gate_at), c_int(gate_ld),
+                                                   c_int(T), c_int(H), c_int(N), _stream())
+        _check(rc, "head_rows")
         return out
     rc = lib("latent_attention").kvb_head_gemm(c_void_p(_at(x, first)), c_int(x.stride(0)), c_int(head_stride), _p(w),
                                                _p(out), c_int(out.stride(0)), c_int(N), c_int(x.shape[0]), c_int(N),
-                                               c_int(K), c_int(H), c_int(dtype_code(x.dtype)), _stream())
+                                               c_int(K), c_int(H), c_void_p(gate_at), c_int(gate_ld),
+                                               c_int(dtype_code(x.dtype)), _stream())
     _check(rc, "head_gemm")
     return out
 
@@ -617,14 +634,15 @@ def _query_tiles(batch, nt: int) -> torch.Tensor:
 
 
 def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_head_stride: int, cos, sin, rdims: int,
-                     pages: torch.Tensor, block_table, batch, sink: torch.Tensor, scale: float, heads: int,
+                     pages: torch.Tensor, block_table, batch, sink: Optional[torch.Tensor], scale: float, heads: int,
                      rank: int, rot: int) -> torch.Tensor:
     """Causal attention of every token over its request's cached rows [latent | rotated part],
-    all heads sharing the rows; softmax with a sink per head.  ``q_abs`` [T, heads * rank]: the
+    all heads sharing the rows; softmax with a sink per head (``sink`` None: without).  ``q_abs`` [T, heads * rank]: the
     queries' plain parts moved into the latent's space; ``q`` holds head h's part to be rotated at
     ``rot_first + h * q_head_stride``.  Returns the attended latents [T, heads * rank]."""
     _need_cuda(q_abs, pages)
-    assert q_abs.is_contiguous() and q.stride(1) == 1 and pages.is_contiguous() and sink.dtype == torch.float32
+    assert q_abs.is_contiguous() and q.stride(1) == 1 and pages.is_contiguous()
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == heads)
     T = q_abs.shape[0]
     out = new((T, heads * rank), q_abs.dtype, q_abs.device)
     if q_abs.dtype == torch.bfloat16 and LATENT_TC and latent_attention_tc_supported(rank, rot):
@@ -873,7 +891,7 @@ class _QkRotArgs(ctypes.Structure):
                 ("sin_t", c_void_p), ("table_len", c_int), ("rot", c_int), ("layout", c_int), ("q_out", c_void_p),
                 ("pages", c_void_p), ("block_table", c_void_p), ("max_pages", c_int), ("page_size", c_int),
                 ("num_pages", c_int), ("positions", c_void_p), ("token_req", c_void_p), ("nq", c_int), ("nkv", c_int),
-                ("Dk", c_int), ("Dv", c_int), ("write", c_int), ("status", c_void_p)]
+                ("Dk", c_int), ("Dv", c_int), ("write", c_int), ("status", c_void_p), ("maps", c_int)]
 
 
 ROTARY_LAYOUTS = {"half": 0, "pairs": 1}
@@ -881,18 +899,22 @@ ROTARY_LAYOUTS = {"half": 0, "pairs": 1}
 
 def qk_rot_append(p: torch.Tensor, first: int, k_off: int, v_off: int, bq, bk, bv, qw, kw, eps: float, cos, sin,
                   rot: int, layout: str, pages: torch.Tensor, block_table, batch, heads: int, kv_heads: int, dk: int,
-                  dv: int, write: bool = True) -> torch.Tensor:
+                  dv: int, write: bool = True, maps: int = 1) -> torch.Tensor:
     """From a product's rows to queries and cached rows.  ``p[:, first:]`` holds a token's ``heads`` queries of
     ``dk``, its ``kv_heads`` keys ``k_off`` columns further and its values ``v_off`` columns further.  Each gets its
     bias (float32 or None); with ``qw`` (float32 [heads * dk]) all queries of a token together are divided by their
     root mean square (``eps`` inside the root) and multiplied by ``qw``, likewise the keys with ``kw``; then the
     first ``rot`` channels of every query and key head turn by the token's position (``cos``, ``sin``: float32
     [positions, rot / 2]; ``layout`` "half": pair (i, i + rot / 2), "pairs": (2 i, 2 i + 1)).  Keys and values go
-    into the request's pages as rows [key | value].  Returns the queries [T, heads * dk]."""
+    into the request's pages as rows [key | value].  ``maps`` 2: every head has two queries and every key/value head two
+    keys (differential attention), one behind the other in ``p``; the rows are then [key 1 | key 2 | value].
+    Returns the queries [T, heads * maps * dk]."""
     _need_cuda(p, pages)
+    heads *= maps
     assert p.stride(1) == 1 and pages.is_contiguous() and pages.dtype == p.dtype
-    assert tuple(pages.shape[1:]) == (kv_heads, pages.shape[2], dk + dv)
-    for v, n in ((bq, heads * dk), (bk, kv_heads * dk), (bv, kv_heads * dv), (qw, heads * dk), (kw, kv_heads * dk)):
+    assert tuple(pages.shape[1:]) == (kv_heads, pages.shape[2], maps * dk + dv)
+    for v, n in ((bq, heads * dk), (bk, kv_heads * maps * dk), (bv, kv_heads * dv), (qw, heads * dk),
+                 (kw, kv_heads * maps * dk)):
         assert v is None or (v.dtype == torch.float32 and v.is_contiguous() and v.numel() == n)
     table_len = 0
     if rot:
@@ -904,7 +926,7 @@ def qk_rot_append(p: torch.Tensor, first: int, k_off: int, v_off: int, bq, bk, b
                    float(eps), cos.data_ptr() if rot else 0, sin.data_ptr() if rot else 0, table_len, int(rot),
                    ROTARY_LAYOUTS[layout], q.data_ptr(), pages.data_ptr(), block_table.data_ptr(), block_table.shape[1],
                    pages.shape[2], pages.shape[0], batch.positions.data_ptr(), batch.token_req.data_ptr(), heads, kv_heads,
-                   dk, dv, 1 if write else 0, batch.status.data_ptr())
+                   dk, dv, 1 if write else 0, batch.status.data_ptr(), maps)
     rc = lib("window_attention").kvb_qk_rot_append(ctypes.byref(a), c_int(T), c_int(dtype_code(p.dtype)), _stream())
     _check(rc, "qk_rot_append")
     return q
@@ -969,6 +991,47 @@ def window_flash_attention(q: torch.Tensor, pages: torch.Tensor, block_table, ba
         _stream())
     _check(rc, "window_flash_attention")
     choices["window_flash_attention"] += 1
+    return out
+
+
+def pair_attention(q: torch.Tensor, pages: torch.Tensor, block_table, batch, heads: int, kv_heads: int, dk: int, dv: int,
+                   scale: float, pair_weight: float, pair_eps: float, out_scale: float, window: int = 0, chunk: int = 0,
+                   tensor_cores: bool = False, wide: Optional[bool] = None) -> torch.Tensor:
+    """Differential attention: two maps per head over the same values.  ``q`` [T, heads * 2 * dk] ([map 1 | map 2] head by
+    head); ``pages`` [num_pages, kv_heads, page_size, 2 dk + dv] with rows [key 1 | key 2 | value].  Each map is a softmax
+    of its own under one mask (``window``, ``chunk`` as for :func:`window_attention`); a head's ``d = a1 - pair_weight *
+    a2`` is divided by its root mean square (``pair_eps`` inside the root) and multiplied by ``out_scale``, all in the
+    attention's launch.  ``tensor_cores``: the form of :func:`window_flash_attention` (bfloat16 steps with runs of query
+    tokens, sizes that :func:`window_flash_attention_supported` takes with twice the group).  Returns [T, heads * dv]."""
+    _need_cuda(q, pages)
+    assert q.stride(1) == 1 and pages.is_contiguous() and pages.dtype == q.dtype
+    assert tuple(pages.shape[1:]) == (kv_heads, pages.shape[2], 2 * dk + dv) and q.shape[1] >= 2 * heads * dk
+    T = q.shape[0]
+    out = new((T, heads * dv), q.dtype, q.device)
+    if tensor_cores:
+        group = 2 * (heads // kv_heads)
+        if wide is None:
+            wide = WINDOW_FLASH_WIDE
+        if wide is None:
+            wide = (T // rows_tokens_per_tile(group, True)) * kv_heads >= 2 * sm_count(q.device)
+        tiles = tiles_of_height(batch, rows_tokens_per_tile(group, bool(wide)))
+        rc = lib("window_flash_attention").kvb_window_flash_attention_pair(
+            _p(q), c_int(q.stride(0)), _p(pages), _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]),
+            c_int(pages.shape[0]), _p(batch.positions), _p(tiles), c_int(tiles.shape[0]), c_int(1 if wide else 0), _p(out),
+            c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv), c_float(scale), c_int(int(window or 0)),
+            c_int(int(chunk or 0)), c_float(pair_weight), c_float(pair_eps), c_float(out_scale), _p(batch.status), _stream())
+        _check(rc, "window_flash_attention")
+        choices["window_flash_attention"] += 1
+        choices["window_flash_attention_pair"] += 1
+        return out
+    rc = lib("window_attention").kvb_window_attention_pair(
+        _p(q), c_int(q.stride(0)), _p(pages), _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]),
+        c_int(pages.shape[0]), _p(batch.positions), _p(batch.token_req), _p(out), c_int(T), c_int(heads), c_int(kv_heads),
+        c_int(dk), c_int(dv), c_float(scale), c_int(int(window or 0)), c_int(int(chunk or 0)), c_float(pair_weight),
+        c_float(pair_eps), c_float(out_scale), c_int(dtype_code(q.dtype)), _p(batch.status), _stream())
+    _check(rc, "window_attention")
+    choices["window_attention"] += 1
+    choices["window_attention_pair"] += 1
     return out
 
 
@@ -1241,6 +1304,56 @@ def ssd_scan(xbc: torch.Tensor, dt, dt_bias: torch.Tensor, a_log: torch.Tensor, 
     return y
 
 
+class _LinearArgs(ctypes.Structure):
+    _fields_ = [("p", c_void_p), ("ld", c_int), ("q_off", c_int), ("f_off", c_int), ("v_off", c_int), ("f_bias", c_void_p),
+                ("lower", c_void_p), ("weight", c_void_p), ("eps", c_float), ("state", c_void_p), ("slot_stride", c_longlong),
+                ("y", c_void_p), ("out", c_void_p), ("q_start", c_void_p), ("req_start", c_void_p), ("slots", c_void_p),
+                ("H", c_int), ("N", c_int), ("Dv", c_int), ("cols", c_int), ("chunk", c_int), ("row_off", c_int),
+                ("local", c_void_p), ("carry", c_void_p), ("decay", c_void_p)]
+
+
+_linear_norms: Dict[tuple, bool] = {}
+
+
+def linear_scan(p: torch.Tensor, q_off: int, f_off: int, v_off: int, f_bias: torch.Tensor, lower: torch.Tensor,
+                weight: torch.Tensor, eps: float, state: torch.Tensor, batch, heads: int, n: int, dv: int) -> torch.Tensor:
+    """A memory ``S`` [n, dv] per head that decays per head and key channel, along every request's tokens of the step::
+
+        q = silu(zq),  f = lower + (1 - lower) sigmoid(zf + f_bias),  S <- diag(f) S + (1 - f) v^T,  o = S^T q
+
+    and each head's o divided by its root mean square (``eps`` inside the root), times ``weight`` (float32 [dv], shared by
+    the heads).  ``p`` [T, ...] holds zq (``heads * n`` from column ``q_off``), zf and v (``heads * dv``); ``f_bias`` and
+    ``lower`` float32 [heads * n].  ``state``: float32 [slots, >= heads * dv * n], zero for a request that starts at
+    position 0.  Returns [T, heads * dv] in ``p``'s type.  A step with a run of ``SCAN_CHUNK_MIN_RUN`` tokens or more walks
+    chunks of its runs side by side (64 tokens a chunk, 128 from runs of 1024 on)."""
+    _need_cuda(p, state)
+    T = p.shape[0]
+    assert p.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= heads * dv * n
+    for v, k in ((f_bias, heads * n), (lower, heads * n), (weight, dv)):
+        assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == k
+    out = new((T, heads * dv), p.dtype, p.device)
+    norms = _linear_norms.get((n, dv))
+    if norms is None:
+        norms = _linear_norms[(n, dv)] = bool(lib("linear_attention").kvb_linear_scan_norms(c_int(n), c_int(dv)))
+    y = 0 if norms else new((T, heads * dv), torch.float32, p.device).data_ptr()
+    max_run = int(getattr(batch, "max_q_len", 0) or 0)
+    chunk = first = local = carry = decay = 0
+    if max_run >= SCAN_CHUNK_MIN_RUN and not _capturing():
+        chunk = 128 if max_run >= 1024 else 64
+        rows, first = _chunk_rows(batch, chunk)
+        mats = new((2, rows, heads * dv * n), torch.float32, p.device)
+        decay_t = new((rows, heads * n), torch.float32, p.device)
+        local, carry, decay = mats[0].data_ptr(), mats[1].data_ptr(), decay_t.data_ptr()
+        choices["linear_scan_chunked"] += 1
+    a = _LinearArgs(p.data_ptr(), p.stride(0), q_off, f_off, v_off, f_bias.data_ptr(), lower.data_ptr(), weight.data_ptr(),
+                    float(eps), state.data_ptr(), state.stride(0), y, out.data_ptr(), batch.q_start.data_ptr(),
+                    batch.req_start.data_ptr(), batch.slots.data_ptr(), heads, n, dv, 0, chunk, first, local, carry, decay)
+    rc = lib("linear_attention").kvb_linear_scan(ctypes.byref(a), c_int(T), c_int(batch.num_reqs), c_int(max_run),
+                                                 c_int(dtype_code(p.dtype)), _stream())
+    _check(rc, "linear_scan")
+    return out
+
+
 class _MlstmArgs(ctypes.Structure):
     _fields_ = [("qkv", c_void_p), ("ld", c_int), ("q_off", c_int), ("k_off", c_int), ("v_off", c_int),
                 ("gates", c_void_p), ("ld_g", c_int), ("bi", c_void_p), ("bf", c_void_p), ("cap", c_float),
@@ -1378,12 +1491,14 @@ def expert_act(p: torch.Tensor, gate: torch.Tensor, experts: int, ff: int, share
 
 
 def limited_act(p: torch.Tensor, gate: torch.Tensor, shared_logit: Optional[torch.Tensor], experts: int, ff: int,
-                shared_ff: int, pad: int, limit: float, shared_limit: float, alpha: float) -> torch.Tensor:
+                shared_ff: int, pad: int, limit: float, shared_limit: float, alpha: float,
+                weigh_output: bool = False) -> torch.Tensor:
     """The activation of experts ``down(a(g) (u + 1))`` with ``g = min(w gate.h, limit)``, ``u = clamp(w up.h, +-limit)``,
     ``a(g) = g sigmoid(alpha g)`` and ``w`` the token's weight for the expert (``gate`` float32 [T, >= experts], 0 where
     not chosen).  ``p`` [T, 2 (experts ff + shared_ff)]: per expert its gate product, then its up product; behind
     them those of an expert that every token uses, whose result is multiplied by ``sigmoid(shared_logit[t])`` (float32
-    column, may be a strided view; None: by 1).  Returns [T, experts ff + shared_ff + pad], the padding zero."""
+    column, may be a strided view; None: by 1).  ``weigh_output``: the weight multiplies ``a(g) (u + 1)`` instead of the
+    two first products.  Returns [T, experts ff + shared_ff + pad], the padding zero."""
     _need_cuda(p, gate)
     assert p.stride(1) == 1 and gate.dtype == torch.float32 and gate.stride(1) == 1
     assert shared_logit is None or (shared_logit.dtype == torch.float32 and shared_logit.shape[0] == p.shape[0])
@@ -1392,8 +1507,8 @@ def limited_act(p: torch.Tensor, gate: torch.Tensor, shared_logit: Optional[torc
     rc = lib("experts").kvb_limited_act(_p(p), c_int(p.stride(0)), _p(gate), c_int(gate.stride(0)), _p(shared_logit),
                                         c_int(0 if shared_logit is None else shared_logit.stride(0)), _p(out),
                                         c_int(p.shape[0]), c_int(experts), c_int(ff), c_int(shared_ff), c_int(pad),
-                                        c_float(limit), c_float(shared_limit), c_float(alpha), c_int(dtype_code(p.dtype)),
-                                        _stream())
+                                        c_float(limit), c_float(shared_limit), c_float(alpha), c_int(1 if weigh_output else 0),
+                                        c_int(dtype_code(p.dtype)), _stream())
     _check(rc, "limited_act")
     return out
 

@@ -20,7 +20,9 @@ nothing of the model it sits in.  Interfaces by family:
   ``x`` as an ``ops.PendingNorm`` (see the prenorm block)
 * stream:        ``forward(residual, delta, embedded) -> delta``: stands in the schedule in front of a layer and
                  changes what is pending on the residual stream (``embedded``: the embedding's output,
-                 kept for the step when a stream part sets ``needs_embedding``)
+                 kept for the step when a stream part sets ``needs_embedding``; or what the part's
+                 ``from_embedding(residual)`` made of it at the step's start, once for all parts with the same
+                 ``embedding_key``)
 * embedding:     ``forward(batch) -> residual``  (float32 [T, hidden])
 * head:          ``forward(x) -> logits``  (float32 [rows, vocab])
 """

@@ -30,7 +30,7 @@ class PreNormBlock(Part):
     def __init__(self, parts):
         self.parts = dict(parts)
         self.mixer, self.mixer_norm = parts["mixer"], parts["mixer_norm"]
-        self.feed_forward, self.ff_norm = parts["feed_forward"], parts["ff_norm"]
+        self.feed_forward, self.ff_norm = parts.get("feed_forward"), parts.get("ff_norm")
         for part, norm in ((self.mixer, self.mixer_norm), (self.feed_forward, self.ff_norm)):
             if (getattr(part, "fuses_residual", False) and part.ctx.dtype == torch.bfloat16
                     and hasattr(norm, "give_up_weight") and norm.weight is not None):
@@ -46,12 +46,21 @@ class PreNormBlock(Part):
             a = self.mixer.forward(x, batch, cache, into=residual)
         else:
             a = self.mixer.forward(self.mixer_norm.forward(residual, delta), batch, cache)
+        if self.feed_forward is None:
+            return residual, a
         if getattr(self.feed_forward, "fuses_residual", False):
             x = self.ff_norm.forward(residual, a, lazy=True)
             f = self.feed_forward.forward(x, batch, into=residual)
         else:
             f = self.feed_forward.forward(self.ff_norm.forward(residual, a), batch)
         return residual, f
+
+
+@register("block", "prenorm_mixer_only")
+class PreNormMixerBlock(PreNormBlock):
+    """The pre-norm block of a layer that has no feed-forward: ``h += mixer(norm1(h))``."""
+
+    part_families = {"mixer": "mixer", "mixer_norm": "norm"}
 
 
 @register("block", "sandwich")

@@ -31,6 +31,26 @@ class TokenEmbedding(Part):
         return ops.embed_gather(self.table, batch.token_ids, batch.status, batch.sampled, self.scale)
 
 
+@register("embedding", "positioned_token_embedding")
+class PositionedTokenEmbedding(TokenEmbedding):
+    """``residual[t] = table[token[t]] * scale + position_table[position[t]]``: a learned vector per position joins the
+    looked-up row, which alone takes the factor; float32, in the gather's launch.
+    params: vocab_size, hidden_size, scale (1 when absent), positions (rows of the position table)."""
+
+    @classmethod
+    def weight_specs(cls, params):
+        return {"table": WeightSpec((params["vocab_size"], params["hidden_size"]), "matrix"),
+                "position_table": WeightSpec((params["positions"], params["hidden_size"]), "matrix")}
+
+    def __init__(self, params, weights, ctx):
+        super().__init__(params, weights, ctx)
+        self.position_table = weights["position_table"]
+
+    def forward(self, batch):
+        return ops.embed_gather(self.table, batch.token_ids, batch.status, batch.sampled, self.scale,
+                                self.position_table, batch.positions)
+
+
 @register("embedding", "normed_token_embedding")
 class NormedTokenEmbedding(TokenEmbedding):
     """``residual[t] = rmsnorm(table[token[t]]) * weight``: the looked-up row passes an RMS norm (float32,

@@ -100,20 +100,23 @@ class LimitedExperts(Part):
 
         g = min(W_gate x, limit),   u = clamp(W_up x, -limit, limit),   expert(x) = W_down (g sigmoid(alpha g) (u + 1)).
 
-    The router's logits ``W_r h`` are float32; the scores are their sigmoids, each by itself; the ``top`` experts with
-    the largest scores are chosen and weighted with their scores as they are.  The weight multiplies the expert's
-    *input*: the layer's output is the sum of ``expert(w h)`` over the chosen experts.  With ``shared_ff`` > 0 one more
+    The router's logits ``W_r h`` are float32.  ``score`` "sigmoid" (the default): the scores are their sigmoids, each by
+    itself; the ``top`` experts with the largest scores are chosen and weighted with their scores as they are.
+    "softmax_chosen": the ``top`` largest logits are chosen, and their weights are the softmax over the chosen alone.
+    ``weigh`` "input" (the default): the weight multiplies the expert's *input*, the layer's output is the sum of
+    ``expert(w h)`` over the chosen experts; "output": the sum of ``w expert(h)``.  With ``shared_ff`` > 0 one more
     expert of the same form (its own ``shared_limit``) runs for every token with weight 1, and its output is multiplied
     by ``sigmoid(w_sg . h)``, one number per token.
 
     All gate and up matrices are stacked into one matrix, expert after expert, and all down matrices side by side
     into another: a step is two products around an activation kernel.  Without biases ``W (w h) = w (W h)``, so the
-    kernel multiplies a chosen expert's two first products by the token's weight before it limits them, and writes 0
+    kernel multiplies a chosen expert's two first products by the token's weight before it limits them (weighed outputs:
+    the activation behind the limits, which a last matrix without bias hands through), and writes 0
     for an expert that was not chosen; the second product's float32 sums then add up exactly the chosen experts.  The
     shared expert's gate multiplies its activation, which for a last matrix without bias is the same as multiplying its
     output.  The router's rows and the shared gate's row are one small product with float32 results.  Every expert is
     computed for every token (see :class:`RoutedExperts` for what that costs).
-    params: hidden_size, experts, top, expert_ff, limit, shared_ff, shared_limit, alpha."""
+    params: hidden_size, experts, top, expert_ff, limit, shared_ff, shared_limit, alpha, score, weigh."""
 
     @classmethod
     def weight_specs(cls, params):
@@ -140,6 +143,10 @@ class LimitedExperts(Part):
         self.limit = float(params["limit"])
         self.shared_limit = float(params.get("shared_limit") or self.limit)
         self.alpha = float(params.get("alpha", 1.702))
+        self.score, self.weigh = str(params.get("score", "sigmoid")), str(params.get("weigh", "input"))
+        if self.score not in ("sigmoid", "softmax_chosen") or self.weigh not in ("input", "output"):
+            raise ValueError(f"limited_experts: score {self.score!r} (sigmoid, softmax_chosen) or weigh {self.weigh!r} "
+                             "(input, output) is not known")
         if not 1 <= self.top <= min(32, self.E):
             raise ValueError(f"limited_experts: {self.top} of {self.E} experts per token is refused (1 to 32)")
         first, second = [], []
@@ -165,8 +172,11 @@ class LimitedExperts(Part):
 
     def forward(self, x, batch):
         logits = ops.linear(x, self.small, out_dtype=torch.float32)
-        gate, _ = ops.route(x, None, None, self.E, 0, self.top, 1.0, logits, score="sigmoid", renormalize=False)
+        # a softmax over all experts, divided by the sum of the chosen, is the softmax over the chosen
+        chosen_only = self.score == "softmax_chosen"
+        gate, _ = ops.route(x, None, None, self.E, 0, self.top, 1.0, logits, score="softmax" if chosen_only else "sigmoid",
+                            renormalize=chosen_only)
         p = ops.linear(x, self.first)
         a = ops.limited_act(p, gate, logits[:, self.E] if self.S else None, self.E, self.F, self.S, self.pad, self.limit,
-                            self.shared_limit, self.alpha)
+                            self.shared_limit, self.alpha, weigh_output=self.weigh == "output")
         return ops.linear(a, self.down)

@@ -19,23 +19,28 @@ class LatentAttention(Part):
     ``c_q = rms(W_dq h) * w_dq`` and ``q = W_uq c_q``, per head ``dim`` plain dimensions followed by
     ``rot_dim`` rotated ones.  ``W_dkv h`` gives ``kv_rank`` rows that, RMS-normed, are the latent c,
     and ``rot_dim`` more that are one rotated key part shared by all heads.  Per head the plain key
-    is ``W_uk c`` and the value ``W_uv c``; score = (q_plain . k_plain + q_rot . k_rot) * scale; the
-    softmax's denominator also holds ``exp(sink_h)``.  Only [c | rotated part] is cached, one
+    is ``W_uk c`` and the value ``W_uv c``; score = (q_plain . k_plain + q_rot . k_rot) * scale; with ``sink`` (the
+    default) the softmax's denominator also holds ``exp(sink_h)``.  With ``gate`` the heads' results are multiplied
+    element by element by ``sigmoid(W_g h)``.  Only [c | rotated part] is cached, one
     row per token (a paged group of one plane).
 
     The key up-projection is applied to the queries instead (q_plain^T W_uk,h c = (W_uk,h^T q_plain)^T c),
     attention runs for all heads over the cached rows, and the value up-projection is applied
     to the attended latents; the output projection follows.
-    params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, eps, position (PartSpec)."""
+    params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, sink, gate, eps, position (PartSpec)."""
 
     @classmethod
     def weight_specs(cls, params):
         h, H, d, r, dv = (params[k] for k in ("hidden_size", "heads", "dim", "rot_dim", "vdim"))
         qr, kr = params["q_rank"], params["kv_rank"]
-        return {"dq": WeightSpec((qr, h)), "dq_norm": WeightSpec((qr,), "vector"), "uq": WeightSpec((H * (d + r), qr)),
+        specs = {"dq": WeightSpec((qr, h)), "dq_norm": WeightSpec((qr,), "vector"), "uq": WeightSpec((H * (d + r), qr)),
                 "dkv": WeightSpec((kr + r, h)), "dkv_norm": WeightSpec((kr,), "vector"),
-                "uk": WeightSpec((H * d, kr)), "uv": WeightSpec((H * dv, kr)), "sink": WeightSpec((H,), "bias"),
-                "o": WeightSpec((h, H * dv))}
+                "uk": WeightSpec((H * d, kr)), "uv": WeightSpec((H * dv, kr)), "o": WeightSpec((h, H * dv))}
+        if params.get("sink", True):
+            specs["sink"] = WeightSpec((H,), "bias")
+        if params.get("gate"):
+            specs["g"] = WeightSpec((H * dv, h))
+        return specs
 
     @classmethod
     def kernel_modules(cls, params, dtype):
@@ -50,9 +55,11 @@ class LatentAttention(Part):
             raise ValueError(f"latent_attention: a latent of {self.rank} is refused (up to 512)")
         if ctx.dtype == torch.bfloat16 and (self.rank + self.rot) % 2:
             raise ValueError("latent_attention: in bfloat16 the cached row (kv_rank + rot_dim) must be even")
-        self.w_in, (_, self.at_kv) = _stack([weights["dq"], weights["dkv"]], ctx.dtype)
+        mats = [weights["dq"], weights["dkv"]] + ([weights["g"]] if params.get("gate") else [])
+        self.w_in, starts = _stack(mats, ctx.dtype)
+        self.at_kv, self.at_g = starts[1], starts[2] if params.get("gate") else None
         self.dq_norm, self.dkv_norm = weights["dq_norm"], weights["dkv_norm"]
-        self.uq, self.o, self.sink = weights["uq"], weights["o"], weights["sink"]
+        self.uq, self.o, self.sink = weights["uq"], weights["o"], weights.get("sink")
         # per head: U_k^T [rank, dim] (absorbs the queries) and U_v [vdim, rank] (up-projects the attended latents)
         self.uk_t = weights["uk"].view(self.heads, self.dim, self.rank).transpose(1, 2).contiguous()
         self.uv = weights["uv"].view(self.heads, self.vdim, self.rank).contiguous()
@@ -91,4 +98,5 @@ class LatentAttention(Part):
         q_abs = ops.head_gemm(q, 0, per_head, self.uk_t)
         lat = ops.latent_attention(q_abs, q, self.dim, per_head, cos, sin, rdims, cache.k, table, batch, self.sink,
                                    self.scale, self.heads, self.rank, self.rot)
-        return ops.linear(ops.head_gemm(lat, 0, self.rank, self.uv), self.o)
+        gate = (d, self.at_g) if self.at_g is not None else None
+        return ops.linear(ops.head_gemm(lat, 0, self.rank, self.uv, gate), self.o)

@@ -14,15 +14,16 @@ class RMSNorm(Part):
     (upstream: base/src/kernels.cu:10-36), where ``v = residual + delta`` is summed
     and kept in float32 (upstream adds in a second kernel and keeps bfloat16,
     base/src/kernels.cu:38-43).  With ``scale`` (a constant on a branch, or on the logits behind the model's last
-    norm) the weight is multiplied by it once, when the model is built.
+    norm) the weight is multiplied by it once, when the model is built.  ``around_zero``: the stored weight is the factor
+    minus one (``y = v / rms * (1 + w)``); one is added once, when the model is built.
 
     The same part may stand behind a branch (``as_pending``): there it is not carried out at once but handed on as
     an :class:`ops.PostNormed`, and whoever brings the residual stream up to date next norms the branch output and
-    adds it in one kernel.  params: size, eps, scale."""
+    adds it in one kernel.  params: size, eps, scale, around_zero."""
 
     @classmethod
     def weight_specs(cls, params):
-        return {"weight": WeightSpec((params["size"],), "vector")}
+        return {"weight": WeightSpec((params["size"],), "bias" if params.get("around_zero") else "vector")}
 
     @classmethod
     def kernel_modules(cls, params, dtype):
@@ -33,6 +34,8 @@ class RMSNorm(Part):
         self.eps = float(params["eps"])
         self.size = int(params["size"])
         self.weight = weights["weight"]
+        if params.get("around_zero"):
+            self.weight = (self.weight + 1.0).contiguous()
         if params.get("scale") is not None and float(params["scale"]) != 1.0:
             self.weight = (self.weight * float(params["scale"])).contiguous()
 

@@ -1,11 +1,12 @@
 """Mixers whose state is a linear recurrence with a decay that depends on the token: a gated diagonal
-recurrence per channel, a matrix state per head with one decay per head (state-space duality), and a matrix
-memory per head with exponential gates and a running maximum (mLSTM).
+recurrence per channel, a matrix state per head with one decay per head (state-space duality), a matrix
+memory per head with exponential gates and a running maximum (mLSTM), and a linear attention whose memory decays
+per head and key channel (HGRN2).
 
 The first two make their projections in one product, pass part of it through a short causal convolution whose last
 inputs live in the request's state slot beside the recurrence's state (float32), and walk the request's
-tokens of the step in one kernel (csrc/kernels/recurrence.cu); the third has no convolution and its kernels are
-csrc/kernels/mlstm.cu.  A request that starts at position 0 starts from a zero state.
+tokens of the step in one kernel (csrc/kernels/recurrence.cu); the others have no convolution and their kernels are
+csrc/kernels/mlstm.cu and csrc/kernels/linear_attention.cu.  A request that starts at position 0 starts from a zero state.
 """
 
 from __future__ import annotations
@@ -210,3 +211,50 @@ class MatrixLSTM(Part):
         y = ops.mlstm_scan(p, self.at_q, self.at_k, self.at_v, gates, self.i_bias, self.f_bias, self.cap,
                            self.D ** -0.5, cache.state, batch, self.H, self.D, self.Dv)
         return ops.linear(ops.head_norm_gate(y, (p, self.at_g), self.norm, self.H, self.eps, self.ctx.dtype), self.o)
+
+
+@register("mixer", "decayed_linear_attention")
+class DecayedLinearAttention(Part):
+    """Linear attention in which the forget gate also decides what is written (HGRN2).  One product lays out
+    [q: heads * dim | f: heads * dim | v: heads * vdim].  Per head, with ``q = silu(q)`` and, channel by channel,
+    ``f = lower + (1 - lower) sigmoid(f + f_bias)`` (``lower``, ``f_bias``: learned, heads * dim numbers):
+
+        S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T   (S is dim x vdim),    o_t = S_t^T q_t,
+
+    from S = 0.  Every head's o is divided by its own root mean square (``eps`` inside the root) and multiplied by ``norm``
+    (``vdim`` numbers, the same for all heads); the heads, side by side, are projected by W_o.  Decays and the memory are
+    float32; the request's state slot holds the matrices.
+    params: hidden_size, heads, dim, vdim, eps."""
+
+    @classmethod
+    def weight_specs(cls, params):
+        h, H, D, Dv = (int(params[k]) for k in ("hidden_size", "heads", "dim", "vdim"))
+        return {"q": WeightSpec((H * D, h)), "f": WeightSpec((H * D, h)), "f_bias": WeightSpec((H * D,), "bias"),
+                "lower": WeightSpec((H * D,), "bias"), "v": WeightSpec((H * Dv, h)), "norm": WeightSpec((Dv,), "vector"),
+                "o": WeightSpec((h, H * Dv))}
+
+    @classmethod
+    def kernel_modules(cls, params, dtype):
+        return ("linear_attention",) + _gemm_modules(dtype)
+
+    def __init__(self, params, weights, ctx):
+        super().__init__(params, weights, ctx)
+        self.H, self.D, self.Dv = (int(params[k]) for k in ("heads", "dim", "vdim"))
+        self.eps = float(params["eps"])
+        if not 1 <= self.D <= 256:
+            raise ValueError(f"decayed_linear_attention: memories of {self.D} rows are refused (1 to 256)")
+        self.w_in, (self.at_q, self.at_f, self.at_v) = _stack([weights["q"], weights["f"], weights["v"]], ctx.dtype)
+        self.f_bias, self.lower, self.norm, self.o = weights["f_bias"], weights["lower"], weights["norm"], weights["o"]
+
+    def cache_spec(self):
+        return SlotStateSpec((self.H * self.Dv * self.D,), torch.float32)
+
+    def activation_widths(self):
+        inner = self.H * self.Dv
+        return [self.w_in.shape[0], 2 * inner, inner, self.o.shape[0]]
+
+    def forward(self, x, batch, cache):
+        p = ops.linear(x, self.w_in)
+        y = ops.linear_scan(p, self.at_q, self.at_f, self.at_v, self.f_bias, self.lower, self.norm, self.eps, cache.state,
+                            batch, self.H, self.D, self.Dv)
+        return ops.linear(y, self.o)

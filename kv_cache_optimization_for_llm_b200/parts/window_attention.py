@@ -1,12 +1,13 @@
 """Attention over a sliding window with one row [key | value] per token and key/value head in the pages: one whose
 queries, keys and values pass a short convolution first and whose window keeps the sequence's first tokens; one
 whose scores are shaped on their way to the softmax (a factor per head, a soft cap, a bias that grows with the
-distance); one that rotates queries and keys and masks by blocks of positions; and the arrangement of two mixers
-side by side."""
+distance); one that rotates queries and keys and masks by blocks of positions; one that subtracts two attention maps
+over the same values; and the arrangement of two mixers side by side."""
 
 from __future__ import annotations
 
 import dataclasses
+import math
 
 import torch
 
@@ -343,6 +344,96 @@ class RotaryChunkAttention(Part):
         if self.o_bias is not None:
             y = y + self.o_bias.to(y.dtype)
         return y
+
+
+@register("mixer", "differential_chunk_attention")
+class DifferentialChunkAttention(Part):
+    """Differential grouped-query attention over blocks of positions.
+
+    q (``heads`` x 2 x ``dim``), k (``kv_heads`` x 2 x ``dim``) and v (``kv_heads`` x ``vdim``) come from one product with the
+    row-stacked matrix; a head's rows are [map 1, map 2].  The first ``position.rotary_dim`` channels of every map of
+    every query and key head turn with the position (``position``: "rope_interleaved", or None).  Keys and values go to
+    the request's pages, a row [k1 | k2 | v] per token and key/value head.  Each map is an attention of its own over the
+    same values, ``s = (q . k) * scale``, query i seeing key j <= i only when ``i // chunk == j // chunk`` (blocks counted
+    from the sequence's start; ``chunk`` None: every key up to i), softmax in float32.  With a head's two results a1, a2
+
+        o = a1 - lam * a2,   lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff   (one number, made when the model is built),
+
+    o is divided by its root mean square over the head's ``vdim`` channels (``eps`` inside the root, no weight) and
+    multiplied by ``1 - diff``, in the attention's launch.  Then W_o.
+    params: hidden_size, heads, kv_heads, dim, vdim, scale, diff, chunk, eps, position."""
+
+    @classmethod
+    def weight_specs(cls, params):
+        h, H, G, D, Dv = (int(params[k]) for k in ("hidden_size", "heads", "kv_heads", "dim", "vdim"))
+        specs = {"q": WeightSpec((H * 2 * D, h)), "k": WeightSpec((G * 2 * D, h)), "v": WeightSpec((G * Dv, h)),
+                 "o": WeightSpec((h, H * Dv))}
+        specs.update({n: WeightSpec((D,), "bias") for n in ("lq1", "lk1", "lq2", "lk2")})
+        return specs
+
+    @classmethod
+    def kernel_modules(cls, params, dtype):
+        if dtype == torch.float32:
+            return ("window_attention", "gemm_f32")
+        flash = ("window_flash_attention",) if cls._flash_sizes(params, dtype) else ()
+        return ("window_attention",) + flash + ("gemm_bf16", "gemm_bf16_wide")
+
+    @staticmethod
+    def _flash_sizes(params, dtype, page_size=16):
+        # two rows of a tile per head: as many as a group of twice the heads
+        return ops.window_flash_attention_supported(int(params["dim"]), int(params["vdim"]),
+                                                    2 * (int(params["heads"]) // max(1, int(params["kv_heads"]))), page_size, dtype)
+
+    def __init__(self, params, weights, ctx):
+        super().__init__(params, weights, ctx)
+        self.heads, self.kv_heads = int(params["heads"]), int(params["kv_heads"])
+        self.dim, self.vdim = int(params["dim"]), int(params["vdim"])
+        if self.kv_heads < 1 or self.heads % self.kv_heads:
+            raise ValueError(f"differential_chunk_attention: {self.heads} query heads cannot be grouped over "
+                             f"{self.kv_heads} key/value heads")
+        if not (1 <= self.dim <= 256 and 1 <= self.vdim <= 256):
+            raise ValueError(f"differential_chunk_attention: head sizes {self.dim} x {self.vdim} are refused (1 to 256)")
+        self.scale, self.eps, self.diff = float(params["scale"]), float(params["eps"]), float(params["diff"])
+        self.chunk = int(params["chunk"]) if params.get("chunk") else None
+        dots = [float((weights["lq" + n].double() * weights["lk" + n].double()).sum()) for n in ("1", "2")]
+        self.lam = math.exp(dots[0]) - math.exp(dots[1]) + self.diff
+        self.w_in, (_, self.k_off, self.v_off) = _stack_rows([weights["q"], weights["k"], weights["v"]])
+        self.o = weights["o"]
+        pos = params.get("position")
+        self.position, self.rot = None, 0
+        if pos is not None:
+            if pos.kind != "rope_interleaved":
+                raise ValueError(f"differential_chunk_attention: a position encoding of kind {pos.kind!r} is not taken")
+            self.position = (ctx.make("position", pos) if ctx.make is not None
+                             else lookup("position", pos.kind)(pos.params, {}, ctx))
+            self.rot = int(self.position.rotary_dim)
+            if self.rot > self.dim:
+                raise ValueError(f"differential_chunk_attention: {self.rot} turning channels in maps of {self.dim}")
+
+    def cache_spec(self):
+        # a block never reaches further back than ``chunk`` keys: a windowed group of that size
+        return PagedKVSpec(self.kv_heads, 2 * self.dim + self.vdim, self.chunk, planes=1)
+
+    def activation_widths(self):
+        return [self.w_in.shape[0], 2 * self.heads * self.dim, self.heads * self.vdim, self.o.shape[0]]
+
+    def query_tile_heights(self):
+        if not self._flash_sizes(self.params, self.ctx.dtype):
+            return []
+        g = 2 * (self.heads // self.kv_heads)
+        return [ops.rows_tokens_per_tile(g, False), ops.rows_tokens_per_tile(g, True)]
+
+    def forward(self, x, batch, cache):
+        p = ops.linear(x, self.w_in)
+        table = batch.block_tables[cache.group]
+        cos, sin = self.position.tables() if self.rot else (None, None)
+        q = ops.qk_rot_append(p, 0, self.k_off, self.v_off, None, None, None, None, None, self.eps, cos, sin, self.rot,
+                              "pairs", cache.k, table, batch, self.heads, self.kv_heads, self.dim, self.vdim,
+                              write=cache.write, maps=2)
+        flash = not batch.decode_only and self._flash_sizes(self.params, self.ctx.dtype, cache.page_size)
+        a = ops.pair_attention(q, cache.k, table, batch, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.lam,
+                               self.eps, 1.0 - self.diff, chunk=self.chunk or 0, tensor_cores=flash)
+        return ops.linear(a, self.o)
 
 
 def _stack_rows(mats):
