@@ -480,6 +480,29 @@ def tevanex_config(z, chunk=1024):
             "max_position_embeddings": CONTEXT_LEN}
 
 
+def zatusun_config(z, chunk=1024):
+    """Six layers at the comparison's sizes: a linear attention with a decay per channel (heads of 64 x 64, the state of
+    Tevanex's matrix memory), a differential attention (half as many heads, two maps of 64 each over values of 128, a
+    quarter as many key/value heads: the projections of Tevanex's attention; every channel turning, blocks of 1024
+    positions) and a latent attention of Rezusun's sizes with an output gate; on every layer 32 experts of which a token
+    uses four, together as wide as Tevanex's experts with their shared one; the last three layers are a run that goes
+    through once."""
+    H = z["heads"]
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 32 + z["ff"] // 128, "limit": 7.0}, "router": {"experts": 32, "top": 4}}
+    lin = {"heads": H, "dim": 64, "vdim": 64}
+    att = {"heads": H // 2, "kv_heads": H // 8, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5, "mask": {"size": chunk},
+           "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["lat_rot"], "vdim": z["lat_vdim"], "q_rank": z["q_rank"],
+           "kv_rank": z["kv_rank"], "scale": (z["lat_dim"] + z["lat_rot"]) ** -0.5,
+           "rot": {"base": 10000.0, "dims": z["lat_rot"], "scaling": {"factor": 4.0, "original": 2048, "fast": 32.0, "slow": 1.0}}}
+    kinds = [("hgrn2", lin), ("attention", att), ("latent_attention", lat)]
+    n = z["layers"]
+    return {"architecture": "Zatusun", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "logit_softcap": 30.0, "max_positions": CONTEXT_LEN,
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe} for i in range(n)],
+            "loop": {"start": n // 2, "stop": n, "times": 1}}
+
+
 def llama_config_like(z):
     cfg = dict(LLAMA_1B)
     cfg.update(hidden_size=z["width"], intermediate_size=z["ff"], vocab_size=z["vocab"], num_hidden_layers=z["layers"],
@@ -792,6 +815,100 @@ def run_compare_tevanex(size):
             "kernel_roofline_fractions": kernels, "clocks": sampler.summary(list(_compare_windows) or [(w0, w1)])}
 
 
+def run_compare_zatusun(size):
+    """The Zatusun design beside Tevanex (the closest design on the engine: attention over blocks of positions in a
+    windowed page group, a matrix state per head in state slots, limited experts computed for every token) at equal
+    width, depth and vocabulary; the latent attention's kernels beside Rezusun's at equal sizes."""
+    z = COMPARE_SIZES[size]
+    pk = peaks()
+    sampler = ClockSampler()
+    sampler.start()
+    w0 = time.perf_counter()
+    chunk = 1024
+    log(f"{size}: Tevanex")
+    tev = measure_design(tevanex_config(z, chunk))
+    log(f"{size}: Rezusun")
+    rez = measure_design(rezusun_config(z))
+    log(f"{size}: Zatusun")
+    zat = measure_design(zatusun_config(z, chunk))
+    w1 = time.perf_counter()
+    sampler.stop()
+    T, R, ctx = PREFILL_TOKENS, 64, PROMPT_LEN
+    pairs = T * (T + 1) // 2
+    seen = sum(i % chunk + 1 for i in range(T))
+    H, G, W = z["heads"], z["heads"] // 4, z["width"]
+    dc = z["kv_rank"] + z["lat_rot"]
+    cols = 32 * (z["ff"] // 32) + z["ff"] // 4
+    # per token: the product's q, k, v read, the queries written, the rows written (Tevanex: the two attentions' mean)
+    tev_qkv = ((H + 2 * G) * 64 + (H // 2 + 2 * (H // 8)) * 128) / 2
+    zat_qkv = (H + 2 * G) * 64
+
+    def per_launch(d, phase, key, *names):
+        for name in names:
+            n, ms = d[phase][key].get(name, (0, 0.0))
+            if n:
+                return ms / n
+        return None
+
+    def frac(work, ms, peak_per_s):
+        return None if not ms else round(work / (ms * 1e-3) / peak_per_s, 4)
+    tensor, hbm, fma = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9, FP32_FMA_TFLOPS_NOMINAL * 1e12
+    pre, dec = ("prefill_2048", "operators"), ("decode_b64", "operators_launched")
+    lat_names = ("latent_attention_tc", "latent_attention")
+    kernels = {
+        "tevanex attention, 2048 tokens (of the measured bf16 peak)": frac(
+            seen * 4 * H * 64, per_launch(tev, *pre, "flash_attention_rows", "window_flash_attention", "window_attention"), tensor),
+        # two maps a head: 2 (dim + vdim) FLOP each per seen pair
+        "zatusun attention, 2048 tokens (of the measured bf16 peak)": frac(
+            seen * 2 * (64 + 128) * 2 * (H // 2), per_launch(zat, *pre, "window_flash_attention", "window_attention"), tensor),
+        "tevanex window_attention, batch 64 (of the measured copy peak)": frac(
+            R * min(ctx, chunk) * 2 * G * 64 * 2, per_launch(tev, *dec, "window_attention"), hbm),
+        "zatusun window_attention, batch 64 (of the measured copy peak)": frac(
+            R * min(ctx, chunk) * (H // 8) * 256 * 2, per_launch(zat, *dec, "window_attention"), hbm),
+        "tevanex qk_rot_append, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * tev_qkv * 2, per_launch(tev, *pre, "qk_rot_append"), hbm),
+        "zatusun qk_rot_append, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * zat_qkv * 2, per_launch(zat, *pre, "qk_rot_append"), hbm),
+        # per element of the memory and token: keep and add (2 FLOP), read out (2)
+        "tevanex mlstm_scan, 2048 tokens (of the nominal fp32 FMA peak)": frac(
+            T * H * 64 * 65 * 4, per_launch(tev, *pre, "mlstm_scan"), fma),
+        "zatusun linear_scan, 2048 tokens (of the nominal fp32 FMA peak)": frac(
+            T * H * 64 * 64 * 4, per_launch(zat, *pre, "linear_scan"), fma),
+        "tevanex mlstm_scan, batch 64 (of the measured copy peak)": frac(
+            2 * R * H * 64 * 65 * 4, per_launch(tev, *dec, "mlstm_scan"), hbm),
+        "zatusun linear_scan, batch 64 (of the measured copy peak)": frac(
+            2 * R * H * 64 * 64 * 4, per_launch(zat, *dec, "linear_scan"), hbm),
+        "rezusun latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
+            pairs * z["lat_heads"] * 2 * (dc + z["kv_rank"]), per_launch(rez, *pre, *lat_names), tensor),
+        "zatusun latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
+            pairs * z["lat_heads"] * 2 * (dc + z["kv_rank"]), per_launch(zat, *pre, *lat_names), tensor),
+        "rezusun latent_attention, batch 64 (of the measured copy peak)": frac(
+            R * ctx * dc * 2, per_launch(rez, *dec, *lat_names), hbm),
+        "zatusun latent_attention, batch 64 (of the measured copy peak)": frac(
+            R * ctx * dc * 2, per_launch(zat, *dec, *lat_names), hbm),
+        "rezusun latent_prep, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * (z["q_rank"] + dc) * 2, per_launch(rez, *pre, "latent_prep"), hbm),
+        "zatusun latent_prep, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * (z["q_rank"] + dc) * 2, per_launch(zat, *pre, "latent_prep"), hbm),
+        "tevanex add_norm, 2048 tokens (of the measured copy peak)": frac(
+            T * W * 12, per_launch(tev, *pre, "add_norm"), hbm),
+        "zatusun add_rmsnorm, 2048 tokens (of the measured copy peak)": frac(
+            T * W * 12, per_launch(zat, *pre, "add_rmsnorm"), hbm),
+        # the start of a pass: the product's rows and the embedding's share read, the stream and the normed rows written
+        "zatusun join_norm, 2048 tokens (of the measured copy peak)": frac(
+            T * W * 14, per_launch(zat, *pre, "join_norm"), hbm),
+        "tevanex limited_act, 2048 tokens (of the measured copy peak)": frac(
+            T * cols * 6, per_launch(tev, *pre, "limited_act"), hbm),
+        "zatusun limited_act, 2048 tokens (of the measured copy peak)": frac(
+            T * cols * 6, per_launch(zat, *pre, "limited_act"), hbm),
+        "tevanex route, 2048 tokens (of the measured copy peak)": frac(T * (33 + 32) * 4, per_launch(tev, *pre, "route"), hbm),
+        "zatusun route, 2048 tokens (of the measured copy peak)": frac(T * (32 + 32) * 4, per_launch(zat, *pre, "route"), hbm),
+    }
+    return {"compare": size, "design": "zatusun", "beside": "tevanex, rezusun", "sizes": z, "chunk": chunk, "dtype": "bf16",
+            "data": "synthetic", "peaks": pk, "tevanex": tev, "rezusun": rez, "zatusun": zat,
+            "kernel_roofline_fractions": kernels, "clocks": sampler.summary(list(_compare_windows) or [(w0, w1)])}
+
+
 def run_compare(size):
     """The Rezusun design beside Llama at equal width, depth, feed-forward and vocabulary."""
     z = COMPARE_SIZES[size]
@@ -868,14 +985,14 @@ def main():
                     help="instead of the headline: prefill and decode of another design (--design) beside a Llama model of "
                          "equal width, depth, feed-forward and vocabulary (random weights), with the time of every "
                          "operator and roofline fractions of the designs' own kernels; prints its own JSON line")
-    ap.add_argument("--design", default="rezusun", choices=["rezusun", "solulix", "nonetar", "tevanex"],
-                    help="with --compare: which design stands beside Llama (nonetar and tevanex: beside Solulix, the "
-                         "closest design)")
+    ap.add_argument("--design", default="rezusun", choices=["rezusun", "solulix", "nonetar", "tevanex", "zatusun"],
+                    help="with --compare: which design stands beside Llama (nonetar and tevanex: beside Solulix; zatusun: "
+                         "beside Tevanex and Rezusun, the closest designs)")
     args = ap.parse_args()
 
     if args.compare:
         result = {"solulix": run_compare_solulix, "nonetar": run_compare_nonetar,
-                  "tevanex": run_compare_tevanex}.get(args.design, run_compare)(args.compare)
+                  "tevanex": run_compare_tevanex, "zatusun": run_compare_zatusun}.get(args.design, run_compare)(args.compare)
         print(json.dumps(result), flush=True)
         return 0
     if args.impl == "reference":

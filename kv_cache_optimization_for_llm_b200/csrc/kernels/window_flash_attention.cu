@@ -40,12 +40,20 @@ struct RowsArgs {
   float scale; int window, keep_first, one_more;
   ScoreShape shape;
   int* status;
+  int num_tiles, period;      // period > 0: tiles per block of positions; the grid is a multiple of it
 };
+
+// 2^x by the hardware's instruction (x at most 0 here; results below the smallest normal number become 0).
+__device__ __forceinline__ float exp2_hw(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 
 // KS: k-steps of 16 key channels (the padded key size is KS * 16); DP: pairs of 8 value channels (the padded
 // value size is DP * 16); NW: warps, 16 query rows each.
 template <int KS, int DP, int NW, bool PAIR>
-__global__ void __launch_bounds__(NW * 32)
+__global__ void __launch_bounds__(NW * 32, PAIR ? 16 / NW : 1)
 window_flash_attention_kernel(RowsArgs p) {
   constexpr int BM = NW * 16;
   constexpr int MAPS = PAIR ? 2 : 1, MROWS = BM / MAPS;   // rows of one map
@@ -61,8 +69,14 @@ window_flash_attention_kernel(RowsArgs p) {
 
   pdl_trigger();
   pdl_wait();
-  // the last tiles of a request read the most keys: they start first
-  const TileDesc tile = p.tiles[gridDim.x - 1 - blockIdx.x];
+  // the last tiles of a request read the most keys: they start first; with blocks of positions, the last ones of every block
+  int at = gridDim.x - 1 - blockIdx.x;
+  if (p.period > 0) {
+    const int n_blocks = gridDim.x / p.period;
+    at = blockIdx.x % n_blocks * p.period + p.period - 1 - blockIdx.x / n_blocks;
+    if (at >= p.num_tiles) return;
+  }
+  const TileDesc tile = p.tiles[at];
   const int hk = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int G = p.G, gp_shift = p.gp_shift, gp = 1 << gp_shift;
@@ -79,6 +93,7 @@ window_flash_attention_kernel(RowsArgs p) {
   const int pos_last = p.positions[tile.t0 + tile.n_tok - 1];
   const int k_hi = pos_last + 1;                                    // keys [.., k_hi) are read
   const int k_lo = first_seen_key(pos_first, window, p.shape.chunk);    // positions ascend: no row of the tile sees less
+  const int lo_last = first_seen_key(pos_last, window, p.shape.chunk);  // none sees more before its own position than from here
   const int first_tile = k_lo / BN, last_tile = (k_hi - 1) / BN;
   const int keep = window > 0 ? p.keep_first : 0;
   const int keep_tiles = min((keep + BN - 1) / BN, first_tile);
@@ -197,18 +212,44 @@ window_flash_attention_kernel(RowsArgs p) {
     // shape, mask and running softmax; from here on the scores are in units of log2
     const int kbase = t * BN + ((lane & 3) << 1);
     float mx[2] = {-CUDART_INF_F, -CUDART_INF_F};
+    if constexpr (PAIR) {
+      // no cap, no bias; a tile that every row sees whole needs no mask
+      const float f = p.scale * kLog2e;
+      if ((t + 1) * BN - 1 <= pos_first && t * BN >= lo_last) {
 #pragma unroll
-    for (int n = 0; n < BN / 8; ++n) {
+        for (int n = 0; n < BN / 8; ++n) {
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int j = kbase + n * 8 + (e & 1);
-        const int rr = e >> 1;
-        const bool ok = j <= pos_r[rr] && (j >= lo_r[rr] || j < keep);
-        float v = s[n][e] * hs[rr];
-        if (cap > 0.f) v = cap * tanhf(v * inv_cap);
-        v = fmaf(-slope[rr], (float)(pos_r[rr] - j), v);
-        s[n][e] = ok ? v * kLog2e : -CUDART_INF_F;
-        mx[rr] = fmaxf(mx[rr], s[n][e]);
+          for (int e = 0; e < 4; ++e) {
+            s[n][e] *= f;
+            mx[e >> 1] = fmaxf(mx[e >> 1], s[n][e]);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int n = 0; n < BN / 8; ++n) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int j = kbase + n * 8 + (e & 1);
+            const int rr = e >> 1;
+            s[n][e] = j <= pos_r[rr] && j >= lo_r[rr] ? s[n][e] * f : -CUDART_INF_F;
+            mx[rr] = fmaxf(mx[rr], s[n][e]);
+          }
+        }
+      }
+    } else {
+#pragma unroll
+      for (int n = 0; n < BN / 8; ++n) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = kbase + n * 8 + (e & 1);
+          const int rr = e >> 1;
+          const bool ok = j <= pos_r[rr] && (j >= lo_r[rr] || j < keep);
+          float v = s[n][e] * hs[rr];
+          if (cap > 0.f) v = cap * tanhf(v * inv_cap);
+          v = fmaf(-slope[rr], (float)(pos_r[rr] - j), v);
+          s[n][e] = ok ? v * kLog2e : -CUDART_INF_F;
+          mx[rr] = fmaxf(mx[rr], s[n][e]);
+        }
       }
     }
     float corr[2], m_use[2];
@@ -222,15 +263,23 @@ window_flash_attention_kernel(RowsArgs p) {
       m_run[rr] = m_new;
       l_run[rr] *= corr[rr];
     }
+    if (!PAIR || __any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {
 #pragma unroll
-    for (int n = 0; n < DT; ++n) {
-      o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
+      for (int n = 0; n < DT; ++n) {
+        o[n][0] *= corr[0]; o[n][1] *= corr[0]; o[n][2] *= corr[1]; o[n][3] *= corr[1];
+      }
     }
     unsigned pf[BN / 16][4];
 #pragma unroll
     for (int n = 0; n < BN / 8; ++n) {
-      const float p0 = exp2f(s[n][0] - m_use[0]), p1 = exp2f(s[n][1] - m_use[0]);
-      const float p2 = exp2f(s[n][2] - m_use[1]), p3 = exp2f(s[n][3] - m_use[1]);
+      float p0, p1, p2, p3;
+      if constexpr (PAIR) {
+        p0 = exp2_hw(s[n][0] - m_use[0]); p1 = exp2_hw(s[n][1] - m_use[0]);
+        p2 = exp2_hw(s[n][2] - m_use[1]); p3 = exp2_hw(s[n][3] - m_use[1]);
+      } else {
+        p0 = exp2f(s[n][0] - m_use[0]); p1 = exp2f(s[n][1] - m_use[0]);
+        p2 = exp2f(s[n][2] - m_use[1]); p3 = exp2f(s[n][3] - m_use[1]);
+      }
       l_run[0] += p0 + p1;
       l_run[1] += p2 + p3;
       // the accumulator layout of two neighbouring score tiles is the A layout of one k-step
@@ -341,7 +390,16 @@ int launch(const RowsArgs& a, int num_tiles, cudaStream_t stream) {
                                          cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  kvb_launch(window_flash_attention_kernel<KS, DP, NW, PAIR>, dim3(num_tiles, a.nkv), dim3(NW * 32), smem, stream, a);
+  RowsArgs b = a;
+  b.num_tiles = num_tiles;
+  int grid_x = num_tiles;
+  const int per_tile = BM / ((PAIR ? 2 : 1) << a.gp_shift);       // tokens
+  b.period = 0;
+  if (a.shape.chunk > 0 && per_tile > 0 && a.shape.chunk % per_tile == 0 && a.shape.chunk / per_tile < num_tiles) {
+    b.period = a.shape.chunk / per_tile;
+    grid_x = (num_tiles + b.period - 1) / b.period * b.period;
+  }
+  kvb_launch(window_flash_attention_kernel<KS, DP, NW, PAIR>, dim3(grid_x, a.nkv), dim3(NW * 32), smem, stream, b);
   return kvb_launch_result();
 }
 
