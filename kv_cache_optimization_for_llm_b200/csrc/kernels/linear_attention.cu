@@ -1,4 +1,4 @@
-// Linear attention whose memory decays per head and key channel, the decay also deciding what is written.
+// Linear attention whose memory decays per head and key channel and takes in what the decay makes room for.
 //
 // Per head, with raw projections zq, zf of N channels and v of Dv:
 //     q = silu(zq),   f = l + (1 - l) sigmoid(zf + b)          l, b: learned, per head and channel

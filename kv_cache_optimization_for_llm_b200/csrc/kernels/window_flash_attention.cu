@@ -93,7 +93,7 @@ window_flash_attention_kernel(RowsArgs p) {
   const int pos_last = p.positions[tile.t0 + tile.n_tok - 1];
   const int k_hi = pos_last + 1;                                    // keys [.., k_hi) are read
   const int k_lo = first_seen_key(pos_first, window, p.shape.chunk);    // positions ascend: no row of the tile sees less
-  const int lo_last = first_seen_key(pos_last, window, p.shape.chunk);  // none sees more before its own position than from here
+  const int lo_last = first_seen_key(pos_last, window, p.shape.chunk);  // from here on every row of the tile sees the keys up to its own position
   const int first_tile = k_lo / BN, last_tile = (k_hi - 1) / BN;
   const int keep = window > 0 ? p.keep_first : 0;
   const int keep_tiles = min((keep + BN - 1) / BN, first_tile);

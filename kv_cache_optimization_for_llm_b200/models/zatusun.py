@@ -3,8 +3,8 @@
 A token's embedding times a constant, plus a learned vector of its position, starts the residual stream.  Sublayers
 read the stream through an RMS norm whose weight is stored around zero.  Mixers are of three kinds: attention over a
 cached latent with stretched rotary frequencies and an output gate; a differential attention (two maps over the same
-values, subtracted and normed per head) over blocks of positions; and a linear attention whose forget gate per head
-and channel also decides what is written.  The feed-forward is a set of small gated experts with limited activations,
+values, subtracted and normed per head) over blocks of positions; and a linear attention with a memory whose rows
+decay one by one and take in what the decay makes room for.  The feed-forward is a set of small gated experts with limited activations,
 chosen by a router whose chosen logits alone enter a softmax.  A run of layers may be repeated with the same weights,
 each pass keeping a cache or state of its own; every pass starts from a product over the stream and the embedding's
 output side by side, plus a learned vector.  The logits are capped.  config.json names the layers one by one.

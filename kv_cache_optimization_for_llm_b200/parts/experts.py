@@ -102,7 +102,7 @@ class LimitedExperts(Part):
 
     The router's logits ``W_r h`` are float32.  ``score`` "sigmoid" (the default): the scores are their sigmoids, each by
     itself; the ``top`` experts with the largest scores are chosen and weighted with their scores as they are.
-    "softmax_chosen": the ``top`` largest logits are chosen, and their weights are the softmax over the chosen alone.
+    "softmax_chosen": the ``top`` experts of the highest logits, each weighing its share of a softmax that leaves out all others.
     ``weigh`` "input" (the default): the weight multiplies the expert's *input*, the layer's output is the sum of
     ``expert(w h)`` over the chosen experts; "output": the sum of ``w expert(h)``.  With ``shared_ff`` > 0 one more
     expert of the same form (its own ``shared_limit``) runs for every token with weight 1, and its output is multiplied

@@ -215,7 +215,7 @@ class MatrixLSTM(Part):
 
 @register("mixer", "decayed_linear_attention")
 class DecayedLinearAttention(Part):
-    """Linear attention in which the forget gate also decides what is written (HGRN2).  One product lays out
+    """Linear attention whose memory decays per key channel and takes in what the decay makes room for (HGRN2).  One product lays out
     [q: heads * dim | f: heads * dim | v: heads * vdim].  Per head, with ``q = silu(q)`` and, channel by channel,
     ``f = lower + (1 - lower) sigmoid(f + f_bias)`` (``lower``, ``f_bias``: learned, heads * dim numbers):
 

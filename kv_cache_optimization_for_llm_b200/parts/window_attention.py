@@ -353,8 +353,8 @@ class DifferentialChunkAttention(Part):
     q (``heads`` x 2 x ``dim``), k (``kv_heads`` x 2 x ``dim``) and v (``kv_heads`` x ``vdim``) come from one product with the
     row-stacked matrix; a head's rows are [map 1, map 2].  The first ``position.rotary_dim`` channels of every map of
     every query and key head turn with the position (``position``: "rope_interleaved", or None).  Keys and values go to
-    the request's pages, a row [k1 | k2 | v] per token and key/value head.  Each map is an attention of its own over the
-    same values, ``s = (q . k) * scale``, query i seeing key j <= i only when ``i // chunk == j // chunk`` (blocks counted
+    the request's pages, a row [k1 | k2 | v] per token and key/value head.  Either map has scores
+    ``s = (q . k) * scale`` and weighs the same values, query i seeing key j <= i only when ``i // chunk == j // chunk`` (blocks counted
     from the sequence's start; ``chunk`` None: every key up to i), softmax in float32.  With a head's two results a1, a2
 
         o = a1 - lam * a2,   lam = exp(lq1 . lk1) - exp(lq2 . lk2) + diff   (one number, made when the model is built),
