@@ -14,6 +14,7 @@ group, a pool and tables of their own.
 
 from __future__ import annotations
 
+import dataclasses
 from typing import Dict, List, Optional, Sequence, Tuple
 
 import torch
@@ -31,13 +32,15 @@ class PagedCache:
                  page_size: int, num_pages: int, num_slots: int, max_model_len: int,
                  dtype: torch.dtype, device, allocate: bool = True):
         """``entry_specs[i]``: what schedule entry i's mixer asks for (PagedKVSpec,
-        SlotStateSpec or None).  ``cache_of[i]``: entry whose cache entry i reads."""
+        SlotStateSpec or None).  ``cache_of[i]``: entry whose cache entry i reads; where the two want to see
+        differently far back, the pages are kept for the one that sees further."""
         self.page_size, self.num_pages, self.num_slots = int(page_size), int(num_pages), int(num_slots)
         self.dtype, self.device = dtype, torch.device(device)
         host = host_runtime()
         group_keys: List[Tuple] = []
         self.entry_group: List[Optional[Tuple[int, int]]] = []  # (group, index inside it)
         counts: List[int] = []
+        entry_specs = self._widened(entry_specs, cache_of)
         for i, wish in enumerate(entry_specs):
             spec = paged_part(wish)
             if cache_of[i] is not None or spec is None:
@@ -55,7 +58,7 @@ class PagedCache:
             if src is not None:
                 if type(entry_specs[i]) is not type(entry_specs[src]):
                     raise ValueError(f"schedule entry {i} cannot read the cache of entry {src}: different kinds")
-                if paged_part(entry_specs[i]) is not None and entry_specs[i] != entry_specs[src]:
+                if paged_part(entry_specs[i]) is not None and not self._same_rows(entry_specs[i], entry_specs[src]):
                     raise ValueError(f"schedule entry {i} cannot read the cache of entry {src}: "
                                      f"{entry_specs[i]} against {entry_specs[src]}")
         self.group_keys = group_keys
@@ -83,6 +86,26 @@ class PagedCache:
                 if spec is not None and cache_of[i] is None:
                     self.states[i] = torch.zeros((self.num_slots + 1,) + tuple(spec.shape), dtype=spec.dtype,
                                                  device=self.device)
+
+    @staticmethod
+    def _same_rows(a, b) -> bool:
+        """Whether two wishes are for the same cached rows; how long they are kept (window, first tokens) may differ."""
+        pa, pb = paged_part(a), paged_part(b)
+        rows = [(p.num_kv_heads, p.head_dim, p.planes) for p in (pa, pb)]
+        return rows[0] == rows[1] and state_part(a) == state_part(b)
+
+    @staticmethod
+    def _widened(entry_specs, cache_of):
+        """The wishes, those whose rows other entries read widened to what all of the readers need: the largest window
+        (None: every key) and the most kept first tokens."""
+        out = list(entry_specs)
+        for i, src in enumerate(cache_of):
+            if src is None or not isinstance(out[i], PagedKVSpec) or not isinstance(out[src], PagedKVSpec):
+                continue
+            a, b = out[src], out[i]
+            window = max(a.window, b.window) if a.window and b.window else None
+            out[src] = dataclasses.replace(a, window=window, keep_first=max(a.keep_first, b.keep_first) if window else 0)
+        return out
 
     @property
     def scratch_page(self) -> int:

@@ -689,3 +689,118 @@ class ZatusunConfig:
         for t in range(times):
             order += [(i, t if i == a else None) for i in range(a, b)]
         return order + [(i, None) for i in range(b, n)]
+
+
+@dataclass(frozen=True)
+class LobuzenLayerConfig:
+    """One entry of ``layers``: the mixer's kind (``latent_attention`` or ``attention``) and sizes, and the feed-forward
+    (None: the layer has only its mixer)."""
+    type: str
+    mixer: Mapping[str, Any]
+    mlp: Optional[Mapping[str, Any]]
+
+    @property
+    def window(self) -> Optional[int]:
+        """How many of the last positions a token sees, its own included (None: all of them)."""
+        mask = self.mixer.get("mask")
+        return int(mask["size"]) if mask else None
+
+    @property
+    def latent_of(self) -> Optional[int]:
+        """The layer whose latents this one attends to (None: its own)."""
+        src = self.mixer.get("kv_from")
+        return None if src is None else int(src)
+
+
+_LOBUZEN_MIXER_KEYS = {
+    "latent_attention": ("heads", "dim", "vdim", "kv_rank", "scale"),
+    "attention": ("heads", "kv_heads", "dim", "vdim", "scale"),
+}
+
+
+@dataclass(frozen=True)
+class LobuzenConfig:
+    """The keys of a Lobuzen config.json: ``vocab``, ``width``, ``norm.eps``, ``token_side.dim`` (columns of a token's own
+    row that every layer gets) and ``layers`` (each with ``type``, ``mixer`` and ``mlp``).  A ``latent_attention`` names
+    ``heads``, ``dim``, ``vdim``, ``kv_rank``, ``scale``, optionally ``mask.size`` and ``kv_from`` (an earlier layer
+    with latents of its own); an ``attention`` ``heads``, ``kv_heads``, ``dim``, ``vdim``, ``scale`` and optionally
+    ``mask.size``.  A feed-forward is of ``kind`` ``dense`` (``ff``, ``limit``) or ``moe`` (``expert.ff``, ``router`` with
+    ``experts``, ``top`` and optionally ``groups`` with ``count`` and ``keep``)."""
+    architecture: str
+    vocab: int
+    width: int
+    norm_eps: float
+    token_dim: int              # 0: the layers get nothing from their tokens
+    layers: Tuple[LobuzenLayerConfig, ...]
+    max_position_embeddings: int
+    eos_token_ids: Tuple[int, ...] = field(default_factory=tuple)
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "LobuzenConfig":
+        norm = d.get("norm") or {}
+        entries = list(d.get("layers") or [])
+        layers = []
+        for i, entry in enumerate(entries):
+            kind = entry.get("type")
+            if kind not in _LOBUZEN_MIXER_KEYS:
+                raise ConfigError(f"config.json: layer {i} has a mixer of type {kind!r}; known: "
+                                  + ", ".join(sorted(_LOBUZEN_MIXER_KEYS)))
+            mixer = entry.get("mixer") or {}
+            for key in _LOBUZEN_MIXER_KEYS[kind]:
+                if mixer.get(key) is None:
+                    raise ConfigError(f"config.json: layer {i} ({kind}): mixer key {key!r} is missing")
+            if mixer.get("mask") and int(mixer["mask"].get("size") or 0) < 1:
+                raise ConfigError(f"config.json: layer {i}: mixer.mask.size must be a positive number of positions")
+            if kind == "attention":
+                if int(mixer["kv_heads"]) < 1 or int(mixer["heads"]) % int(mixer["kv_heads"]):
+                    raise ConfigError(f"config.json: layer {i}: {mixer['heads']} query heads cannot be grouped over "
+                                      f"{mixer['kv_heads']} key/value heads")
+            elif mixer.get("kv_from") is not None:
+                src = int(mixer["kv_from"])
+                if not 0 <= src < i or layers[src].type != kind or layers[src].latent_of is not None:
+                    raise ConfigError(f"config.json: layer {i}: mixer.kv_from {src} must name an earlier layer of type "
+                                      f"{kind!r} that makes latents of its own")
+                if int(layers[src].mixer["kv_rank"]) != int(mixer["kv_rank"]):
+                    raise ConfigError(f"config.json: layer {i}: mixer.kv_rank {mixer['kv_rank']} differs from the "
+                                      f"{layers[src].mixer['kv_rank']} of layer {src}, whose latents it uses")
+            mlp = entry.get("mlp")
+            if mlp is not None:
+                if mlp.get("kind") == "dense":
+                    for key in ("ff", "limit"):
+                        if mlp.get(key) is None:
+                            raise ConfigError(f"config.json: layer {i}: mlp.{key} is missing")
+                elif mlp.get("kind") == "moe":
+                    for group, keys in (("expert", ("ff",)), ("router", ("experts", "top"))):
+                        for key in keys:
+                            if (mlp.get(group) or {}).get(key) is None:
+                                raise ConfigError(f"config.json: layer {i}: mlp.{group}.{key} is missing")
+                    r = mlp["router"]
+                    if not 1 <= int(r["top"]) <= int(r["experts"]):
+                        raise ConfigError(f"config.json: layer {i}: mlp.router.top must lie between 1 and mlp.router.experts")
+                    groups = r.get("groups")
+                    if groups:
+                        for key in ("count", "keep"):
+                            if groups.get(key) is None:
+                                raise ConfigError(f"config.json: layer {i}: mlp.router.groups.{key} is missing")
+                        n, keep = int(groups["count"]), int(groups["keep"])
+                        if n < 1 or int(r["experts"]) % n or not 1 <= keep <= n:
+                            raise ConfigError(f"config.json: layer {i}: mlp.router.groups: {r['experts']} experts do not form "
+                                              f"{n} equal groups of which {keep} are kept")
+                        if int(r["top"]) > keep * (int(r["experts"]) // n):
+                            raise ConfigError(f"config.json: layer {i}: mlp.router.top {r['top']} exceeds the experts of "
+                                              f"{keep} groups")
+                else:
+                    raise ConfigError(f"config.json: layer {i}: a feed-forward of kind {mlp.get('kind')!r} is not known "
+                                      "(known: 'dense', 'moe')")
+            layers.append(LobuzenLayerConfig(str(kind), dict(mixer), dict(mlp) if mlp is not None else None))
+        if not layers:
+            raise ConfigError("config.json: 'layers' is missing or empty")
+        eos = d.get("eos_token_id")
+        eos_ids = () if eos is None else (tuple(int(e) for e in eos) if isinstance(eos, (list, tuple)) else (int(eos),))
+        cfg = cls(architecture=str(d.get("architecture") or (d.get("architectures") or ["Lobuzen"])[0]),
+                  vocab=_need(d, "vocab", int), width=_need(d, "width", int), norm_eps=_need(norm, "eps", float),
+                  token_dim=int((d.get("token_side") or {}).get("dim") or 0), layers=tuple(layers),
+                  max_position_embeddings=int(d.get("max_position_embeddings") or 131072), eos_token_ids=eos_ids)
+        if cfg.vocab < 1 or cfg.width < 1 or cfg.token_dim < 0 or not cfg.norm_eps > 0:
+            raise ConfigError("config.json: vocab and width must be positive, token_side.dim not negative and norm.eps above zero")
+        return cfg

@@ -3,7 +3,8 @@
 //   * route_kernel: the router.  A block per up to eight tokens: logits z = W_r h in float32 (W_r float32, h as
 //     stored; or handed in by the caller, who made them with a product of float32 sums), scores s = softmax(z) over
 //     all experts (or, score_fn 1, s = sigmoid(z) of each), the `top` experts with the largest s + correction
-//     (ties go to the lower index), their weights s / (sum of the chosen s + 1e-20) * scale (or, without renorm,
+//     (ties go to the lower index; where the experts form groups of neighbours, only from the groups with the
+//     largest sums of their two best s + correction), their weights s / (sum of the chosen s + 1e-20) * scale (or, without renorm,
 //     s * scale).  It
 //     leaves a dense table gate[t, e] (0 for an expert that was not chosen) and, for the last
 //     `identity` experts, which have no matrices and hand their input on, the sum of their weights.
@@ -33,7 +34,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32)
 route_kernel(const T* __restrict__ h, int ld_h, const float* __restrict__ w_router, const float* __restrict__ logits,
              int ld_logits, const float* __restrict__ correction, float* __restrict__ gate,
              float* __restrict__ identity_weight, int T_, int K, int E, int n_identity, int top, float scale, int score_fn,
-             int renorm, int tb) {
+             int renorm, int groups, int keep, int tb) {
   extern __shared__ float smem[];
   pdl_trigger();
   pdl_wait();
@@ -43,7 +44,8 @@ route_kernel(const T* __restrict__ h, int ld_h, const float* __restrict__ w_rout
   const int n_all = E + n_identity;
   float* s_all = smem;                                  // [tb][n_all] logits, then scores
   float* c_all = s_all + (size_t)tb * n_all;            // [tb][n_all] choice scores; -inf once chosen
-  float* part_all = c_all + (size_t)tb * n_all;         // [kRouteWarps][tb][n_all] the warps' sums (not with logits)
+  float* g_all = c_all + (size_t)tb * n_all;            // [tb][groups] what a group is judged by
+  float* part_all = g_all + (size_t)tb * groups;        // [kRouteWarps][tb][n_all] the warps' sums (not with logits)
   float* x = part_all + (size_t)kRouteWarps * tb * n_all;   // [tb][K] the tokens' inputs, float32 (not with logits)
   if (logits != nullptr) {
     for (int i = threadIdx.x; i < n_tok * n_all; i += blockDim.x) {
@@ -122,6 +124,27 @@ route_kernel(const T* __restrict__ h, int ld_h, const float* __restrict__ w_rout
       gate[(size_t)t * n_all + e] = 0.f;
     }
     __syncwarp();
+    if (groups > 0) {
+      // a group's score is the sum of its two best choice scores; the experts of all but the `keep` best groups are out
+      float* gs = g_all + (size_t)tt * groups;
+      const int per = n_all / groups;
+      for (int g = lane; g < groups; g += 32) {
+        float a = -CUDART_INF_F, b = -CUDART_INF_F;
+        for (int i = 0; i < per; ++i) {
+          const float v = c[g * per + i];
+          if (v > a) { b = a; a = v; } else if (v > b) b = v;
+        }
+        gs[g] = per > 1 ? a + b : a;
+      }
+      __syncwarp();
+      for (int g = lane; g < groups; g += 32) {
+        int better = 0;
+        for (int o = 0; o < groups; ++o) better += gs[o] > gs[g] || (gs[o] == gs[g] && o < g);
+        if (better >= keep)
+          for (int i = 0; i < per; ++i) c[g * per + i] = -CUDART_INF_F;
+      }
+      __syncwarp();
+    }
     // the chosen experts, one after the other; their indices end up in lane 0 .. top - 1's `mine`
     int mine = -1;
     float chosen_sum = 0.f;
@@ -158,23 +181,26 @@ route_kernel(const T* __restrict__ h, int ld_h, const float* __restrict__ w_rout
 
 // logits: float32 [T, >= E + n_identity] with row stride ld_logits, the router's products if the caller has made them
 // (h and w_router are not read then), else null.  correction: may be null.  score_fn 0: softmax over all experts, 1: a
-// sigmoid of each.  renorm 0: the chosen scores are the weights as they are (times scale).
+// sigmoid of each.  renorm 0: the chosen scores are the weights as they are (times scale).  groups > 0: the experts form
+// that many equal groups of neighbours, of which the best `keep` may be chosen from.
 // Refuses: more than 32 chosen experts per token, more than 4096 experts, K above 16384.
 KVB_EXPORT int kvb_route(const void* h, int ld_h, const float* w_router, const float* logits, int ld_logits,
                          const float* correction, float* gate, float* identity_weight, int T_, int K, int E,
-                         int n_identity, int top, float scale, int score_fn, int renorm, int dtype, cudaStream_t stream) {
+                         int n_identity, int top, float scale, int score_fn, int renorm, int groups, int keep, int dtype,
+                         cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (score_fn < 0 || score_fn > 1 || (logits != nullptr && ld_logits < E + n_identity)) return KVB_ERR_BAD_SIZE;
   if (E < 0 || n_identity < 0 || E + n_identity < 1 || E + n_identity > 4096 || top < 1 || top > 32 || K < 1 || K > 16384)
     return KVB_ERR_BAD_SIZE;
   const int n_all = E + n_identity;
+  if (groups < 0 || (groups > 0 && (n_all % groups != 0 || keep < 1 || keep > groups))) return KVB_ERR_BAD_SIZE;
   // as many tokens a block as their inputs fit 160 KB with, 8 at most; few tokens are spread over more blocks
   int tb = kRouteTokens;
   const size_t x_floats = logits ? 0 : (size_t)K + (size_t)kRouteWarps * n_all;
   // half of that once the step has blocks enough to fill the GPU either way: more blocks per SM hide more latency
-  while (tb > 1 && ((size_t)tb * (x_floats + 2 * n_all) * sizeof(float) > 160 * 1024 || (T_ + tb - 1) / tb < 64)) tb >>= 1;
+  while (tb > 1 && ((size_t)tb * (x_floats + 2 * n_all + groups) * sizeof(float) > 160 * 1024 || (T_ + tb - 1) / tb < 64)) tb >>= 1;
   if (tb == kRouteTokens && T_ / (tb / 2) >= 4 * kvb_sm_count()) tb >>= 1;
-  const size_t smem = (size_t)tb * (x_floats + 2 * n_all) * sizeof(float);
+  const size_t smem = (size_t)tb * (x_floats + 2 * n_all + groups) * sizeof(float);
   if (smem > 200 * 1024) return KVB_ERR_BAD_SIZE;
   KVB_DISPATCH_DTYPE(dtype, T, {
     if (smem > 48 * 1024) {
@@ -182,7 +208,7 @@ KVB_EXPORT int kvb_route(const void* h, int ld_h, const float* w_router, const f
       if (err != cudaSuccess) return (int)err;
     }
     kvb_launch(route_kernel<T>, dim3((T_ + tb - 1) / tb), dim3(kRouteWarps * 32), smem, stream, (const T*)h, ld_h, w_router,
-               logits, ld_logits, correction, gate, identity_weight, T_, K, E, n_identity, top, scale, score_fn, renorm, tb);
+               logits, ld_logits, correction, gate, identity_weight, T_, K, E, n_identity, top, scale, score_fn, renorm, groups, keep, tb);
   });
   return kvb_launch_result();
 }
@@ -259,20 +285,20 @@ KVB_EXPORT int kvb_expert_act(const void* p, const float* gate, int ld_gate, voi
   return kvb_launch_result();
 }
 
-// Experts of the form  down (a(g) (u + 1)),  g = min(w gate.h, limit),  u = clamp(w up.h, -limit, limit),
-// a(g) = g sigmoid(alpha g),  where w is the token's weight for the expert: it multiplies the expert's input, which for
+// Experts of the form  down (a(g) (u + offset)),  g = min(w gate.h, limit),  u = clamp(w up.h, -limit, limit),
+// a(g) = g sigmoid(alpha g)  (limit infinite, alpha 1, offset 0: the plain gated form silu(gate.h) up.h),  where w is the token's weight for the expert: it multiplies the expert's input, which for
 // matrices without biases is the same as multiplying both first products, before the limits.
 // p [T, ld_p]: per routed expert e its gate product (F features from column 2 e F) and its up product (the next F);
 // behind the E routed experts one that every token uses: S gate features, then S up features, with a limit of its own
 // and w = 1, whose result is multiplied by sigmoid(shared_logit[t * ld_s]) (float32; null: by 1), which for a last
 // matrix without bias is the same as multiplying its output.  gate [T, ld_gate] float32: the weights, 0 for an expert
-// that was not chosen.  weigh_output: the weight multiplies a(g) (u + 1) instead, behind the limits.
+// that was not chosen.  weigh_output: the weight multiplies a(g) (u + offset) instead, behind the limits.
 // out [T, E F + S + pad] dense, the padding columns zero.
 template <typename T>
 __global__ void limited_act_kernel(const T* __restrict__ p, int ld_p, const float* __restrict__ gate, int ld_gate,
                                    const float* __restrict__ shared_logit, int ld_s, T* __restrict__ out, int E, int F,
-                                   int S, int width, float limit, float shared_limit, float alpha, int weigh_output,
-                                   size_t total) {
+                                   int S, int width, float limit, float shared_limit, float alpha, float offset,
+                                   int weigh_output, size_t total) {
   pdl_trigger();
   pdl_wait();
   const int EF = E * F;
@@ -288,14 +314,14 @@ __global__ void limited_act_kernel(const T* __restrict__ p, int ld_p, const floa
         const float w_in = weigh_output ? 1.0f : w;
         const float g = fminf(w_in * to_f32(p[t * ld_p + 2 * e * F + i]), limit);
         const float u = fminf(fmaxf(w_in * to_f32(p[t * ld_p + 2 * e * F + F + i]), -limit), limit);
-        a = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+        a = g / (1.0f + expf(-alpha * g)) * (u + offset);
         if (weigh_output) a *= w;
       }
     } else if (j < EF + S) {
       const int i = j - EF;
       const float g = fminf(to_f32(p[t * ld_p + 2 * EF + i]), shared_limit);
       const float u = fminf(fmaxf(to_f32(p[t * ld_p + 2 * EF + S + i]), -shared_limit), shared_limit);
-      a = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+      a = g / (1.0f + expf(-alpha * g)) * (u + offset);
       if (shared_logit != nullptr) a *= 1.0f / (1.0f + expf(-shared_logit[t * ld_s]));
     }
     out[idx] = from_f32<T>(a);
@@ -304,16 +330,16 @@ __global__ void limited_act_kernel(const T* __restrict__ p, int ld_p, const floa
 
 // bfloat16 rows whose experts are multiples of 8 features wide: eight results per thread from two 16-byte loads, one
 // look at the token's weight for the expert, and no load at all for an expert that was not chosen.
-__device__ __forceinline__ float limited_one(float g, float u, float w, float limit, float alpha) {
+__device__ __forceinline__ float limited_one(float g, float u, float w, float limit, float alpha, float offset) {
   g = fminf(w * g, limit);
   u = fminf(fmaxf(w * u, -limit), limit);
-  return g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+  return g / (1.0f + expf(-alpha * g)) * (u + offset);
 }
 
 __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, int ld_p, const float* __restrict__ gate,
                                           int ld_gate, const float* __restrict__ shared_logit, int ld_s,
                                           __nv_bfloat16* __restrict__ out, int E, int F, int S, int width, float limit,
-                                          float shared_limit, float alpha, int weigh_output, size_t groups) {
+                                          float shared_limit, float alpha, float offset, int weigh_output, size_t groups) {
   pdl_trigger();
   pdl_wait();
   const int EF = E * F, gpr = width >> 3;
@@ -345,9 +371,10 @@ __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, i
       unsigned r[4];
 #pragma unroll
       for (int k = 0; k < 4; ++k) {
-        const float a = limited_one(__uint_as_float(gw[k] << 16), __uint_as_float(uw[k] << 16), w, lim, alpha) * post;
+        const float a = limited_one(__uint_as_float(gw[k] << 16), __uint_as_float(uw[k] << 16), w, lim, alpha,
+                                    offset) * post;
         const float b = limited_one(__uint_as_float(gw[k] & 0xffff0000u), __uint_as_float(uw[k] & 0xffff0000u), w, lim,
-                                    alpha) * post;
+                                    alpha, offset) * post;
         __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
         r[k] = *reinterpret_cast<unsigned*>(&v);
       }
@@ -359,7 +386,7 @@ __global__ void limited_act_bf16x8_kernel(const __nv_bfloat16* __restrict__ p, i
 
 KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int ld_gate, const float* shared_logit,
                                int ld_s, void* out, int T_, int E, int F, int S, int pad, float limit, float shared_limit,
-                               float alpha, int weigh_output, int dtype, cudaStream_t stream) {
+                               float alpha, float offset, int weigh_output, int dtype, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   const int width = E * F + S + pad;
   if (E < 0 || F < 1 || S < 0 || pad < 0 || E * F + S < 1 || ld_p < 2 * (E * F + S)) return KVB_ERR_BAD_SIZE;
@@ -369,7 +396,7 @@ KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int l
     const size_t want8 = (groups + 255) / 256;
     const int blocks8 = (int)(want8 < (size_t)kvb_sm_count() * 16 ? want8 : (size_t)kvb_sm_count() * 16);
     kvb_launch(limited_act_bf16x8_kernel, dim3(blocks8), dim3(256), 0, stream, (const __nv_bfloat16*)p, ld_p, gate, ld_gate,
-               shared_logit, ld_s, (__nv_bfloat16*)out, E, F, S, width, limit, shared_limit, alpha, weigh_output,
+               shared_logit, ld_s, (__nv_bfloat16*)out, E, F, S, width, limit, shared_limit, alpha, offset, weigh_output,
                groups);
     return kvb_launch_result();
   }
@@ -378,7 +405,7 @@ KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int l
   const int blocks = (int)(want < (size_t)kvb_sm_count() * 16 ? want : (size_t)kvb_sm_count() * 16);
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(limited_act_kernel<T>, dim3(blocks), dim3(256), 0, stream, (const T*)p, ld_p,
                                             gate, ld_gate, shared_logit, ld_s, (T*)out, E, F, S, width, limit,
-                                            shared_limit, alpha, weigh_output, total)));
+                                            shared_limit, alpha, offset, weigh_output, total)));
   return kvb_launch_result();
 }
 

@@ -6,14 +6,15 @@
 // (U_h^T q).c, so every head attends with an "absorbed" query [U_h^T q_plain | q_rot] over the
 // same cached rows, the weighted sum of the latents comes out [rank] wide per head and the
 // value up-projection is applied to it afterwards.  The kernels:
-//   latent_prep       per token: RMS norm of the query latent, RMS norm of the key/value latent,
-//                     interleaved rotary encoding of the shared key part, cache write
+//   latent_prep       per token: RMS norm of the query latent (where queries have one), RMS norm of the
+//                     key/value latent, interleaved rotary encoding of the shared key part, cache write
 //   head_gemm         a product per head, out[t, h, :] = W[h] . in[t, h, :]  (absorbs the queries,
 //                     and up-projects the attended latents; with a gate its result is multiplied by
 //                     the gate's sigmoid)
 //   head_rows         for steps whose per-head products the library made: [heads, tokens, N] back to one
 //                     row per token, with the same optional gate
-//   latent_attention  causal softmax attention of all heads over the cached rows, optionally with a sink:
+//   latent_attention  causal softmax attention of all heads over the cached rows, optionally over a sliding
+//                     window (position i sees j with i - j < window), optionally with a sink:
 //                     the denominator also holds exp(sink_h), a key without a value
 // Scores, softmax weights, sums and angles are float32.  Keys are walked in chunks of 32 by
 // absolute position, so a token's result does not depend on how its request was cut into steps,
@@ -25,7 +26,7 @@
 // ---------------------------------------------------------------- prep
 // d_in [T, ld]: the query latent at column 0 (q_rank wide), the key/value latent at column
 // kv_off (rank wide) followed by the shared key part (rot wide).
-// cq[t] = rms(d_in[t, :q_rank]) * wq;  page row = [ rms(latent) * wkv | rotate(shared part) ].
+// cq[t] = rms(d_in[t, :q_rank]) * wq (q_rank 0: no query latent);  page row = [ rms(latent) * wkv | rotate(shared part) ].
 // Rotation: pairs (2i, 2i + 1) for i < rdims / 2 turn by cos/sin[pos, i]; the rest passes.
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -83,7 +84,7 @@ KVB_EXPORT int kvb_latent_prep(const void* d_in, int ld, int q_rank, int kv_off,
                                int max_pages, int page_size, int num_pages, void* cq, void* pages, int write,
                                int T_, int dtype, int* status, cudaStream_t stream) {
   if (T_ <= 0) return 0;
-  if (q_rank < 1 || rank < 1 || rot < 0 || rdims < 0 || (rdims & 1) || rdims > rot) return KVB_ERR_BAD_SIZE;
+  if (q_rank < 0 || rank < 1 || rot < 0 || rdims < 0 || (rdims & 1) || rdims > rot) return KVB_ERR_BAD_SIZE;
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(latent_prep_kernel<T>, dim3(T_), dim3(128), 0, stream, (const T*)d_in, ld,
                                             q_rank, kv_off, rank, rot, rdims, wq, wkv, eps, cos_t, sin_t, table_len,
                                             positions, token_req, block_table, max_pages, page_size, num_pages,
@@ -252,7 +253,7 @@ latent_attention_kernel(const T* __restrict__ q_abs, int ld_qa, int hs_qa,     /
                         const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len, int rdims,
                         const T* __restrict__ pages, const int* __restrict__ block_table, int max_pages,
                         int page_size, int num_pages, const int* __restrict__ positions,
-                        const int* __restrict__ token_req, const float* __restrict__ sink, float scale,
+                        const int* __restrict__ token_req, const float* __restrict__ sink, float scale, int window,
                         T* __restrict__ out, int ld_out, int hs_out, int H, int rank, int rot, int* status) {
   extern __shared__ unsigned lat_smem[];
   constexpr int EW = Word<T>::N;
@@ -293,12 +294,13 @@ latent_attention_kernel(const T* __restrict__ q_abs, int ld_qa, int hs_qa,     /
 #pragma unroll
   for (int r = 0; r < NR; ++r) acc[r] = 0.f;
 
-  for (int c0 = 0; c0 <= pos; c0 += 32) {
+  const int lowest = window > 0 ? max(0, pos - window + 1) : 0;     // the first key the token sees
+  for (int c0 = lowest & ~31; c0 <= pos; c0 += 32) {
     const int n_keys = min(32, pos - c0 + 1);
     __syncthreads();                                  // the chunk before is used up (and q_s is written)
     if (threadIdx.x < 32) {
       long long off = -1;
-      if (threadIdx.x < n_keys) {
+      if (threadIdx.x < n_keys && c0 + (int)threadIdx.x >= lowest) {
         const int j = c0 + threadIdx.x;
         const int lp = j / page_size;
         const int page = lp < max_pages ? table[lp] : -1;
@@ -355,8 +357,8 @@ template <typename T, int NR>
 static int launch_latent(const void* q_abs, int ld_qa, int hs_qa, const void* q_raw, int ld_q, int hs_q,
                          const float* cos_t, const float* sin_t, int table_len, int rdims, const void* pages,
                          const int* block_table, int max_pages, int page_size, int num_pages, const int* positions,
-                         const int* token_req, const float* sink, float scale, void* out, int ld_out, int hs_out,
-                         int T_, int H, int rank, int rot, int* status, cudaStream_t stream) {
+                         const int* token_req, const float* sink, float scale, int window, void* out, int ld_out,
+                         int hs_out, int T_, int H, int rank, int rot, int* status, cudaStream_t stream) {
   const int Dc = rank + rot;
   const int words = Dc / Word<T>::N;
   const size_t smem = ((size_t)kLatWarps * Dc + 32 * (size_t)(words | 1)) * 4;
@@ -368,19 +370,20 @@ static int launch_latent(const void* q_abs, int ld_qa, int hs_qa, const void* q_
   }
   kvb_launch(latent_attention_kernel<T, NR>, dim3(T_, (H + kLatWarps - 1) / kLatWarps), dim3(kLatWarps * 32), smem,
              stream, (const T*)q_abs, ld_qa, hs_qa, (const T*)q_raw, ld_q, hs_q, cos_t, sin_t, table_len, rdims,
-             (const T*)pages, block_table, max_pages, page_size, num_pages, positions, token_req, sink, scale, (T*)out,
-             ld_out, hs_out, H, rank, rot, status);
+             (const T*)pages, block_table, max_pages, page_size, num_pages, positions, token_req, sink, scale, window,
+             (T*)out, ld_out, hs_out, H, rank, rot, status);
   return kvb_launch_result();
 }
 
-// Refuses: rank > 512; in bfloat16 an odd rank + rot or a cache that is not 4-byte aligned.
+// window 0: every key up to the token's own.  Refuses: rank > 512; in bfloat16 an odd rank + rot or a cache that is not 4-byte aligned.
 KVB_EXPORT int kvb_latent_attention(const void* q_abs, int ld_qa, int hs_qa, const void* q_raw, int ld_q, int hs_q,
                                     const float* cos_t, const float* sin_t, int table_len, int rdims,
                                     const void* pages, const int* block_table, int max_pages, int page_size,
                                     int num_pages, const int* positions, const int* token_req, const float* sink,
-                                    float scale, void* out, int ld_out, int hs_out, int T_, int H, int rank, int rot,
-                                    int dtype, int* status, cudaStream_t stream) {
+                                    float scale, int window, void* out, int ld_out, int hs_out, int T_, int H, int rank,
+                                    int rot, int dtype, int* status, cudaStream_t stream) {
   if (T_ <= 0) return 0;
+  if (window < 0) return KVB_ERR_BAD_SIZE;
   if (rank < 1 || rank > 512 || rot < 0 || H < 1 || (rdims & 1) || rdims > rot) return KVB_ERR_BAD_SIZE;
   if (dtype == KVB_BF16 && ((rank + rot) & 1)) return KVB_ERR_BAD_SIZE;
   if (reinterpret_cast<uintptr_t>(pages) & 3) return KVB_ERR_ALIGN;
@@ -388,8 +391,8 @@ KVB_EXPORT int kvb_latent_attention(const void* q_abs, int ld_qa, int hs_qa, con
   KVB_DISPATCH_DTYPE(dtype, T, return (launch_latent<T, NR>(q_abs, ld_qa, hs_qa, q_raw, ld_q, hs_q, cos_t, sin_t,  \
                                                             table_len, rdims, pages, block_table, max_pages,       \
                                                             page_size, num_pages, positions, token_req, sink,      \
-                                                            scale, out, ld_out, hs_out, T_, H, rank, rot, status,  \
-                                                            stream)))
+                                                            scale, window, out, ld_out, hs_out, T_, H, rank, rot,  \
+                                                            status, stream)))
   if (rank <= 64) { KVB_LATENT(2); }
   else if (rank <= 128) { KVB_LATENT(4); }
   else if (rank <= 256) { KVB_LATENT(8); }
@@ -436,8 +439,8 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
                            const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table, int max_pages,
                            int page_size, int num_pages, const int* __restrict__ positions,
                            const int* __restrict__ q_start, const int* __restrict__ tiles, int tokens_per_tile,
-                           const float* __restrict__ sink, float scale, __nv_bfloat16* __restrict__ out, int ld_out,
-                           int hs_out, int H, int rank, int rot, int* status) {
+                           const float* __restrict__ sink, float scale, int window, __nv_bfloat16* __restrict__ out,
+                           int ld_out, int hs_out, int H, int rank, int rot, int* status) {
   extern __shared__ uint4 tc_smem4[];
   const int Dc = rank + rot, DcP = Dc + 8;
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(tc_smem4);              // [64][DcP]
@@ -498,6 +501,9 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     }
   }
   const int max_pos = ntok > 0 ? positions[first + ntok - 1] : -1;
+  // the first key that any row of the tile sees; the chunk it lies in is the first one walked
+  const int lowest = window > 0 && ntok > 0 ? max(0, positions[first] - window + 1) : 0;
+  const int c_first = lowest / TC_KEYS * TC_KEYS;
 
   const int g = lane >> 2, t4 = lane & 3;
   const int mrow = (warp & 3) * 16;
@@ -514,7 +520,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     for (int j = warp; j < TC_KEYS; j += TC_THREADS / 32) {
       const int key = c0 + j;
       long long off = -1;
-      if (key <= max_pos) {
+      if (key <= max_pos && key >= lowest) {
         const int lp = key / page_size;
         const int page = lp < max_pages ? table[lp] : -1;
         if (page < 0 || page >= num_pages) { if (lane == 0) atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE); }
@@ -534,10 +540,10 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  if (max_pos >= 0) request_chunk(0, 0);
+  if (max_pos >= 0) request_chunk(c_first, 0);
   const bool row_group_live = mrow < rows_used;   // a warp whose 16 rows are all empty only keeps the barriers
   int it = 0;
-  for (int c0 = 0; c0 <= max_pos; c0 += TC_KEYS, ++it) {
+  for (int c0 = c_first; c0 <= max_pos; c0 += TC_KEYS, ++it) {
     const int n_keys = min(TC_KEYS, max_pos - c0 + 1);
     const __nv_bfloat16* Ks = Ks0 + (size_t)(it & 1) * TC_KEYS * DcP;
     const int* ok = row_ok[it & 1];
@@ -584,11 +590,12 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
     {
       const int row = tid >> 2, k0 = (tid & 3) * 8;
       const int pos_r = pos_s[row];
+      const int low_r = window > 0 ? pos_r - window + 1 : 0;
       float sv[8], mx = -CUDART_INF_F;
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const int kk = k0 + e;
-        const bool valid = kk < n_keys && c0 + kk <= pos_r && ok[kk];
+        const bool valid = kk < n_keys && c0 + kk <= pos_r && c0 + kk >= low_r && ok[kk];
         sv[e] = valid ? Ss[(size_t)row * TC_SPAD + kk] : -CUDART_INF_F;
         mx = fmaxf(mx, sv[e]);
       }
@@ -627,7 +634,7 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
         ldsm_x4(a0, a1, a2, a3, a_ptr + ks);
 #pragma unroll
         for (int np = 0; np < NT / 2; ++np) {
-          if (2 * np < nt_used) {
+          if (2 * np < nt_used) {              // an odd last tile takes a neighbour along whose sums nobody reads
             unsigned b0, b1, b2, b3;
             ldsm_x4_trans(b0, b1, b2, b3, b_ptr + (size_t)ks * DcP + np * 16);
             mma_bf16_16816(acc[2 * np], a0, a1, a2, a3, b0, b1);
@@ -658,17 +665,17 @@ latent_attention_tc_kernel(const __nv_bfloat16* __restrict__ q_abs, int ld_qa, i
 // Rows of (token, head) pairs per tile: tokens per tile for a number of heads.
 KVB_EXPORT int kvb_latent_attention_tc_tokens_per_tile(int H) { return H >= TC_ROWS ? 1 : TC_ROWS / H; }
 
-// Whether the tensor-core form takes these sizes: rank a multiple of 32 up to 512, rank + rot a multiple of 16.
+// Whether the tensor-core form takes these sizes: rank and rank + rot multiples of 16, rank up to 512.
 KVB_EXPORT int kvb_latent_attention_tc_supported(int rank, int rot) {
-  return rank >= 32 && rank <= 512 && rank % 32 == 0 && (rank + rot) % 16 == 0 ? 1 : 0;
+  return rank >= 16 && rank <= 512 && rank % 16 == 0 && (rank + rot) % 16 == 0 ? 1 : 0;
 }
 
 template <int NT>
 static int launch_latent_tc(const void* q_abs, int ld_qa, int hs_qa, const void* q_raw, int ld_q, int hs_q,
                             const float* cos_t, const float* sin_t, int table_len, int rdims, const void* pages,
                             const int* block_table, int max_pages, int page_size, int num_pages, const int* positions,
-                            const int* q_start, const int* tiles, int n_tiles, const float* sink, float scale, void* out,
-                            int ld_out, int hs_out, int H, int rank, int rot, int* status, cudaStream_t stream) {
+                            const int* q_start, const int* tiles, int n_tiles, const float* sink, float scale, int window,
+                            void* out, int ld_out, int hs_out, int H, int rank, int rot, int* status, cudaStream_t stream) {
   const int DcP = rank + rot + 8;
   const size_t smem = (size_t)(TC_ROWS + 2 * TC_KEYS) * DcP * 2 + (size_t)TC_ROWS * TC_PPAD * 2 +
                       (size_t)TC_ROWS * TC_SPAD * 4 + 4 * TC_ROWS * 4;
@@ -682,7 +689,7 @@ static int launch_latent_tc(const void* q_abs, int ld_qa, int hs_qa, const void*
   kvb_launch(latent_attention_tc_kernel<NT>, dim3(n_tiles, (H + TC_ROWS - 1) / TC_ROWS), dim3(TC_THREADS), smem, stream,
              (const B*)q_abs, ld_qa, hs_qa, (const B*)q_raw, ld_q, hs_q, cos_t, sin_t, table_len, rdims, (const B*)pages,
              block_table, max_pages, page_size, num_pages, positions, q_start, tiles,
-             kvb_latent_attention_tc_tokens_per_tile(H), sink, scale, (B*)out, ld_out, hs_out, H, rank, rot, status);
+             kvb_latent_attention_tc_tokens_per_tile(H), sink, scale, window, (B*)out, ld_out, hs_out, H, rank, rot, status);
   return kvb_launch_result();
 }
 
@@ -693,16 +700,17 @@ KVB_EXPORT int kvb_latent_attention_tc(const void* q_abs, int ld_qa, int hs_qa, 
                                        const float* cos_t, const float* sin_t, int table_len, int rdims,
                                        const void* pages, const int* block_table, int max_pages, int page_size,
                                        int num_pages, const int* positions, const int* q_start, const int* tiles,
-                                       int n_tiles, const float* sink, float scale, void* out, int ld_out, int hs_out,
-                                       int H, int rank, int rot, int* status, cudaStream_t stream) {
+                                       int n_tiles, const float* sink, float scale, int window, void* out, int ld_out,
+                                       int hs_out, int H, int rank, int rot, int* status, cudaStream_t stream) {
   if (n_tiles <= 0) return 0;
+  if (window < 0) return KVB_ERR_BAD_SIZE;
   if (!kvb_latent_attention_tc_supported(rank, rot) || H < 1 || (rdims & 1) || rdims > rot) return KVB_ERR_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(pages) & 15) || (reinterpret_cast<uintptr_t>(out) & 3) || (ld_out & 1) || (hs_out & 1))
     return KVB_ERR_ALIGN;
 #define KVB_LATENT_TC(NT)                                                                                            \
   return launch_latent_tc<NT>(q_abs, ld_qa, hs_qa, q_raw, ld_q, hs_q, cos_t, sin_t, table_len, rdims, pages,        \
                               block_table, max_pages, page_size, num_pages, positions, q_start, tiles, n_tiles, sink, \
-                              scale, out, ld_out, hs_out, H, rank, rot, status, stream)
+                              scale, window, out, ld_out, hs_out, H, rank, rot, status, stream)
   if (rank <= 64) { KVB_LATENT_TC(4); }
   if (rank <= 128) { KVB_LATENT_TC(8); }
   if (rank <= 256) { KVB_LATENT_TC(16); }

@@ -130,8 +130,6 @@ def kernel_modules_of(spec: ModelSpec, dtype: torch.dtype) -> List[str]:
     from ..models.spec import iter_parts
     mods: List[str] = []
     for family, ps in iter_parts(spec):
-        if family == "block":
-            continue
         cls = lookup(family, ps.kind)
         for m in (cls.kernel_modules(ps.params, dtype) if hasattr(cls, "kernel_modules") else ()):
             if m not in mods:

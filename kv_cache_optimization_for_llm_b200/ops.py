@@ -535,14 +535,14 @@ def conv_silu(x: torch.Tensor, first: int, channels: int, w: torch.Tensor, tails
 # ------------------------------------------------------------------ attention over a cached latent
 
 def latent_prep(d_in: torch.Tensor, q_rank: int, kv_off: int, rank: int, rot: int, rdims: int, wq, wkv, eps: float,
-                cos, sin, batch, block_table, pages: torch.Tensor, write: bool) -> torch.Tensor:
-    """RMS norm of the query latent (returned, [T, q_rank]); RMS norm of the key/value latent and
+                cos, sin, batch, block_table, pages: torch.Tensor, write: bool) -> Optional[torch.Tensor]:
+    """RMS norm of the query latent (returned, [T, q_rank]; ``q_rank`` 0: None); RMS norm of the key/value latent and
     interleaved rotary encoding of the shared key part, both written to the token's cache row."""
     _need_cuda(d_in, pages)
     assert d_in.stride(1) == 1 and pages.is_contiguous() and pages.dtype == d_in.dtype
     assert pages.shape[1] == 1 and pages.shape[3] == rank + rot
     T = d_in.shape[0]
-    cq = new((T, q_rank), d_in.dtype, d_in.device)
+    cq = new((T, q_rank), d_in.dtype, d_in.device) if q_rank else None
     rc = lib("latent_attention").kvb_latent_prep(
         _p(d_in), c_int(d_in.stride(0)), c_int(q_rank), c_int(kv_off), c_int(rank), c_int(rot), c_int(rdims), _p(wq),
         _p(wkv), c_float(eps), _p(cos), _p(sin), c_int(0 if cos is None else cos.shape[0]), _p(batch.positions),
@@ -635,9 +635,9 @@ def _query_tiles(batch, nt: int) -> torch.Tensor:
 
 def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_head_stride: int, cos, sin, rdims: int,
                      pages: torch.Tensor, block_table, batch, sink: Optional[torch.Tensor], scale: float, heads: int,
-                     rank: int, rot: int) -> torch.Tensor:
+                     rank: int, rot: int, window: int = 0) -> torch.Tensor:
     """Causal attention of every token over its request's cached rows [latent | rotated part],
-    all heads sharing the rows; softmax with a sink per head (``sink`` None: without).  ``q_abs`` [T, heads * rank]: the
+    all heads sharing the rows; query i sees key j when ``0 <= i - j < window`` (``window`` 0: every key up to i); softmax with a sink per head (``sink`` None: without).  ``q_abs`` [T, heads * rank]: the
     queries' plain parts moved into the latent's space; ``q`` holds head h's part to be rotated at
     ``rot_first + h * q_head_stride``.  Returns the attended latents [T, heads * rank]."""
     _need_cuda(q_abs, pages)
@@ -656,8 +656,8 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_hea
             _p(q_abs), c_int(q_abs.stride(0)), c_int(rank), c_void_p(_at(q, rot_first)), c_int(q.stride(0)),
             c_int(q_head_stride), _p(cos), _p(sin), c_int(0 if cos is None else cos.shape[0]), c_int(rdims), _p(pages),
             _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]), c_int(pages.shape[0]),
-            _p(batch.positions), _p(batch.q_start), _p(tiles), c_int(n_tiles), _p(sink), c_float(scale), _p(out),
-            c_int(out.stride(0)), c_int(rank), c_int(heads), c_int(rank), c_int(rot), _p(batch.status), _stream())
+            _p(batch.positions), _p(batch.q_start), _p(tiles), c_int(n_tiles), _p(sink), c_float(scale), c_int(int(window or 0)),
+            _p(out), c_int(out.stride(0)), c_int(rank), c_int(heads), c_int(rank), c_int(rot), _p(batch.status), _stream())
         _check(rc, "latent_attention_tc")
         choices["latent_attention_tc"] += 1
         return out
@@ -665,8 +665,8 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_hea
         _p(q_abs), c_int(q_abs.stride(0)), c_int(rank), c_void_p(_at(q, rot_first)), c_int(q.stride(0)),
         c_int(q_head_stride), _p(cos), _p(sin), c_int(0 if cos is None else cos.shape[0]), c_int(rdims), _p(pages),
         _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]), c_int(pages.shape[0]), _p(batch.positions),
-        _p(batch.token_req), _p(sink), c_float(scale), _p(out), c_int(out.stride(0)), c_int(rank), c_int(T),
-        c_int(heads), c_int(rank), c_int(rot), c_int(dtype_code(q_abs.dtype)), _p(batch.status), _stream())
+        _p(batch.token_req), _p(sink), c_float(scale), c_int(int(window or 0)), _p(out), c_int(out.stride(0)), c_int(rank),
+        c_int(T), c_int(heads), c_int(rank), c_int(rot), c_int(dtype_code(q_abs.dtype)), _p(batch.status), _stream())
     _check(rc, "latent_attention")
     choices["latent_attention"] += 1
     return out
@@ -1447,7 +1447,8 @@ def gated_group_norm(y: torch.Tensor, z, weight: torch.Tensor, groups: int, eps:
 # ------------------------------------------------------------------ routed experts
 
 def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], experts: int, identity: int, top: int,
-          scale: float, logits: Optional[torch.Tensor] = None, score: str = "softmax", renormalize: bool = True):
+          scale: float, logits: Optional[torch.Tensor] = None, score: str = "softmax", renormalize: bool = True,
+          groups: int = 0, keep_groups: int = 0):
     """The router of a feed-forward of many experts.  ``w_router`` float32 [experts + identity, K],
     ``correction`` float32 [experts + identity] (added to the scores for the choice only).  Returns
     ``gate`` float32 [T, experts + identity], a token's weight for every expert (0 where not chosen), and
@@ -1456,7 +1457,9 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
     product that adds up in float32; further columns behind them are left alone), in which case the kernel only
     chooses.  ``score`` "softmax": the scores are the logits' softmax over all experts; "sigmoid": each logit's sigmoid.
     ``renormalize`` False: a chosen expert's weight is its score times ``scale``, not divided by the chosen scores' sum.
-    ``correction`` None: the choice goes by the scores alone."""
+    ``correction`` None: the choice goes by the scores alone.  ``groups`` > 0: the experts form that many equal groups of
+    neighbours; a group is judged by the sum of its two largest choice scores, and only experts of the ``keep_groups``
+    best groups can be chosen."""
     _need_cuda(h, w_router)
     T, K = h.shape
     n_all = experts + identity
@@ -1473,7 +1476,7 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
                                   c_int(0 if logits is None else logits.stride(0)), _p(correction), _p(gate), _p(idw), c_int(T),
                                   c_int(K), c_int(experts), c_int(identity), c_int(top), c_float(scale),
                                   c_int({"softmax": 0, "sigmoid": 1}[score]), c_int(1 if renormalize else 0),
-                                  c_int(dtype_code(h.dtype)), _stream())
+                                  c_int(int(groups)), c_int(int(keep_groups)), c_int(dtype_code(h.dtype)), _stream())
     _check(rc, "route")
     return gate, idw
 
@@ -1490,26 +1493,44 @@ def expert_act(p: torch.Tensor, gate: torch.Tensor, experts: int, ff: int, share
     return out
 
 
-def limited_act(p: torch.Tensor, gate: torch.Tensor, shared_logit: Optional[torch.Tensor], experts: int, ff: int,
+def limited_act(p: torch.Tensor, gate: Optional[torch.Tensor], shared_logit: Optional[torch.Tensor], experts: int, ff: int,
                 shared_ff: int, pad: int, limit: float, shared_limit: float, alpha: float,
-                weigh_output: bool = False) -> torch.Tensor:
-    """The activation of experts ``down(a(g) (u + 1))`` with ``g = min(w gate.h, limit)``, ``u = clamp(w up.h, +-limit)``,
+                weigh_output: bool = False, offset: float = 1.0) -> torch.Tensor:
+    """The activation of experts ``down(a(g) (u + offset))`` with ``g = min(w gate.h, limit)``, ``u = clamp(w up.h, +-limit)``,
     ``a(g) = g sigmoid(alpha g)`` and ``w`` the token's weight for the expert (``gate`` float32 [T, >= experts], 0 where
     not chosen).  ``p`` [T, 2 (experts ff + shared_ff)]: per expert its gate product, then its up product; behind
     them those of an expert that every token uses, whose result is multiplied by ``sigmoid(shared_logit[t])`` (float32
-    column, may be a strided view; None: by 1).  ``weigh_output``: the weight multiplies ``a(g) (u + 1)`` instead of the
-    two first products.  Returns [T, experts ff + shared_ff + pad], the padding zero."""
+    column, may be a strided view; None: by 1).  ``weigh_output``: the weight multiplies ``a(g) (u + offset)`` instead of the
+    two first products.  An infinite ``limit``, ``alpha`` 1 and ``offset`` 0 are the plain gated form ``silu(gate.h) up.h``.
+    ``experts`` 0 (``gate`` None): only the feed-forward that every token uses.  Returns [T, experts ff + shared_ff + pad], the padding zero."""
     _need_cuda(p, gate)
-    assert p.stride(1) == 1 and gate.dtype == torch.float32 and gate.stride(1) == 1
+    assert p.stride(1) == 1 and (experts == 0 or (gate.dtype == torch.float32 and gate.stride(1) == 1))
     assert shared_logit is None or (shared_logit.dtype == torch.float32 and shared_logit.shape[0] == p.shape[0])
     width = experts * ff + shared_ff + pad
     out = new((p.shape[0], width), p.dtype, p.device)
-    rc = lib("experts").kvb_limited_act(_p(p), c_int(p.stride(0)), _p(gate), c_int(gate.stride(0)), _p(shared_logit),
+    rc = lib("experts").kvb_limited_act(_p(p), c_int(p.stride(0)), _p(gate), c_int(0 if gate is None else gate.stride(0)),
+                                        _p(shared_logit),
                                         c_int(0 if shared_logit is None else shared_logit.stride(0)), _p(out),
                                         c_int(p.shape[0]), c_int(experts), c_int(ff), c_int(shared_ff), c_int(pad),
-                                        c_float(limit), c_float(shared_limit), c_float(alpha), c_int(1 if weigh_output else 0),
+                                        c_float(limit), c_float(shared_limit), c_float(alpha), c_float(offset), c_int(1 if weigh_output else 0),
                                         c_int(dtype_code(p.dtype)), _stream())
     _check(rc, "limited_act")
+    return out
+
+
+def token_gate(p: torch.Tensor, table: torch.Tensor, first: int, batch, width: int) -> torch.Tensor:
+    """``gelu_tanh(p[t, j]) * table[token[t], first + j]`` for every column j of ``p``; the result is ``width`` columns
+    wide, those behind ``p``'s zero.  Tokens that are still on the device are found as in :func:`embed_gather`."""
+    _need_cuda(p, table)
+    assert p.stride(1) == 1 and table.is_contiguous() and table.dtype == p.dtype and width >= p.shape[1]
+    T, n = p.shape
+    out = new((T, width), p.dtype, p.device)
+    sampled = batch.sampled
+    rc = lib("token_input").kvb_token_gate(_p(p), c_int(p.stride(0)), _p(table), c_int(table.shape[1]), c_int(int(first)),
+                                           c_int(table.shape[0]), _p(batch.token_ids), _p(sampled),
+                                           c_int(0 if sampled is None else sampled.numel()), _p(out), c_int(T), c_int(n),
+                                           c_int(width), c_int(dtype_code(p.dtype)), _p(batch.status), _stream())
+    _check(rc, "token_gate")
     return out
 
 

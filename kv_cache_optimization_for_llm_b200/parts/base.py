@@ -23,6 +23,7 @@ nothing of the model it sits in.  Interfaces by family:
                  kept for the step when a stream part sets ``needs_embedding``; or what the part's
                  ``from_embedding(residual)`` made of it at the step's start, once for all parts with the same
                  ``embedding_key``)
+* token_input:   ``forward(x, batch) -> delta``: what a layer makes of its tokens' own rows and the stream
 * embedding:     ``forward(batch) -> residual``  (float32 [T, hidden])
 * head:          ``forward(x) -> logits``  (float32 [rows, vocab])
 """

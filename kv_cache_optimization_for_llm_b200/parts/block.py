@@ -114,6 +114,10 @@ class PostNormBlock(Part):
 
     part_families = {"mixer": "mixer", "mixer_post_norm": "norm", "feed_forward": "feed_forward", "ff_post_norm": "norm"}
 
+    @classmethod
+    def kernel_modules(cls, params, dtype):
+        return ("rowwise",)
+
     def __init__(self, parts):
         self.parts = dict(parts)
         self.mixer, self.mixer_post = parts["mixer"], parts["mixer_post_norm"]
@@ -140,6 +144,30 @@ class PostNormMixerBlock(PostNormBlock):
     """The post-norm block of a layer that has no feed-forward: ``h += post1(mixer(h))``."""
 
     part_families = {"mixer": "mixer", "mixer_post_norm": "norm"}
+
+
+@register("block", "postnorm_token_input")
+class PostNormTokenInputBlock(PostNormBlock):
+    """The post-norm block with a third branch behind the feed-forward, fed by the tokens themselves:
+    ``h += post1(mixer(h)); h += post2(ff(h)); h += post3(token_input(h))``."""
+
+    part_families = {**PostNormBlock.part_families, "token_input": "token_input", "token_input_post_norm": "norm"}
+
+    def __init__(self, parts):
+        super().__init__(parts)
+        self.token_input, self.token_input_post = parts["token_input"], parts["token_input_post_norm"]
+
+    def forward(self, residual, delta, batch, cache):
+        residual, pending = super().forward(residual, delta, batch, cache)
+        x = ops.add_norm(residual, pending, "copy", None, 0.0, self.mixer.ctx.dtype)
+        return residual, self.token_input_post.as_pending(self.token_input.forward(x, batch))
+
+
+@register("block", "postnorm_token_input_mixer_only")
+class PostNormTokenInputMixerBlock(PostNormTokenInputBlock):
+    """The same of a layer that has no feed-forward: ``h += post1(mixer(h)); h += post3(token_input(h))``."""
+
+    part_families = {n: f for n, f in PostNormTokenInputBlock.part_families.items() if n not in ("feed_forward", "ff_post_norm")}
 
 
 @register("block", "parallel")

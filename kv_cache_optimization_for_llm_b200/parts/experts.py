@@ -98,10 +98,14 @@ class RoutedExperts(Part):
 class LimitedExperts(Part):
     """``experts`` gated feed-forward layers without biases, of which a token uses ``top``:
 
-        g = min(W_gate x, limit),   u = clamp(W_up x, -limit, limit),   expert(x) = W_down (g sigmoid(alpha g) (u + 1)).
+        g = min(W_gate x, limit),   u = clamp(W_up x, -limit, limit),   expert(x) = W_down (g sigmoid(alpha g) (u + offset)).
 
+    (``limit`` None: no limits; with ``alpha`` 1 and ``offset`` 0 that is ``W_down (silu(W_gate x) W_up x)``.)
     The router's logits ``W_r h`` are float32.  ``score`` "sigmoid" (the default): the scores are their sigmoids, each by
-    itself; the ``top`` experts with the largest scores are chosen and weighted with their scores as they are.
+    itself; the ``top`` experts with the largest scores are chosen and weighted with their scores as they are.  With
+    ``correction`` a learned number per expert joins the score for the choice only.  With ``groups`` the experts form that
+    many equal groups of neighbours, a group is judged by the sum of its two largest choice scores, and only experts of
+    the ``keep_groups`` best groups can be chosen.
     "softmax_chosen": the ``top`` experts of the highest logits, each weighing its share of a softmax that leaves out all others.
     ``weigh`` "input" (the default): the weight multiplies the expert's *input*, the layer's output is the sum of
     ``expert(w h)`` over the chosen experts; "output": the sum of ``w expert(h)``.  With ``shared_ff`` > 0 one more
@@ -116,12 +120,15 @@ class LimitedExperts(Part):
     shared expert's gate multiplies its activation, which for a last matrix without bias is the same as multiplying its
     output.  The router's rows and the shared gate's row are one small product with float32 results.  Every expert is
     computed for every token (see :class:`RoutedExperts` for what that costs).
-    params: hidden_size, experts, top, expert_ff, limit, shared_ff, shared_limit, alpha, score, weigh."""
+    params: hidden_size, experts, top, expert_ff, limit, shared_ff, shared_limit, alpha, offset, score, weigh, correction,
+    groups, keep_groups."""
 
     @classmethod
     def weight_specs(cls, params):
         h, E, F, S = (int(params[k]) for k in ("hidden_size", "experts", "expert_ff", "shared_ff"))
         specs = {"router": WeightSpec((E, h))}
+        if params.get("correction"):
+            specs["correction"] = WeightSpec((E,), "bias")
         for e in range(E):
             specs[f"gate{e}"] = WeightSpec((F, h))
             specs[f"up{e}"] = WeightSpec((F, h))
@@ -140,9 +147,15 @@ class LimitedExperts(Part):
         self.hidden = int(params["hidden_size"])
         self.E, self.top = int(params["experts"]), int(params["top"])
         self.F, self.S = int(params["expert_ff"]), int(params.get("shared_ff") or 0)
-        self.limit = float(params["limit"])
+        self.limit = float("inf") if params["limit"] is None else float(params["limit"])
         self.shared_limit = float(params.get("shared_limit") or self.limit)
-        self.alpha = float(params.get("alpha", 1.702))
+        self.alpha, self.offset = float(params.get("alpha", 1.702)), float(params.get("offset", 1.0))
+        self.correction = weights.get("correction")
+        self.groups = int(params.get("groups") or 0)
+        self.keep_groups = int(params.get("keep_groups") or 0)
+        if self.groups and (self.E % self.groups or not 1 <= self.keep_groups <= self.groups):
+            raise ValueError(f"limited_experts: {self.E} experts in {self.groups} equal groups of which {self.keep_groups} are "
+                             "kept is refused")
         self.score, self.weigh = str(params.get("score", "sigmoid")), str(params.get("weigh", "input"))
         if self.score not in ("sigmoid", "softmax_chosen") or self.weigh not in ("input", "output"):
             raise ValueError(f"limited_experts: score {self.score!r} (sigmoid, softmax_chosen) or weigh {self.weigh!r} "
@@ -174,9 +187,10 @@ class LimitedExperts(Part):
         logits = ops.linear(x, self.small, out_dtype=torch.float32)
         # a softmax over all experts, divided by the sum of the chosen, is the softmax over the chosen
         chosen_only = self.score == "softmax_chosen"
-        gate, _ = ops.route(x, None, None, self.E, 0, self.top, 1.0, logits, score="softmax" if chosen_only else "sigmoid",
-                            renormalize=chosen_only)
+        gate, _ = ops.route(x, None, self.correction, self.E, 0, self.top, 1.0, logits,
+                            score="softmax" if chosen_only else "sigmoid", renormalize=chosen_only, groups=self.groups,
+                            keep_groups=self.keep_groups)
         p = ops.linear(x, self.first)
         a = ops.limited_act(p, gate, logits[:, self.E] if self.S else None, self.E, self.F, self.S, self.pad, self.limit,
-                            self.shared_limit, self.alpha, weigh_output=self.weigh == "output")
+                            self.shared_limit, self.alpha, weigh_output=self.weigh == "output", offset=self.offset)
         return ops.linear(a, self.down)

@@ -132,3 +132,39 @@ class DenseXIELU(Part):
 
     def forward(self, x, batch):
         return ops.linear(ops.xielu(ops.linear(x, self.up), self.act), self.down)
+
+
+@register("feed_forward", "limited_dense")
+class LimitedDense(Part):
+    """``down( g sigmoid(alpha g) (u + offset) )`` with ``g = min(gate(x), limit)`` and ``u = clamp(up(x), -limit, limit)``, no
+    biases: the form that :class:`..experts.LimitedExperts` has chosen by a router, here for every token.
+    params: hidden_size, intermediate_size, limit, alpha (1.702), offset (1)."""
+
+    @classmethod
+    def weight_specs(cls, params):
+        h, i = int(params["hidden_size"]), int(params["intermediate_size"])
+        return {"gate": WeightSpec((i, h)), "up": WeightSpec((i, h)), "down": WeightSpec((h, i))}
+
+    @classmethod
+    def kernel_modules(cls, params, dtype):
+        return ("experts",) + (("gemm_f32",) if dtype == torch.float32 else ("gemm_bf16", "gemm_bf16_wide"))
+
+    def __init__(self, params, weights, ctx):
+        super().__init__(params, weights, ctx)
+        self.inter, self.limit = int(params["intermediate_size"]), float(params["limit"])
+        self.alpha, self.offset = float(params.get("alpha", 1.702)), float(params.get("offset", 1.0))
+        self.gate_up = torch.cat([weights["gate"], weights["up"]], dim=0).contiguous()
+        # the second product's inner size is padded to a multiple of 8 (16-byte rows), the padding being zeros
+        self.pad = -self.inter % 8
+        down = weights["down"]
+        if self.pad:
+            down = torch.cat([down, down.new_zeros((down.shape[0], self.pad))], dim=1)
+        self.down = down.contiguous()
+
+    def activation_widths(self):
+        return [2 * self.inter, self.inter + self.pad, self.down.shape[0]]
+
+    def forward(self, x, batch):
+        a = ops.limited_act(ops.linear(x, self.gate_up), None, None, 0, 1, self.inter, self.pad, self.limit, self.limit, self.alpha,
+                            offset=self.offset)
+        return ops.linear(a, self.down)

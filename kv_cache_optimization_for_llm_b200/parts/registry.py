@@ -5,7 +5,7 @@ from __future__ import annotations
 
 from typing import Dict
 
-FAMILIES = ("embedding", "mixer", "feed_forward", "norm", "position", "block", "head", "stream")
+FAMILIES = ("embedding", "mixer", "feed_forward", "norm", "position", "block", "head", "stream", "token_input")
 _REG: Dict[str, Dict[str, type]] = {f: {} for f in FAMILIES}
 
 
@@ -36,4 +36,4 @@ def known(family: str):
 
 def _load_builtin() -> None:
     from . import (attention, block, delta_rule, embedding, experts, feed_forward, hyper, latent_attention, norm,  # noqa: F401
-                   position, recurrence, stream, window_attention)
+                   position, recurrence, stream, token_input, window_attention)

@@ -115,7 +115,8 @@ class ShapedWindowAttention(Part):
 
     q (``heads`` x ``dim``), k (``kv_heads`` x ``dim``) and v (``kv_heads`` x ``vdim``) come from one product with the
     row-stacked matrix; with ``bias`` each gets a bias; with ``qk_norm`` every query and key head is divided by its
-    root mean square (eps inside the root) and multiplied by a weight of ``dim`` shared by the heads.  Keys and values
+    root mean square (eps inside the root) and multiplied by a weight of ``dim`` shared by the heads ("unweighted": no
+    weight).  Keys and values
     go to the request's pages, a row [k | v] per token and key/value head.  No rotation.  For query i and key j
 
         s = (q . k) * scale * temp[h];    s <- softcap * tanh(s / softcap);    s <- s - slope_h * (i - j),
@@ -135,7 +136,7 @@ class ShapedWindowAttention(Part):
         if params.get("bias"):
             specs.update(q_bias=WeightSpec((H * D,), "bias"), k_bias=WeightSpec((G * D,), "bias"),
                          v_bias=WeightSpec((G * Dv,), "bias"))
-        if params.get("qk_norm"):
+        if params.get("qk_norm") and params["qk_norm"] != "unweighted":
             specs.update(q_norm=WeightSpec((D,), "vector"), k_norm=WeightSpec((D,), "vector"))
         if params.get("head_temperature"):
             specs["temp"] = WeightSpec((H,), "bias")
@@ -146,12 +147,22 @@ class ShapedWindowAttention(Part):
         if dtype == torch.float32:
             return ("window_attention", "gemm_f32")
         flash = ("window_flash_attention",) if cls._flash_sizes(params, dtype) else ()
+        if cls._plain_rows(params, dtype):
+            flash += ("flash_attention",)
         return ("window_attention",) + flash + ("gemm_bf16", "gemm_bf16_wide")
 
     @staticmethod
     def _flash_sizes(params, dtype, page_size=16):
         return ops.window_flash_attention_supported(int(params["dim"]), int(params["vdim"]),
                                                     int(params["heads"]) // max(1, int(params["kv_heads"])), page_size, dtype)
+
+    @staticmethod
+    def _plain_rows(params, dtype):
+        """Scores that nothing shapes, over keys and values of one size that the tcgen05 kernel of prompt portions takes
+        (bfloat16, 64 or 128)."""
+        return (dtype == torch.bfloat16 and int(params["dim"]) == int(params["vdim"]) and int(params["dim"]) in (64, 128)
+                and not params.get("softcap") and not params.get("head_temperature") and params.get("slope_power") is None
+                and float(params.get("out_scale", 1.0)) == 1.0)
 
     def __init__(self, params, weights, ctx):
         super().__init__(params, weights, ctx)
@@ -169,6 +180,8 @@ class ShapedWindowAttention(Part):
         self.w_in, (_, self.k_off, self.v_off) = _stack_rows([weights["q"], weights["k"], weights["v"]])
         self.q_bias, self.k_bias, self.v_bias = (weights.get(n) for n in ("q_bias", "k_bias", "v_bias"))
         self.q_norm, self.k_norm = weights.get("q_norm"), weights.get("k_norm")
+        if params.get("qk_norm") == "unweighted":
+            self.q_norm = self.k_norm = torch.ones(self.dim, dtype=torch.float32, device=ctx.device)
         self.temp = weights.get("temp")
         self.slopes = None
         if params.get("slope_power") is not None:
@@ -189,7 +202,10 @@ class ShapedWindowAttention(Part):
         if not self._flash_sizes(self.params, self.ctx.dtype):
             return []
         g = self.heads // self.kv_heads
-        return [ops.rows_tokens_per_tile(g, False), ops.rows_tokens_per_tile(g, True)]
+        heights = [ops.rows_tokens_per_tile(g, False), ops.rows_tokens_per_tile(g, True)]
+        if self._plain_rows(self.params, self.ctx.dtype):
+            heights += [ops.flash_tokens_per_tile(g, True)]
+        return heights
 
     def readout(self, p, first, batch, cache):
         """From the product ``p`` (this mixer's columns start at ``first``) to the heads' results [T, heads * vdim]."""
@@ -197,6 +213,12 @@ class ShapedWindowAttention(Part):
         q = ops.qk_norm_append(p, first, self.k_off, self.v_off, self.q_bias, self.k_bias, self.v_bias, self.q_norm,
                                self.k_norm, self.eps, cache.k, table, batch, self.heads, self.kv_heads, self.dim,
                                self.vdim, write=cache.write)
+        if (not batch.decode_only and self._plain_rows(self.params, self.ctx.dtype)
+                and ops.flash_attention_rows_masked_wanted(batch, self.heads, self.kv_heads, self.dim, self.vdim,
+                                                           cache.page_size, self.ctx.dtype, q)):
+            # long bfloat16 steps: the tcgen05 kernel with roles
+            return ops.flash_attention_rows(q, cache.k, table, batch, self.heads, self.kv_heads, self.dim, self.scale,
+                                            self.window or 0, 0, False, wide=3)
         if not batch.decode_only and self._flash_sizes(self.params, self.ctx.dtype, cache.page_size):
             return ops.window_flash_attention(q, cache.k, table, batch, self.heads, self.kv_heads, self.dim, self.vdim,
                                               self.scale, self.window or 0, 0, False, head_scale=self.temp,
