@@ -503,6 +503,28 @@ def zatusun_config(z, chunk=1024):
             "loop": {"start": n // 2, "stop": n, "times": 1}}
 
 
+def lobuzen_config(z, window=1024):
+    """Six layers at the comparison's sizes: a latent attention of Rezusun's sizes (no rotated part, a sink per head), one
+    that attends to that layer's latents, and an attention with heads of 64 and a quarter as many key/value heads, all three
+    over a window of 1024 tokens; a dense feed-forward of Llama's width on the first layer, on the others 32 experts in four
+    groups of which two are kept, four experts a token, of the width of Zatusun's; behind every layer a vector of a
+    sixteenth of the width from each token."""
+    H, W = z["heads"], z["width"]
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 32 + z["ff"] // 128},
+           "router": {"experts": 32, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "vdim": z["lat_vdim"], "kv_rank": z["kv_rank"],
+           "scale": z["lat_dim"] ** -0.5, "mask": {"size": window}}
+    att = {"heads": H, "kv_heads": H // 4, "dim": 64, "vdim": 64, "scale": 0.125, "mask": {"size": window}}
+    layers = []
+    for i in range(z["layers"]):
+        kind = i % 3
+        mixer = att if kind == 2 else (dict(lat, kv_from=i - 1) if kind == 1 else lat)
+        layers.append({"type": "attention" if kind == 2 else "latent_attention", "mixer": mixer, "mlp": moe if i else dense})
+    return {"architecture": "Lobuzen", "vocab": z["vocab"], "width": W, "norm": {"eps": 1e-6}, "token_side": {"dim": W // 16},
+            "layers": layers, "max_position_embeddings": CONTEXT_LEN}
+
+
 def llama_config_like(z):
     cfg = dict(LLAMA_1B)
     cfg.update(hidden_size=z["width"], intermediate_size=z["ff"], vocab_size=z["vocab"], num_hidden_layers=z["layers"],
@@ -909,6 +931,94 @@ def run_compare_zatusun(size):
             "kernel_roofline_fractions": kernels, "clocks": sampler.summary(list(_compare_windows) or [(w0, w1)])}
 
 
+def run_compare_lobuzen(size):
+    """The Lobuzen design beside the two closest on the engine at equal width, depth and vocabulary: Zatusun (latent
+    attention, experts without a shared one) and Tevanex (norms behind the sublayers only, attention with heads of 64 over
+    [key | value] rows in a windowed page group)."""
+    z = COMPARE_SIZES[size]
+    pk = peaks()
+    sampler = ClockSampler()
+    sampler.start()
+    w0 = time.perf_counter()
+    window = 1024
+    log(f"{size}: Tevanex")
+    tev = measure_design(tevanex_config(z, window))
+    log(f"{size}: Zatusun")
+    zat = measure_design(zatusun_config(z, window))
+    log(f"{size}: Lobuzen")
+    lob = measure_design(lobuzen_config(z, window))
+    w1 = time.perf_counter()
+    sampler.stop()
+    T, R, ctx = PREFILL_TOKENS, 64, PROMPT_LEN
+    H, G, W, n = z["heads"], z["heads"] // 4, z["width"], z["layers"]
+    pairs = T * (T + 1) // 2
+    seen = sum(min(i + 1, window) for i in range(T))
+    in_block = sum(i % window + 1 for i in range(T))
+    dc, kr, side = z["kv_rank"] + z["lat_rot"], z["kv_rank"], z["width"] // 16
+    tev_cols = 32 * (z["ff"] // 32) + z["ff"] // 4
+    moe_cols = 32 * (z["ff"] // 32 + z["ff"] // 128)
+    lob_cols = (z["ff"] + (n - 1) * moe_cols) / n
+    tev_qkv = ((H + 2 * G) * 64 + (H // 2 + 2 * (H // 8)) * 128) / 2
+
+    def per_launch(d, phase, key, *names):
+        for name in names:
+            calls, ms = d[phase][key].get(name, (0, 0.0))
+            if calls:
+                return ms / calls
+        return None
+
+    def frac(work, ms, peak_per_s):
+        return None if not ms else round(work / (ms * 1e-3) / peak_per_s, 4)
+    tensor, hbm = pk["bf16_tflops"] * 1e12, pk["hbm_gbs"] * 1e9
+    pre, dec = ("prefill_2048", "operators"), ("decode_b64", "operators_launched")
+    lat_names = ("latent_attention_tc", "latent_attention")
+    att_names = ("flash_attention_rows", "window_flash_attention", "window_attention")
+    kernels = {
+        "zatusun latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
+            pairs * z["lat_heads"] * 2 * (dc + kr), per_launch(zat, *pre, *lat_names), tensor),
+        "lobuzen latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
+            seen * z["lat_heads"] * 2 * (kr + kr), per_launch(lob, *pre, *lat_names), tensor),
+        "zatusun latent_attention, batch 64 (of the measured copy peak)": frac(
+            R * ctx * dc * 2, per_launch(zat, *dec, *lat_names), hbm),
+        "lobuzen latent_attention, batch 64 (of the measured copy peak)": frac(
+            R * min(ctx, window) * kr * 2, per_launch(lob, *dec, *lat_names), hbm),
+        "zatusun latent_prep, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * (z["q_rank"] + dc) * 2, per_launch(zat, *pre, "latent_prep"), hbm),
+        "lobuzen latent_prep, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * kr * 2, per_launch(lob, *pre, "latent_prep"), hbm),
+        "tevanex attention, 2048 tokens (of the measured bf16 peak)": frac(
+            in_block * 4 * H * 64, per_launch(tev, *pre, *att_names), tensor),
+        "lobuzen attention, 2048 tokens (of the measured bf16 peak)": frac(
+            seen * 4 * H * 64, per_launch(lob, *pre, *att_names), tensor),
+        "tevanex window_attention, batch 64 (of the measured copy peak)": frac(
+            R * min(ctx, window) * 2 * G * 64 * 2, per_launch(tev, *dec, "window_attention"), hbm),
+        "lobuzen window_attention, batch 64 (of the measured copy peak)": frac(
+            R * min(ctx, window) * 2 * G * 64 * 2, per_launch(lob, *dec, "window_attention"), hbm),
+        "tevanex qk_rot_append, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * tev_qkv * 2, per_launch(tev, *pre, "qk_rot_append"), hbm),
+        "lobuzen qk_norm_append, 2048 tokens (of the measured copy peak)": frac(
+            T * 2 * (H + 2 * G) * 64 * 2, per_launch(lob, *pre, "qk_norm_append"), hbm),
+        "tevanex add_norm, 2048 tokens (of the measured copy peak)": frac(T * W * 12, per_launch(tev, *pre, "add_norm"), hbm),
+        "lobuzen add_norm, 2048 tokens (of the measured copy peak)": frac(T * W * 12, per_launch(lob, *pre, "add_norm"), hbm),
+        "tevanex limited_act, 2048 tokens (of the measured copy peak)": frac(
+            T * tev_cols * 6, per_launch(tev, *pre, "limited_act"), hbm),
+        "zatusun limited_act, 2048 tokens (of the measured copy peak)": frac(
+            T * moe_cols * 6, per_launch(zat, *pre, "limited_act"), hbm),
+        "lobuzen limited_act, 2048 tokens (of the measured copy peak)": frac(
+            T * lob_cols * 6, per_launch(lob, *pre, "limited_act"), hbm),
+        "zatusun route, 2048 tokens (of the measured copy peak)": frac(T * (32 + 32) * 4, per_launch(zat, *pre, "route"), hbm),
+        "lobuzen route, 2048 tokens (of the measured copy peak)": frac(T * (32 + 32) * 4, per_launch(lob, *pre, "route"), hbm),
+        # the gate products and the table's rows read, the gated rows written
+        "lobuzen token_gate, 2048 tokens (of the measured copy peak)": frac(T * side * 6, per_launch(lob, *pre, "token_gate"), hbm),
+        # both matrices, the pending branch output read, the stream read and written, its copy written
+        "lobuzen token_input_step, batch 64 (of the measured copy peak)": frac(
+            2 * W * side * 2 + R * W * 12, per_launch(lob, *dec, "token_input_step"), hbm),
+    }
+    return {"compare": size, "design": "lobuzen", "beside": "tevanex, zatusun", "sizes": z, "window": window, "dtype": "bf16",
+            "data": "synthetic", "peaks": pk, "tevanex": tev, "zatusun": zat, "lobuzen": lob,
+            "kernel_roofline_fractions": kernels, "clocks": sampler.summary(list(_compare_windows) or [(w0, w1)])}
+
+
 def run_compare(size):
     """The Rezusun design beside Llama at equal width, depth, feed-forward and vocabulary."""
     z = COMPARE_SIZES[size]
@@ -985,14 +1095,15 @@ def main():
                     help="instead of the headline: prefill and decode of another design (--design) beside a Llama model of "
                          "equal width, depth, feed-forward and vocabulary (random weights), with the time of every "
                          "operator and roofline fractions of the designs' own kernels; prints its own JSON line")
-    ap.add_argument("--design", default="rezusun", choices=["rezusun", "solulix", "nonetar", "tevanex", "zatusun"],
+    ap.add_argument("--design", default="rezusun", choices=["rezusun", "solulix", "nonetar", "tevanex", "zatusun", "lobuzen"],
                     help="with --compare: which design stands beside Llama (nonetar and tevanex: beside Solulix; zatusun: "
-                         "beside Tevanex and Rezusun, the closest designs)")
+                         "beside Tevanex and Rezusun; lobuzen: beside Tevanex and Zatusun, the closest designs)")
     args = ap.parse_args()
 
     if args.compare:
         result = {"solulix": run_compare_solulix, "nonetar": run_compare_nonetar,
-                  "tevanex": run_compare_tevanex, "zatusun": run_compare_zatusun}.get(args.design, run_compare)(args.compare)
+                  "tevanex": run_compare_tevanex, "zatusun": run_compare_zatusun,
+                  "lobuzen": run_compare_lobuzen}.get(args.design, run_compare)(args.compare)
         print(json.dumps(result), flush=True)
         return 0
     if args.impl == "reference":

@@ -4,6 +4,8 @@
 //
 //   * token_gate_kernel: for steps whose two products are made by the step's matrix product kernels: the middle,
 //     a[t, j] = gelu_tanh(p[t, j]) * table[token, first + j].
+//   * token_input_step_kernel: for steps of few tokens: all of it in one launch, the norm and the addition of the
+//     branch that is still pending in front of it included.
 #include "common.cuh"
 
 __device__ __forceinline__ float gelu_tanh(float z) {
@@ -53,4 +55,296 @@ KVB_EXPORT int kvb_token_gate(const void* p, int ld_p, const void* table, int ld
                                             (const T*)table, ld_table, first, V, ids, sampled, n_sampled, (T*)out, n,
                                             ld_out, total, status)));
   return kvb_launch_result();
+}
+
+// ---------------------------------------------------------------- the whole branch in one launch
+// A cluster of kStepBlocks blocks takes NT tokens.  Block r owns columns [c0, c1) of the stream, for the rows of x, for
+// the columns of W_g and for the rows of W_p alike, so the stream itself never leaves its block; what crosses the
+// cluster (written into every block's shared memory, then one hardware barrier) is three sets of partial sums: the
+// squares of the pending branch output, the products W_g x, and the squares of y.  Both products run on plain FMAs:
+// the weights are read once per cluster, and a step of few tokens is bound by bringing them.  Their lines are requested
+// into L2 before the kernel waits for its predecessor.
+// Every sum is taken in an order that depends on the sizes only.
+constexpr int kStepBlocks = 8, kStepThreads = 256, kStepWarps = kStepThreads / 32;
+
+__device__ __forceinline__ void cluster_meet() {
+  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// v into the same place of block `rank`'s shared memory
+__device__ __forceinline__ void store_in_block(float* p, int rank, float v) {
+  unsigned local = (unsigned)__cvta_generic_to_shared(p), remote;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
+  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
+}
+
+template <typename T> struct Piece;      // 16 bytes of a row
+template <> struct Piece<float> {
+  static constexpr int N = 4;
+  static __device__ __forceinline__ void open(const uint4& u, float* f) {
+    f[0] = __uint_as_float(u.x); f[1] = __uint_as_float(u.y); f[2] = __uint_as_float(u.z); f[3] = __uint_as_float(u.w);
+  }
+};
+template <> struct Piece<__nv_bfloat16> {
+  static constexpr int N = 8;
+  static __device__ __forceinline__ void open(const uint4& u, float* f) {
+    const unsigned w[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { f[2 * i] = __uint_as_float(w[i] << 16); f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+  }
+};
+
+// acc[n] = row . v[n] for NT vectors of shared memory (stride ldv): the `lanes` lanes of a group share the row, each its
+// pieces of 16 bytes; the group's sums are added across it, so that all of its lanes hold them.
+template <typename T, int NT>
+__device__ __forceinline__ void group_dots(const T* row, const float* v, int ldv, int n_cols, int lane, int lanes, bool live,
+                                           float (&acc)[NT]) {
+  constexpr int N = Piece<T>::N;
+#pragma unroll
+  for (int n = 0; n < NT; ++n) acc[n] = 0.f;
+  if (live) {
+#pragma unroll 4
+    for (int c = lane * N; c < n_cols; c += lanes * N) {
+      float w[N];
+      Piece<T>::open(*reinterpret_cast<const uint4*>(row + c), w);
+#pragma unroll
+      for (int n = 0; n < NT; ++n) {
+        const float* x = v + n * ldv + c;
+#pragma unroll
+        for (int i = 0; i < N; i += 4) {
+          const float4 f = *reinterpret_cast<const float4*>(x + i);
+          acc[n] = fmaf(w[i], f.x, acc[n]);
+          acc[n] = fmaf(w[i + 1], f.y, acc[n]);
+          acc[n] = fmaf(w[i + 2], f.z, acc[n]);
+          acc[n] = fmaf(w[i + 3], f.w, acc[n]);
+        }
+      }
+    }
+  }
+  for (int o = lanes >> 1; o > 0; o >>= 1)
+#pragma unroll
+    for (int n = 0; n < NT; ++n) acc[n] += __shfl_xor_sync(0xffffffffu, acc[n], o);
+}
+
+// The sum of v[n] over the block for NT values at once, into every block's `slots` [kStepBlocks][NT] at this block's place.
+template <int NT>
+__device__ __forceinline__ void share_sums(const float (&v)[NT], float* part, float* slots, int rank) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const float s = warp_sum(v[n]);
+    if (lane == 0) part[warp * NT + n] = s;
+  }
+  __syncthreads();
+  if (threadIdx.x < NT * kStepBlocks) {
+    const int n = threadIdx.x % NT, to = threadIdx.x / NT;
+    float s = 0.f;
+    for (int w = 0; w < kStepWarps; ++w) s += part[w * NT + n];
+    store_in_block(slots + rank * NT + n, to, s);
+  }
+}
+
+// delta null: nothing is pending; post_w null: delta joins as it is, else x = resid + delta / rms(delta) * post_w.
+template <typename T, int NT>
+__global__ void __launch_bounds__(kStepThreads)
+token_input_step_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ post_w, float post_eps,
+                        const T* __restrict__ w_gate, const T* __restrict__ w_proj, const float* __restrict__ norm_w,
+                        float eps, const T* __restrict__ table, int ld_table, int first, int V, const int* __restrict__ ids,
+                        const int* __restrict__ sampled, int n_sampled, T* __restrict__ out, int T_, int W, int dim, int dim_p,
+                        int slice, int* status) {
+  extern __shared__ float4 step_smem[];
+  float* xs = reinterpret_cast<float*>(step_smem);      // [NT][slice] the stream, as the product reads it
+  float* act = xs + NT * slice;                         // [NT][dim_p]
+  float* sums = act + NT * dim_p;                       // [kStepBlocks][NT][dim] every block's share of W_g x
+  float* ys = sums + kStepBlocks * NT * dim;            // [NT][slice]
+  float* rs = ys + NT * slice;                          // [NT][slice] the float32 stream
+  __shared__ float part[kStepWarps * NT];
+  __shared__ float sq_pending[kStepBlocks * NT], sq_y[kStepBlocks * NT];
+  __shared__ int token[NT];
+  constexpr int N = Piece<T>::N;
+  pdl_trigger();
+  const int rank = blockIdx.x % kStepBlocks, t0 = blockIdx.x / kStepBlocks * NT;      // the cluster is kStepBlocks neighbours along x
+  const int tid = threadIdx.x;
+  const int n_tok = min(NT, T_ - t0);
+  const int c0 = min(W, rank * slice), c1 = min(W, c0 + slice), nc = c1 - c0;
+  if (t0 == 0) {       // the weights do not depend on what runs before: the first cluster asks for their lines
+    constexpr int line = 128 / (int)sizeof(T);
+    for (int i = tid; i < dim * ((nc + line - 1) / line); i += kStepThreads) {
+      const int per = (nc + line - 1) / line, j = i / per;
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(w_gate + (size_t)j * W + c0 + (i - j * per) * line));
+    }
+    for (int i = tid * line; i < nc * dim_p; i += kStepThreads * line)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(w_proj + (size_t)c0 * dim_p + i));
+  }
+  cluster_meet();                                         // every block of the cluster runs before another writes into it
+  pdl_wait();
+  // ---- the stream, brought up to date
+  float v[NT];
+  if (delta != nullptr && post_w != nullptr) {
+#pragma unroll
+    for (int n = 0; n < NT; ++n) {
+      v[n] = 0.f;
+      if (n < n_tok)
+        for (int i = tid; i < nc; i += kStepThreads) {
+          const float d = to_f32(delta[(size_t)(t0 + n) * W + c0 + i]);
+          v[n] = fmaf(d, d, v[n]);
+        }
+    }
+    share_sums<NT>(v, part, sq_pending, rank);
+  }
+  if (tid < NT) {
+    int id = -1;
+    if (tid < n_tok) {
+      id = token_of(ids, sampled, n_sampled, t0 + tid, V);
+      if (id < 0 && rank == 0) atomicCAS(status, 0, KVB_STATUS_BAD_TOKEN);
+    }
+    token[tid] = id;
+  }
+  cluster_meet();
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    float f = 1.f;
+    if (delta != nullptr && post_w != nullptr) {
+      float s = 0.f;
+      for (int b = 0; b < kStepBlocks; ++b) s += sq_pending[b * NT + n];
+      f = 1.0f / sqrtf(s / (float)W + post_eps);
+    }
+    for (int i = tid; i < slice; i += kStepThreads) {
+      float x = 0.f;
+      if (n < n_tok && i < nc) {
+        const size_t at = (size_t)(t0 + n) * W + c0 + i;
+        x = resid[at];
+        if (delta != nullptr) x += to_f32(delta[at]) * f * (post_w != nullptr ? post_w[c0 + i] : 1.f);
+      }
+      rs[n * slice + i] = x;
+      xs[n * slice + i] = to_f32(from_f32<T>(x));
+    }
+  }
+  __syncthreads();
+  // ---- this block's columns of W_g x, for all of its rows, to every block of the cluster
+  {
+    constexpr int lanes = 8, groups = kStepThreads / lanes;
+    const int lane = tid % lanes, group = tid / lanes;
+    for (int j0 = 0; j0 < dim; j0 += groups) {
+      const int j = j0 + group;
+      float acc[NT];
+      group_dots<T, NT>(w_gate + (size_t)j * W + c0, xs, slice, nc, lane, lanes, j < dim, acc);
+      if (j < dim)
+#pragma unroll
+        for (int n = 0; n < NT; ++n) store_in_block(sums + (rank * NT + n) * dim + j, lane, acc[n]);   // lane l feeds block l
+    }
+  }
+  cluster_meet();
+  for (int i = tid; i < NT * dim_p; i += kStepThreads) {
+    const int n = i / dim_p, j = i - n * dim_p;
+    float a = 0.f;
+    if (j < dim && n < n_tok && token[n] >= 0) {
+      float z = 0.f;
+      for (int b = 0; b < kStepBlocks; ++b) z += sums[(b * NT + n) * dim + j];
+      a = gelu_tanh(to_f32(from_f32<T>(z))) * to_f32(table[(size_t)token[n] * ld_table + first + j]);
+      a = to_f32(from_f32<T>(a));
+    }
+    act[i] = a;
+  }
+  __syncthreads();
+  // ---- this block's rows of y = W_p a
+  {
+    int lanes = 1;
+    while (lanes < 8 && lanes * N < dim_p) lanes <<= 1;
+    const int groups = kStepThreads / lanes, lane = tid % lanes, group = tid / lanes;
+    for (int r0 = 0; r0 < nc; r0 += groups) {
+      const int r = r0 + group;
+      float acc[NT];
+      group_dots<T, NT>(w_proj + (size_t)(c0 + r) * dim_p, act, dim_p, dim_p, lane, lanes, r < nc, acc);
+      if (r < nc && lane == 0)
+#pragma unroll
+        for (int n = 0; n < NT; ++n) ys[n * slice + r] = acc[n];
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    v[n] = 0.f;
+    for (int i = tid; i < nc; i += kStepThreads) v[n] = fmaf(ys[n * slice + i], ys[n * slice + i], v[n]);
+  }
+  share_sums<NT>(v, part, sq_y, rank);
+  cluster_meet();                                         // the last time anything is written into another block
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    if (n >= n_tok) break;
+    float s = 0.f;
+    for (int b = 0; b < kStepBlocks; ++b) s += sq_y[b * NT + n];
+    const float f = 1.0f / sqrtf(s / (float)W + eps);
+    for (int i = tid; i < nc; i += kStepThreads) {
+      const size_t at = (size_t)(t0 + n) * W + c0 + i;
+      const float x = rs[n * slice + i] + ys[n * slice + i] * f * norm_w[c0 + i];
+      resid[at] = x;
+      out[at] = from_f32<T>(x);
+    }
+  }
+}
+
+template <typename T, int NT>
+static int launch_step(float* resid, const void* delta, const float* post_w, float post_eps, const void* w_gate,
+                       const void* w_proj, const float* norm_w, float eps, const void* table, int ld_table, int first, int V,
+                       const int* ids, const int* sampled, int n_sampled, void* out, int T_, int W, int dim, int dim_p,
+                       int slice, size_t smem, int* status, cudaStream_t stream) {
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(token_input_step_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3((T_ + NT - 1) / NT * kStepBlocks);
+  cfg.blockDim = dim3(kStepThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = kStepBlocks;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = kvb_pdl_enabled() ? 2 : 1;
+  cudaError_t e = cudaLaunchKernelEx(&cfg, token_input_step_kernel<T, NT>, resid, (const T*)delta, post_w, post_eps,
+                                     (const T*)w_gate, (const T*)w_proj, norm_w, eps, (const T*)table, ld_table, first, V, ids,
+                                     sampled, n_sampled, (T*)out, T_, W, dim, dim_p, slice, status);
+  return e != cudaSuccess ? (int)e : kvb_launch_result();
+}
+
+static size_t step_smem_bytes(int nt, int slice, int dim, int dim_p) {
+  return sizeof(float) * ((size_t)3 * nt * slice + (size_t)nt * dim_p + (size_t)kStepBlocks * nt * dim);
+}
+
+// Tokens that a cluster takes in a step of T_ tokens: one while the clusters do not fill the GPU, then more.
+static int step_tokens(int T_) { return T_ <= 16 ? 1 : (T_ <= 32 ? 2 : 4); }
+
+// Whether one launch can do the branch for steps of up to T_ tokens: W a multiple of 8, the shared memory at hand.
+KVB_EXPORT int kvb_token_input_step_supported(int T_, int W, int dim, int dim_p) {
+  if (W < 8 || W % 8 != 0 || dim < 1 || dim_p < dim || dim_p % 8 != 0) return 0;
+  const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
+  return step_smem_bytes(step_tokens(T_), slice, dim, dim_p) <= 200 * 1024 ? 1 : 0;
+}
+
+// resid [T, W] float32, in place; delta [T, W] or null, post_w null or the weight of the RMS norm it passes first;
+// w_gate [dim, W], w_proj [W, dim_p] (columns behind dim zero), norm_w [W]; table [V, ld_table], columns first ..
+// first + dim - 1; out [T, W]: the new stream in the activations' type.  Everything dense, rows 16-byte aligned.
+KVB_EXPORT int kvb_token_input_step(float* resid, const void* delta, const float* post_w, float post_eps, const void* w_gate,
+                                    const void* w_proj, const float* norm_w, float eps, const void* table, int ld_table,
+                                    int first, int V, const int* ids, const int* sampled, int n_sampled, void* out, int T_,
+                                    int W, int dim, int dim_p, int dtype, int* status, cudaStream_t stream) {
+  if (T_ <= 0) return 0;
+  if (!kvb_token_input_step_supported(T_, W, dim, dim_p) || first < 0 || first + dim > ld_table) return KVB_ERR_BAD_SIZE;
+  if ((reinterpret_cast<uintptr_t>(w_gate) | reinterpret_cast<uintptr_t>(w_proj)) & 15) return KVB_ERR_ALIGN;
+  const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
+  const int nt = step_tokens(T_);
+  const size_t smem = step_smem_bytes(nt, slice, dim, dim_p);
+#define KVB_STEP(NT)                                                                                                      \
+  KVB_DISPATCH_DTYPE(dtype, T, return (launch_step<T, NT>(resid, delta, post_w, post_eps, w_gate, w_proj, norm_w, eps, table, \
+                                                          ld_table, first, V, ids, sampled, n_sampled, out, T_, W, dim,   \
+                                                          dim_p, slice, smem, status, stream)))
+  if (nt == 1) { KVB_STEP(1); }
+  if (nt == 2) { KVB_STEP(2); }
+  KVB_STEP(4);
+#undef KVB_STEP
+  return KVB_ERR_BAD_DTYPE;
 }

@@ -1534,6 +1534,52 @@ def token_gate(p: torch.Tensor, table: torch.Tensor, first: int, batch, width: i
     return out
 
 
+# Steps of up to this many tokens run a layer's token branch as one launch (0: never).
+TOKEN_STEP_MAX_ROWS = int(os.environ.get('KVB200_TOKEN_STEP_MAX_ROWS', '64'))
+_token_step_ok: Dict[tuple, bool] = {}
+
+
+def token_input_step_wanted(rows: int, width: int, dim: int, dim_padded: int, pending) -> bool:
+    """Whether :func:`token_input_step` takes a step of ``rows`` tokens: few of them, and on the stream nothing pending but a
+    branch output, as it is or in front of an RMS norm without a bias."""
+    if rows > TOKEN_STEP_MAX_ROWS or not (pending is None or isinstance(pending, torch.Tensor)
+                                          or (isinstance(pending, PostNormed) and pending.kind == "rms" and pending.bias is None
+                                              and pending.weight is not None)):
+        return False
+    key = (rows, width, dim, dim_padded)
+    if key not in _token_step_ok:
+        _token_step_ok[key] = bool(lib("token_input").kvb_token_input_step_supported(c_int(rows), c_int(width), c_int(dim),
+                                                                                     c_int(dim_padded)))
+    return _token_step_ok[key]
+
+
+def token_input_step(resid: torch.Tensor, pending, gate: torch.Tensor, proj: torch.Tensor, norm_weight: torch.Tensor, eps: float,
+                     table: torch.Tensor, first: int, batch) -> torch.Tensor:
+    """The whole branch that a layer takes from its tokens, in one launch: ``pending`` joins the float32 stream ``resid`` (as
+    in :func:`add_norm`), then ``y = proj (gelu_tanh(gate x) * table[token, first : first + dim])`` and
+    ``x += y / sqrt(mean(y^2) + eps) * norm_weight``.  ``gate`` [dim, W], ``proj`` [W, dim padded].  ``resid`` is brought up to
+    date in place; its copy in the compute type comes back."""
+    _need_cuda(resid, gate)
+    T, W = resid.shape
+    dim, dim_p = gate.shape[0], proj.shape[1]
+    delta, post_w, post_eps = pending, None, 0.0
+    if isinstance(pending, PostNormed):
+        delta, post_w, post_eps = pending.delta, pending.weight, pending.eps
+    assert resid.dtype == torch.float32 and resid.is_contiguous() and gate.is_contiguous() and proj.is_contiguous()
+    assert gate.dtype == proj.dtype == table.dtype and gate.shape[1] == W and proj.shape[0] == W and table.is_contiguous()
+    assert delta is None or (delta.shape == resid.shape and delta.is_contiguous() and delta.dtype == gate.dtype)
+    out = new((T, W), gate.dtype, resid.device)
+    sampled = batch.sampled
+    rc = lib("token_input").kvb_token_input_step(
+        _p(resid), _p(delta), _p(post_w), c_float(post_eps), _p(gate), _p(proj), _p(norm_weight), c_float(eps), _p(table),
+        c_int(table.shape[1]), c_int(int(first)), c_int(table.shape[0]), _p(batch.token_ids), _p(sampled),
+        c_int(0 if sampled is None else sampled.numel()), _p(out), c_int(T), c_int(W), c_int(dim), c_int(dim_p),
+        c_int(dtype_code(gate.dtype)), _p(batch.status), _stream())
+    _check(rc, "token_input_step")
+    choices["token_input_step"] += 1
+    return out
+
+
 def row_axpy(y: torch.Tensor, x: torch.Tensor, c: torch.Tensor) -> torch.Tensor:
     """``y[t] += c[t] * x[t]`` in place (``c`` float32 [T])."""
     _need_cuda(y, x, c)
@@ -1563,11 +1609,12 @@ def kernel_status(device) -> torch.Tensor:
 
 class Folded:
     """What a product hands on in place of its output once it has added that output into
-    the float32 residual itself: ``xb``, the new residual rows in bfloat16, and ``sumsq``
-    [rows, parts], partial sums of their squares, from which the next norm's 1/rms follows."""
+    the float32 residual itself: ``xb``, the new residual rows in the compute type, and ``sumsq``
+    [rows, parts], partial sums of their squares, from which the next norm's 1/rms follows (None: whoever
+    norms the rows sums them up)."""
     __slots__ = ("xb", "sumsq")
 
-    def __init__(self, xb: torch.Tensor, sumsq: torch.Tensor):
+    def __init__(self, xb: torch.Tensor, sumsq: Optional[torch.Tensor] = None):
         self.xb, self.sumsq = xb, sumsq
 
 

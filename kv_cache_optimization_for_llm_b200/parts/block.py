@@ -128,7 +128,8 @@ class PostNormBlock(Part):
 
     def forward(self, residual, delta, batch, cache):
         dtype = self.mixer.ctx.dtype
-        x = ops.add_norm(residual, delta, "copy", None, 0.0, dtype)
+        # a branch that has joined the stream itself has left the copy as well
+        x = delta.xb if isinstance(delta, ops.Folded) else ops.add_norm(residual, delta, "copy", None, 0.0, dtype)
         if getattr(self.mixer, "hands_over_bias", False):      # the last product's bias rides with the pending output
             pending = self.mixer_post.as_pending(*self.mixer.forward(x, batch, cache, bias_out=True))
         else:
@@ -149,7 +150,8 @@ class PostNormMixerBlock(PostNormBlock):
 @register("block", "postnorm_token_input")
 class PostNormTokenInputBlock(PostNormBlock):
     """The post-norm block with a third branch behind the feed-forward, fed by the tokens themselves:
-    ``h += post1(mixer(h)); h += post2(ff(h)); h += post3(token_input(h))``."""
+    ``h += post1(mixer(h)); h += post2(ff(h)); h += post3(token_input(h))``.  In steps of few tokens the branch may do all of
+    its work, from the addition of the feed-forward's output to that of its own, in one launch (``forward_whole``)."""
 
     part_families = {**PostNormBlock.part_families, "token_input": "token_input", "token_input_post_norm": "norm"}
 
@@ -159,6 +161,9 @@ class PostNormTokenInputBlock(PostNormBlock):
 
     def forward(self, residual, delta, batch, cache):
         residual, pending = super().forward(residual, delta, batch, cache)
+        whole = self.token_input.forward_whole(residual, pending, self.token_input_post, batch)
+        if whole is not None:
+            return residual, whole
         x = ops.add_norm(residual, pending, "copy", None, 0.0, self.mixer.ctx.dtype)
         return residual, self.token_input_post.as_pending(self.token_input.forward(x, batch))
 

@@ -55,7 +55,7 @@ class RMSNorm(Part):
     def forward(self, residual, delta=None, rows=None, lazy=False):
         if isinstance(delta, ops.Folded):
             # the branch before this norm has added its output itself and left the sums of squares
-            if lazy and rows is None and self.weight is None:
+            if lazy and rows is None and self.weight is None and delta.sumsq is not None:
                 return ops.PendingNorm(residual, delta.xb, delta.sumsq, self.eps, self.ctx.dtype)
             delta = None
         if isinstance(delta, ops.PostNormed):

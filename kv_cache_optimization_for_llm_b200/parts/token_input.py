@@ -41,6 +41,16 @@ class GatedTokenRows(Part):
     def activation_widths(self):
         return [self.dim, self.padded, self.proj.shape[0]]
 
+    def forward_whole(self, residual, pending, norm, batch):
+        """The branch in one launch, the additions in front of it and behind it included: ``pending`` joins the stream, the
+        branch reads it, passes the RMS norm ``norm`` and joins it too.  Returns an :class:`ops.Folded`, or None where the step
+        or the sizes want the products' own kernels (:meth:`forward`)."""
+        if norm.kind != "rmsnorm" or not ops.token_input_step_wanted(residual.shape[0], residual.shape[1], self.dim, self.padded,
+                                                                     pending):
+            return None
+        return ops.Folded(ops.token_input_step(residual, pending, self.gate, self.proj, norm.weight, norm.eps, self.table, self.first,
+                                               batch))
+
     def forward(self, x, batch):
         a = ops.token_gate(ops.linear(x, self.gate), self.table, self.first, batch, self.padded)
         return ops.linear(a, self.proj)
