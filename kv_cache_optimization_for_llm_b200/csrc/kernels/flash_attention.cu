@@ -50,9 +50,11 @@ struct TileDesc { int req, t0, n_tok, pad; };
 //   sinks          float32 [query heads] or null: exp(sinks[h]) joins the denominator once, without a value
 //   softcap        > 0: a scaled score s becomes softcap * tanh(s / softcap)
 //   gate, gate_ld  bfloat16 rows [T, >= nq * d] (row stride gate_ld) by whose sigmoid the result is multiplied
+//   head_rows      > 0: a key/value head's rows of all pages lie together, head_rows from one head to the next (rows that
+//                  were made for one step, [nkv, num_pages * page_size, 2 d]), instead of [num_pages, nkv, page_size, 2 d]
 struct MaskExt {
   int kv_row_stride, keep_first, one_more;
-  int chunk; const float* sinks; float softcap; const __nv_bfloat16* gate; int gate_ld;
+  int chunk; const float* sinks; float softcap; const __nv_bfloat16* gate; int gate_ld; int head_rows;
 };
 
 template <int D, int NW, bool EXT>
@@ -895,7 +897,7 @@ paged_flash_attention_ws_kernel(const __grid_constant__ CUtensorMap map_k, const
     // that has no page is requested beyond the end of the map, where TMA delivers zeros.  Keys
     // run two tiles ahead of values: a key stage is free again when the scores of its tile are
     // done, a value stage only when the tile's P V is.
-    const int total_rows = (num_pages * nkv) << page_shift;
+    const int total_rows = EXT && ext.head_rows > 0 ? ext.head_rows * nkv : (num_pages * nkv) << page_shift;
     const int n_box = BNK / box_rows;                 // 1, 2, 4 or 8: a tile never straddles 32 boxes
     auto pages_of = [&](int chunk) -> int {           // this lane's entry of boxes 32 chunk .. 32 chunk + 31 of the walk
       const int vb = chunk * 32 + lane;               // box vb of the walk is box vb % n_box of the walk's tile vb / n_box
@@ -912,6 +914,7 @@ paged_flash_attention_ws_kernel(const __grid_constant__ CUtensorMap map_k, const
         int row = total_rows;                                    // zeros
         if (page >= 0 && page < num_pages) {
           row = (((page * nkv) + hk) << page_shift) + (kj & page_mask);
+          if (EXT && ext.head_rows > 0) row = hk * ext.head_rows + (page << page_shift) + (kj & page_mask);
         } else if (kj < k_hi && (kj + box_rows > k_lo || kj < keep)) {
           atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE);        // keys that a row reads
         }
@@ -1167,7 +1170,7 @@ int launch_ws(const void* q, int q_row_stride, const void* k_pages, const void* 
               cudaStream_t stream, MaskExt ext = MaskExt{DH, 0, 0}) {
   const int page_size = 1 << page_shift;
   const int box_rows = page_size < BNK ? page_size : BNK;
-  const long long rows = (long long)num_pages * nkv * page_size;
+  const long long rows = ext.head_rows > 0 ? (long long)ext.head_rows * nkv : (long long)num_pages * nkv * page_size;
   if (rows >= (1ll << 31)) return KVB_ERR_BAD_SIZE;
   CUtensorMap mk, mv;
   int e = pages_map(&mk, k_pages, rows, box_rows, DH, ext.kv_row_stride);
@@ -1324,16 +1327,19 @@ KVB_EXPORT int kvb_paged_flash_attention_rows(const void* q, int q_row_stride, c
 
 // The tcgen05 form with roles (128-row tiles, pages of at least 8 rows) over the same pool [key | value] for mixers
 // that mask by blocks of positions, count a learned score per head into the denominator, cap their scores or gate
-// their result (see MaskExt): query i sees key j <= i when i / chunk == j / chunk (chunk 0: every key up to i).
+// their result (see MaskExt): query i sees key j <= i when i / chunk == j / chunk (chunk 0: every key up to i), or,
+// without a chunk, when i - j < window (window 0: every key up to i).  head_rows: see MaskExt.
 // sinks float32 [nq] or null; softcap 0 for none; gate bfloat16 [T, >= nq * d], 16-byte aligned, gate_ld a multiple
 // of 8, or null.
 KVB_EXPORT int kvb_paged_flash_attention_rows_masked(const void* q, int q_row_stride, const void* pages,
                                                      const int* block_table, int max_pages, int page_size, int num_pages,
                                                      const int* positions, const void* tiles, int num_tiles, void* out,
-                                                     int nq, int nkv, int d, float scale, int chunk, const float* sinks,
-                                                     float softcap, const void* gate, int gate_ld, int* status,
-                                                     cudaStream_t stream) {
+                                                     int nq, int nkv, int d, float scale, int window, int chunk, const float* sinks,
+                                                     float softcap, const void* gate, int gate_ld, int head_rows,
+                                                     int* status, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
+  if (window < 0 || (window > 0 && chunk > 0) || head_rows < 0 ||
+      (head_rows > 0 && (long long)head_rows < (long long)num_pages * page_size)) return KVB_ERR_BAD_SIZE;
   if (nkv < 1 || nq % nkv || chunk < 0 || softcap < 0.f || !(scale > 0.f)) return KVB_ERR_BAD_SIZE;
   const int G = nq / nkv;
   if (!kvb_flash_attention_supported(d, G, page_size) || nkv > 65535 || page_size < 8) return KVB_ERR_BAD_SIZE;
@@ -1344,11 +1350,11 @@ KVB_EXPORT int kvb_paged_flash_attention_rows_masked(const void* q, int q_row_st
   while ((1 << gp_shift) < G) ++gp_shift;
   if ((128 >> gp_shift) < 1) return KVB_ERR_BAD_SIZE;
   const int page_shift = log2_exact(page_size);
-  const MaskExt ext{2 * d, 0, 0, chunk, sinks, softcap, static_cast<const __nv_bfloat16*>(gate), gate_ld};
+  const MaskExt ext{2 * d, 0, 0, chunk, sinks, softcap, static_cast<const __nv_bfloat16*>(gate), gate_ld, head_rows};
   const void* values = static_cast<const __nv_bfloat16*>(pages) + d;
   if (d == 64)
     return tc5::launch_ws<64, true>(q, q_row_stride, pages, values, block_table, max_pages, page_shift, num_pages,
-                                    positions, tiles, num_tiles, out, nq, nkv, G, gp_shift, scale, 0, status, stream, ext);
+                                    positions, tiles, num_tiles, out, nq, nkv, G, gp_shift, scale, window, status, stream, ext);
   return tc5::launch_ws<128, true>(q, q_row_stride, pages, values, block_table, max_pages, page_shift, num_pages,
-                                   positions, tiles, num_tiles, out, nq, nkv, G, gp_shift, scale, 0, status, stream, ext);
+                                   positions, tiles, num_tiles, out, nq, nkv, G, gp_shift, scale, window, status, stream, ext);
 }

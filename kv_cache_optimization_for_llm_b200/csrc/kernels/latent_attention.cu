@@ -13,6 +13,8 @@
 //                     the gate's sigmoid)
 //   head_rows         for steps whose per-head products the library made: [heads, tokens, N] back to one
 //                     row per token, with the same optional gate
+//   latent_rows       for long runs of tokens, whose keys and values are worth making: the cached rows that the runs see,
+//                     gathered into one matrix that a batched product turns into every head's [key | value] rows
 //   latent_attention  causal softmax attention of all heads over the cached rows, optionally over a sliding
 //                     window (position i sees j with i - j < window), optionally with a sink:
 //                     the denominator also holds exp(sink_h), a key without a value
@@ -224,6 +226,48 @@ KVB_EXPORT int kvb_head_rows(const void* in, void* out, int ld_out, const void* 
   else
     kvb_launch(head_rows_kernel<1>, dim3(blocks), dim3(256), 0, stream, (const B*)in, (B*)out, ld_out, (const B*)gate, ld_gate,
                T_, H, N, total);
+  return kvb_launch_result();
+}
+
+// ---------------------------------------------------------------- the rows that long runs see
+// A block fills one page of `rows_per_page` rows of out [n_pages * rows_per_page, rank]: info [n_pages, 4] int32 holds the
+// request's row in the batch, the position of the page's first row, and the first position that the run sees; rows
+// in front of that or behind the request's last token are zero.  16-byte pieces.
+__global__ void __launch_bounds__(256)
+latent_rows_kernel(const __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table, int max_pages, int page_size,
+                   int num_pages, const int* __restrict__ ctx_len, const int4* __restrict__ info, int rows_per_page,
+                   int vecs, __nv_bfloat16* __restrict__ out, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int4 page_info = info[blockIdx.x];
+  const int req = page_info.x, first = page_info.y, lowest = page_info.z;
+  const int end = ctx_len[req];
+  const int* table = block_table + (size_t)req * max_pages;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int r = warp; r < rows_per_page; r += 8) {
+    const int pos = first + r;
+    const uint4* src = nullptr;
+    if (pos >= lowest && pos < end) {
+      const int lp = pos / page_size;
+      const int page = lp < max_pages ? table[lp] : -1;
+      if (page < 0 || page >= num_pages) { if (lane == 0) atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE); }
+      else src = reinterpret_cast<const uint4*>(pages) + ((size_t)page * page_size + pos % page_size) * vecs;
+    }
+    uint4* dst = reinterpret_cast<uint4*>(out) + ((size_t)blockIdx.x * rows_per_page + r) * vecs;
+    for (int v = lane; v < vecs; v += 32) dst[v] = src != nullptr ? src[v] : make_uint4(0u, 0u, 0u, 0u);
+  }
+}
+
+// bfloat16, rank a multiple of 8, cache rows of rank elements (nothing behind the latent).
+KVB_EXPORT int kvb_latent_rows(const void* pages, const int* block_table, int max_pages, int page_size, int num_pages,
+                               const int* ctx_len, const int* info, int n_pages, int rows_per_page, int rank, void* out,
+                               int* status, cudaStream_t stream) {
+  if (n_pages <= 0) return 0;
+  if (rank < 8 || rank % 8 != 0 || rows_per_page < 1) return KVB_ERR_BAD_SIZE;
+  if ((reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(info) | reinterpret_cast<uintptr_t>(out)) & 15)
+    return KVB_ERR_ALIGN;
+  kvb_launch(latent_rows_kernel, dim3(n_pages), dim3(256), 0, stream, (const __nv_bfloat16*)pages, block_table, max_pages,
+             page_size, num_pages, ctx_len, (const int4*)info, rows_per_page, rank / 8, (__nv_bfloat16*)out, status);
   return kvb_launch_result();
 }
 

@@ -37,6 +37,7 @@ struct RowsArgs {
   const int* positions; const TileDesc* tiles;
   __nv_bfloat16* out;                                // [T, nq * dv]
   int nq, nkv, G, gp_shift, dk, dv;
+  int head_rows;                                     // > 0: pages are [nkv, head_rows, dk + dv] instead (rows made for one step)
   float scale; int window, keep_first, one_more;
   ScoreShape shape;
   int* status;
@@ -128,7 +129,8 @@ window_flash_attention_kernel(RowsArgs p) {
         atomicCAS(p.status, 0, KVB_STATUS_UNMAPPED_PAGE);
         ok = false;
       } else {
-        off = ((((size_t)page * p.nkv + hk) << p.page_shift) + (j & page_mask)) * row_len;
+        off = ((p.head_rows > 0 ? (size_t)hk * p.head_rows + ((size_t)page << p.page_shift)
+                                : ((size_t)page * p.nkv + hk) << p.page_shift) + (j & page_mask)) * row_len;
       }
     }
 #pragma unroll
@@ -448,6 +450,7 @@ int fill_args(RowsArgs& a, const void* q, int q_row_stride, const void* pages, c
   a.nq = nq; a.nkv = nkv; a.G = G; a.dk = dk; a.dv = dv;
   a.gp_shift = 0;
   while ((1 << a.gp_shift) < G) ++a.gp_shift;
+  a.head_rows = 0;
   a.scale = scale; a.window = 0; a.keep_first = 0; a.one_more = 0;
   a.status = status;
   return 0;
@@ -461,15 +464,17 @@ int fill_args(RowsArgs& a, const void* q, int q_row_stride, const void* pages, c
 // all bfloat16, q and pages aligned to 16 bytes, q_row_stride a multiple of 8.  head_scale and slopes are
 // float32 [nq] or null; softcap 0 for none; out_scale multiplies the result.  sinks: float32 [nq] or null; chunk: 0 or
 // the size of the blocks of positions (not together with keep_first); gate: bfloat16 [T, >= nq * dv] with row stride
-// gate_ld, or null.
+// gate_ld, or null.  head_rows > 0: pages are [nkv, head_rows, dk + dv] instead, head_rows >= num_pages * page_size (a
+// head's rows of all pages together: rows that were made for one step).
 KVB_EXPORT int kvb_window_flash_attention_masked(const void* q, int q_row_stride, const void* pages, const int* block_table,
                                                  int max_pages, int page_size, int num_pages, const int* positions,
                                                  const void* tiles, int num_tiles, int wide, void* out, int nq, int nkv,
                                                  int dk, int dv, float scale, int window, int keep_first, int one_more,
                                                  const float* head_scale, const float* slopes, float softcap,
                                                  float out_scale, const float* sinks, int chunk, const void* gate,
-                                                 int gate_ld, int* status, cudaStream_t stream) {
+                                                 int gate_ld, int head_rows, int* status, cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
+  if (head_rows < 0 || (head_rows > 0 && (long long)head_rows < (long long)num_pages * page_size)) return KVB_ERR_BAD_SIZE;
   if (nkv < 1 || nkv > 65535 || nq % nkv || window < 0 || keep_first < 0 || softcap < 0.f) return KVB_ERR_BAD_SIZE;
   if (chunk < 0 || (chunk > 0 && keep_first > 0) || (one_more && sinks != nullptr)) return KVB_ERR_BAD_SIZE;
   RowsArgs a;
@@ -477,6 +482,7 @@ KVB_EXPORT int kvb_window_flash_attention_masked(const void* q, int q_row_stride
                            nkv, dk, dv, scale, status);
   if (rc != 0) return rc;
   a.window = window; a.keep_first = keep_first; a.one_more = one_more;
+  a.head_rows = head_rows;
   a.shape = ScoreShape{head_scale, slopes, softcap, out_scale, sinks, chunk, gate, gate_ld};
   return launch_any<false>(a, num_tiles, wide, stream);
 }
@@ -507,6 +513,6 @@ KVB_EXPORT int kvb_window_flash_attention(const void* q, int q_row_stride, const
                                           int* status, cudaStream_t stream) {
   return kvb_window_flash_attention_masked(q, q_row_stride, pages, block_table, max_pages, page_size, num_pages, positions,
                                            tiles, num_tiles, wide, out, nq, nkv, dk, dv, scale, window, keep_first,
-                                           one_more, head_scale, slopes, softcap, out_scale, nullptr, 0, nullptr, 0,
+                                           one_more, head_scale, slopes, softcap, out_scale, nullptr, 0, nullptr, 0, 0,
                                            status, stream);
 }

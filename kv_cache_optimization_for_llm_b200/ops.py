@@ -635,10 +635,11 @@ def _query_tiles(batch, nt: int) -> torch.Tensor:
 
 def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_head_stride: int, cos, sin, rdims: int,
                      pages: torch.Tensor, block_table, batch, sink: Optional[torch.Tensor], scale: float, heads: int,
-                     rank: int, rot: int, window: int = 0) -> torch.Tensor:
+                     rank: int, rot: int, window: int = 0, singles: bool = False) -> torch.Tensor:
     """Causal attention of every token over its request's cached rows [latent | rotated part],
     all heads sharing the rows; query i sees key j when ``0 <= i - j < window`` (``window`` 0: every key up to i); softmax with a sink per head (``sink`` None: without).  ``q_abs`` [T, heads * rank]: the
-    queries' plain parts moved into the latent's space; ``q`` holds head h's part to be rotated at
+    queries' plain parts moved into the latent's space; with ``singles`` only the step's leading single tokens' rows
+    (``batch.num_single``) are given and answered.  ``q`` holds head h's part to be rotated at
     ``rot_first + h * q_head_stride``.  Returns the attended latents [T, heads * rank]."""
     _need_cuda(q_abs, pages)
     assert q_abs.is_contiguous() and q.stride(1) == 1 and pages.is_contiguous()
@@ -647,8 +648,8 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_hea
     out = new((T, heads * rank), q_abs.dtype, q_abs.device)
     if q_abs.dtype == torch.bfloat16 and LATENT_TC and latent_attention_tc_supported(rank, rot):
         nt = latent_tokens_per_tile(heads)
-        if batch.decode_only:
-            tiles, n_tiles = None, batch.num_reqs           # one tile per request, found in the kernel
+        if batch.decode_only or singles:
+            tiles, n_tiles = None, batch.num_single if singles else batch.num_reqs       # one tile per request, found in the kernel
         else:
             tiles = _query_tiles(batch, nt)
             n_tiles = tiles.shape[0]
@@ -670,6 +671,94 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_hea
     _check(rc, "latent_attention")
     choices["latent_attention"] += 1
     return out
+
+
+class StepRows:
+    """Keys and values that were made for one step's runs of tokens: ``data`` [kv_heads, head_rows, width], a row [key | value]
+    per position that the runs see, in pages of ``PAGE`` positions; ``table`` [requests, columns] int32 finds a request's
+    page of a position as a block table does.  The step's first ``skip`` requests (single tokens beside the runs) have none."""
+    PAGE = 64
+    __slots__ = ("data", "table", "skip")
+
+    def __init__(self, data, table, skip):
+        self.data, self.table, self.skip = data, table, skip
+
+    @property
+    def head_rows(self) -> int:
+        return int(self.data.shape[1])
+
+    def pages(self) -> torch.Tensor:
+        """The rows in the shape in which the attention kernels take pages (which read them by ``head_rows``)."""
+        H, n, width = self.data.shape
+        return self.data.view(n // self.PAGE, H, self.PAGE, width)
+
+
+# Steps whose runs bring at least this many tokens make the keys and values of their latents (0: never), unless the runs
+# see more than LATENT_UP_MAX_KEYS positions per token they bring.
+LATENT_UP_MIN_ROWS = int(os.environ.get('KVB200_LATENT_UP_MIN_ROWS', '256'))
+LATENT_UP_MAX_KEYS = 3
+
+
+def _runs_seen(batch, window: int):
+    """(request row, first position on a page's border, first position seen, end) of every run of a step."""
+    starts, ends = batch.host["req_start"], batch.host["ctx_len"]
+    out = []
+    for r in range(batch.num_single, batch.num_reqs):
+        lowest = max(0, int(starts[r]) - window + 1) if window else 0
+        out.append((r, lowest // StepRows.PAGE * StepRows.PAGE, lowest, int(ends[r])))
+    return out
+
+
+def latent_up_wanted(batch, window: int) -> bool:
+    """Whether a step's runs are long enough for keys and values to be worth making: what the captured graphs replay never
+    is (its launches are sized before the positions are known)."""
+    tokens = batch.num_tokens - batch.num_single
+    if batch.decode_only or not LATENT_UP_MIN_ROWS or tokens < LATENT_UP_MIN_ROWS or _capturing():
+        return False
+    keys = sum(-(-(end - first) // StepRows.PAGE) * StepRows.PAGE for _, first, _, end in _runs_seen(batch, window))
+    return keys <= LATENT_UP_MAX_KEYS * tokens
+
+
+def latent_step_rows(pages: torch.Tensor, block_table, batch, w_kv: torch.Tensor, window: int) -> StepRows:
+    """The keys and values of every position that a step's runs see, made from the cached latents: ``pages`` [num_pages, 1,
+    page_size, rank], ``w_kv`` [heads, key size + value size, rank] (bfloat16).  One gather and one batched product by the
+    library."""
+    _need_cuda(pages, w_kv)
+    H, width, rank = w_kv.shape
+    assert pages.dtype == torch.bfloat16 and pages.is_contiguous() and pages.shape[1] == 1 and pages.shape[3] == rank
+    P = StepRows.PAGE
+    plans = batch.host.setdefault("latent_rows", {})
+    plan = plans.get(window)
+    if plan is None:       # once a step and window: what the gather fills each page with, and the table to find it by
+        import numpy as np
+        runs = _runs_seen(batch, window)
+        counts = [-(-(end - first) // P) for _, first, _, end in runs]
+        n_pages, cols = sum(counts), max(-(-end // P) for *_, end in runs)
+        host = torch.empty(4 * n_pages + batch.num_reqs * cols, dtype=torch.int32, pin_memory=True)
+        h = host.numpy()
+        info, table = h[:4 * n_pages].reshape(n_pages, 4), h[4 * n_pages:].reshape(batch.num_reqs, cols)
+        table.fill(-1)
+        at = 0
+        for (r, first, lowest, _), n in zip(runs, counts):
+            info[at:at + n, 0], info[at:at + n, 2], info[at:at + n, 3] = r, lowest, 0
+            info[at:at + n, 1] = np.arange(first, first + n * P, P)
+            table[r, first // P:first // P + n] = np.arange(at, at + n)
+            at += n
+        dev = host.to(pages.device, non_blocking=True)
+        plan = (dev[:4 * n_pages], dev[4 * n_pages:].view(batch.num_reqs, cols), n_pages, host)     # the pinned source lives as long
+        plans[window] = plan
+    info, table, n_pages, _ = plan
+    c = new((n_pages * P, rank), pages.dtype, pages.device)
+    rc = lib("latent_attention").kvb_latent_rows(_p(pages), _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]),
+                                                 c_int(pages.shape[0]), _p(batch.ctx_len), _p(info), c_int(n_pages), c_int(P),
+                                                 c_int(rank), _p(c), _p(batch.status), _stream())
+    _check(rc, "latent_rows")
+    data = new((H, n_pages * P, width), pages.dtype, pages.device)
+    torch.bmm(c.unsqueeze(0).expand(H, -1, -1), w_kv.transpose(1, 2), out=data)
+    if _marks is not None:
+        _mark("latent_up_library")
+    choices["latent_up_library"] += 1
+    return StepRows(data, table, batch.num_single)
 
 
 # ------------------------------------------------------------------ attention
@@ -834,11 +923,15 @@ def flash_attention_rows_masked_wanted(batch, heads: int, kv_heads: int, dk: int
 
 def flash_attention_rows_masked(q: torch.Tensor, pages: torch.Tensor, block_table, batch, heads: int, kv_heads: int,
                                 d: int, scale: float, chunk: int = 0, sinks: Optional[torch.Tensor] = None,
-                                softcap: float = 0.0, gate=None) -> torch.Tensor:
-    """:func:`window_attention` with a mask by blocks of ``chunk`` positions, ``sinks``, a ``softcap`` and a ``gate`` (as
+                                softcap: float = 0.0, gate=None, window: int = 0, rows=None) -> torch.Tensor:
+    """:func:`window_attention` with a mask by blocks of ``chunk`` positions or a ``window``, ``sinks``, a ``softcap`` and a ``gate`` (as
     there) on the tcgen05 kernel with roles: bfloat16 steps with runs of query tokens, key and value size ``d`` both
-    (64 or 128), 128-row tiles, pages of at least 8 rows.  Queries at ``q[:, : heads * d]``.  Returns [T, heads * d]."""
+    (64 or 128), 128-row tiles, pages of at least 8 rows.  Queries at ``q[:, : heads * d]``.  ``rows`` (:class:`StepRows`):
+    keys and values made for this step instead of ``pages`` and ``block_table``.  Returns [T, heads * d]."""
     _need_cuda(q, pages)
+    head_rows, skip = 0, 0
+    if rows is not None:
+        pages, block_table, head_rows, skip = rows.pages(), rows.table, rows.head_rows, rows.skip
     assert q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16 and pages.is_contiguous() and q.stride(1) == 1
     assert tuple(pages.shape[1:]) == (kv_heads, pages.shape[2], 2 * d)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_contiguous() and sinks.numel() == heads)
@@ -848,13 +941,13 @@ def flash_attention_rows_masked(q: torch.Tensor, pages: torch.Tensor, block_tabl
         gt, gcol = gate
         assert gt.dtype == q.dtype and gt.stride(1) == 1 and gt.shape[0] == T and gt.shape[1] >= gcol + heads * d
         gate_at, gate_ld = _at(gt, gcol), gt.stride(0)
-    tiles = flash_tiles(batch, heads // kv_heads, True)
+    tiles = flash_tiles(batch, heads // kv_heads, True)[skip:]
     out = new((T, heads * d), q.dtype, q.device)
     rc = lib("flash_attention").kvb_paged_flash_attention_rows_masked(
         _p(q), c_int(q.stride(0)), _p(pages), _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]),
         c_int(pages.shape[0]), _p(batch.positions), _p(tiles), c_int(tiles.shape[0]), _p(out), c_int(heads), c_int(kv_heads),
-        c_int(d), c_float(scale), c_int(int(chunk or 0)), _p(sinks), c_float(float(softcap or 0.0)), c_void_p(gate_at),
-        c_int(gate_ld), _p(batch.status), _stream())
+        c_int(d), c_float(scale), c_int(int(window or 0)), c_int(int(chunk or 0)), _p(sinks), c_float(float(softcap or 0.0)),
+        c_void_p(gate_at), c_int(gate_ld), c_int(head_rows), _p(batch.status), _stream())
     _check(rc, "flash_attention_rows")
     choices["flash_attention_rows"] += 1
     choices["flash_attention_rows_masked"] += 1
@@ -958,12 +1051,16 @@ def window_flash_attention(q: torch.Tensor, pages: torch.Tensor, block_table, ba
                            dv: int, scale: float, window: int, keep_first: int, one_more: bool,
                            head_scale: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
                            softcap: float = 0.0, out_scale: float = 1.0, wide: Optional[bool] = None,
-                           sinks: Optional[torch.Tensor] = None, chunk: int = 0, gate=None) -> torch.Tensor:
+                           sinks: Optional[torch.Tensor] = None, chunk: int = 0, gate=None, rows=None) -> torch.Tensor:
     """:func:`window_attention` on tensor cores for bfloat16 steps with runs of query tokens: the same mask (window or
     blocks of ``chunk`` positions), softmax (``sinks`` included), shaping of the scores (float32) and output ``gate``,
     the two products on ``mma.sync`` with the probabilities rounded to bfloat16.
-    Queries at ``q[:, : heads * dk]``; ``pages`` [num_pages, kv_heads, page_size, dk + dv].  Returns [T, heads * dv]."""
+    Queries at ``q[:, : heads * dk]``; ``pages`` [num_pages, kv_heads, page_size, dk + dv].  ``rows`` (:class:`StepRows`): keys
+    and values made for this step instead of ``pages`` and ``block_table``.  Returns [T, heads * dv]."""
     _need_cuda(q, pages)
+    head_rows, skip = 0, 0
+    if rows is not None:
+        pages, block_table, head_rows, skip = rows.pages(), rows.table, rows.head_rows, rows.skip
     assert q.dtype == torch.bfloat16 and pages.dtype == torch.bfloat16 and pages.is_contiguous() and q.stride(1) == 1
     assert tuple(pages.shape[1:]) == (kv_heads, pages.shape[2], dk + dv)
     for v in (head_scale, slopes, sinks):
@@ -980,15 +1077,15 @@ def window_flash_attention(q: torch.Tensor, pages: torch.Tensor, block_table, ba
         wide = WINDOW_FLASH_WIDE
     if wide is None:
         wide = (T // rows_tokens_per_tile(group, True)) * kv_heads >= 2 * sm_count(q.device)
-    tiles = tiles_of_height(batch, rows_tokens_per_tile(group, bool(wide)))
+    tiles = tiles_of_height(batch, rows_tokens_per_tile(group, bool(wide)))[skip:]
     out = new((T, heads * dv), q.dtype, q.device)
     rc = lib("window_flash_attention").kvb_window_flash_attention_masked(
         _p(q), c_int(q.stride(0)), _p(pages), _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]),
         c_int(pages.shape[0]), _p(batch.positions), _p(tiles), c_int(tiles.shape[0]), c_int(1 if wide else 0), _p(out),
         c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv), c_float(scale), c_int(int(window or 0)),
         c_int(int(keep_first or 0)), c_int(1 if one_more else 0), _p(head_scale), _p(slopes), c_float(float(softcap or 0.0)),
-        c_float(float(out_scale)), _p(sinks), c_int(int(chunk or 0)), c_void_p(gate_at), c_int(gate_ld), _p(batch.status),
-        _stream())
+        c_float(float(out_scale)), _p(sinks), c_int(int(chunk or 0)), c_void_p(gate_at), c_int(gate_ld), c_int(head_rows),
+        _p(batch.status), _stream())
     _check(rc, "window_flash_attention")
     choices["window_flash_attention"] += 1
     return out

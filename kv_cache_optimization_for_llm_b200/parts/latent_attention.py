@@ -28,7 +28,10 @@ class LatentAttention(Part):
 
     The key up-projection is applied to the queries instead (q_plain^T W_uk,h c = (W_uk,h^T q_plain)^T c),
     attention runs for all heads over the cached rows, and the value up-projection is applied
-    to the attended latents; the output projection follows.
+    to the attended latents; the output projection follows.  Long runs of tokens in bfloat16 (no rotated part, no gate,
+    sizes that the prompt kernels for [key | value] rows take) go the other way: the keys and values of all positions that
+    the runs see are made once (``ops.latent_step_rows``), and every head attends to rows of its own, which is a multiple
+    fewer operations per query and key (dim + vdim against twice the latent) on a faster kernel.
     params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, window, sink, gate, borrows_latent, eps,
     position (PartSpec)."""
 
@@ -51,7 +54,22 @@ class LatentAttention(Part):
 
     @classmethod
     def kernel_modules(cls, params, dtype):
-        return ("latent_attention",) + (("gemm_f32",) if dtype == torch.float32 else ("gemm_bf16", "gemm_bf16_wide"))
+        if dtype == torch.float32:
+            return ("latent_attention", "gemm_f32")
+        up = ()
+        if cls._up_sizes(params, dtype):
+            up = ("window_flash_attention",) + (("flash_attention",) if cls._one_size(params) else ())
+        return ("latent_attention",) + up + ("gemm_bf16", "gemm_bf16_wide")
+
+    @staticmethod
+    def _up_sizes(params, dtype):
+        """Whether long runs may make their keys and values: what the prompt kernels over such rows take."""
+        return (dtype == torch.bfloat16 and not int(params["rot_dim"]) and not params.get("gate") and int(params["kv_rank"]) % 8 == 0
+                and ops.window_flash_attention_supported(int(params["dim"]), int(params["vdim"]), 1, ops.StepRows.PAGE, dtype))
+
+    @staticmethod
+    def _one_size(params):
+        return int(params["dim"]) == int(params["vdim"]) and int(params["dim"]) in (64, 128)
 
     def __init__(self, params, weights, ctx):
         super().__init__(params, weights, ctx)
@@ -78,6 +96,10 @@ class LatentAttention(Part):
         # per head: U_k^T [rank, dim] (absorbs the queries) and U_v [vdim, rank] (up-projects the attended latents)
         self.uk_t = weights["uk"].view(self.heads, self.dim, self.rank).transpose(1, 2).contiguous()
         self.uv = weights["uv"].view(self.heads, self.vdim, self.rank).contiguous()
+        # and, for long runs, a head's [U_k; U_v] together
+        self.ukv = None
+        if self._up_sizes(params, ctx.dtype):
+            self.ukv = torch.cat([weights["uk"].view(self.heads, self.dim, self.rank), self.uv], dim=1).contiguous()
         pos = params.get("position")
         self.position = None
         if pos is not None and self.rot:
@@ -91,15 +113,42 @@ class LatentAttention(Part):
 
     def activation_widths(self):
         H = self.heads
-        return [self.w_in.shape[0], self.q_rank, H * (self.dim + self.rot), 3 * H * self.rank, 2 * H * self.vdim,
-                self.o.shape[0]]
+        widths = [self.w_in.shape[0], self.q_rank, H * (self.dim + self.rot), 3 * H * self.rank, 2 * H * self.vdim,
+                  self.o.shape[0]]
+        if self.ukv is not None:
+            widths.append(ops.LATENT_UP_MAX_KEYS * (H * (self.dim + self.vdim) + self.rank))
+        return widths
 
     def query_tile_heights(self):
         """Tokens per tile of the tensor-core attention (bfloat16, sizes it takes): the step's batch
         lays the tiles out for it."""
-        if self.ctx.dtype != torch.bfloat16 or not ops.LATENT_TC or not ops.latent_attention_tc_supported(self.rank, self.behind):
-            return []
-        return [ops.latent_tokens_per_tile(self.heads)]
+        heights = []
+        if self.ctx.dtype == torch.bfloat16 and ops.LATENT_TC and ops.latent_attention_tc_supported(self.rank, self.behind):
+            heights.append(ops.latent_tokens_per_tile(self.heads))
+        if self.ukv is not None:
+            heights += [ops.rows_tokens_per_tile(1, False), ops.rows_tokens_per_tile(1, True)]
+            if self._one_size(self.params):
+                heights.append(ops.flash_tokens_per_tile(1, True))
+        return heights
+
+    def _over_made_rows(self, q, table, batch, cache):
+        """The heads' results [T, heads * vdim] of a step with long runs; ``q`` holds the queries from column 0 on.  Single
+        tokens beside the runs attend to the cached rows as in every other step."""
+        rows = ops.latent_step_rows(cache.k, table, batch, self.ukv, self.window or 0)
+        if self._one_size(self.params) and ops.flash_attention_rows_masked_wanted(batch, self.heads, self.heads, self.dim, self.vdim,
+                                                                                  rows.PAGE, self.ctx.dtype, q):
+            a = ops.flash_attention_rows_masked(q, None, None, batch, self.heads, self.heads, self.dim, self.scale, sinks=self.sink,
+                                                window=self.window or 0, rows=rows)
+        else:
+            a = ops.window_flash_attention(q, None, None, batch, self.heads, self.heads, self.dim, self.vdim, self.scale,
+                                           self.window or 0, 0, False, sinks=self.sink, rows=rows)
+        n = batch.num_single
+        if n:
+            q_abs = ops.head_gemm(q[:n], 0, self.dim, self.uk_t)
+            lat = ops.latent_attention(q_abs, q[:n], 0, self.dim, None, None, 0, cache.k, table, batch, self.sink, self.scale,
+                                       self.heads, self.rank, self.behind, self.window or 0, singles=True)
+            a[:n].copy_(ops.head_gemm(lat, 0, self.rank, self.uv))
+        return a
 
     def forward(self, x, batch, cache):
         d = ops.linear(x, self.w_in)
@@ -112,6 +161,8 @@ class LatentAttention(Part):
                                  self.eps, cos, sin, batch, table, cache.k, cache.write and not self.borrows)
         q = ops.linear(cq, self.uq) if self.q_rank else d         # without a latent the queries are the product's first columns
         per_head = self.dim + self.rot
+        if self.ukv is not None and ops.latent_up_wanted(batch, self.window or 0):
+            return ops.linear(self._over_made_rows(q, table, batch, cache), self.o)
         q_abs = ops.head_gemm(q, 0, per_head, self.uk_t)
         lat = ops.latent_attention(q_abs, q, self.dim if self.rot else 0, per_head, cos, sin, rdims, cache.k, table, batch, self.sink,
                                    self.scale, self.heads, self.rank, self.behind, self.window or 0)

@@ -95,7 +95,7 @@ def _run_in_steps(mixer, ctx, x, steps, page=8, state_slots=3, tables=None):
         binding = PagedKVBinding(k=store[0], v=store[1] if pg.planes > 1 else None, group=0, page_size=page, state=state)
     else:
         binding = SlotStateBinding(state=state)
-    builder = BatchBuilder(1024, 8, [64], ctx.device, ctx.status)
+    builder = BatchBuilder(1024, 8, [128], ctx.device, ctx.status)
     at = {r: 0 for r in x}
     outs = {r: [] for r in x}
     for step in steps:

@@ -170,10 +170,11 @@ def test_latent_attention_alone_in_portions_and_beside_another_request(dtype, sh
     assert np.abs(bare - plain(x)).max() > 0.02 * np.abs(plain(x)).max()
 
 
-def _spiked_latents(dtype, window, T, query, key, rank, heads, sink):
+def _spiked_latents(dtype, window, T, query, key, rank, heads, sink, made=None):
     """The kernel alone: cached row j holds the unit vector 1 + j mod (rank - 1), the row at ``key`` also a 5 in channel 0,
     which only the query at ``query`` looks for, so that their score is 30 among zeros.  What every head of the query reads
-    in a prompt (one portion) and decoded alone, and the plain answer."""
+    in a prompt (one portion) and decoded alone, and the plain answer.  ``made``: runs attend to keys and values made for the
+    step (from matrices that hand the latent through), by the tcgen05 kernel ("roles") or with tiles of 64 or 128 rows."""
     from kv_cache_optimization_for_llm_b200 import ops
     from kv_cache_optimization_for_llm_b200.engine.batch import BatchBuilder, StepEntry
     ctx, page = _ctx(dtype), 8
@@ -196,6 +197,17 @@ def _spiked_latents(dtype, window, T, query, key, rank, heads, sink):
         first = max(0, at - window + 1) // page if window else 0
         table[:first] = [-1] * first                    # pages behind the window are gone
         batch = builder.build([StepEntry(0, [0] * n, at, ())], _Manager({0: table}, {0: 0}))
+        if made is not None and n > 1:
+            eye = torch.eye(rank, dtype=DT[dtype], device="cuda")
+            rows = ops.latent_step_rows(pages, batch.block_tables[0], batch, torch.cat([eye, eye])[None].repeat(heads, 1, 1), window or 0)
+            if made == "roles":
+                got = ops.flash_attention_rows_masked(qt[at:at + n], None, None, batch, heads, heads, rank, 1.0, sinks=_f32(sinks),
+                                                      window=window or 0, rows=rows)
+            else:
+                got = ops.window_flash_attention(qt[at:at + n], None, None, batch, heads, heads, rank, rank, 1.0, window or 0, 0, False,
+                                                 sinks=_f32(sinks), rows=rows, wide=made == "wide")
+            outs.append(got[query - at].float().cpu().numpy().reshape(heads, rank))
+            continue
         got = ops.latent_attention(qt[at:at + n].contiguous(), qt, 0, 0, None, None, 0, pages, batch.block_tables[0], batch, _f32(sinks),
                                    1.0, heads, rank, 0, window or 0)
         outs.append(got[query - at].float().cpu().numpy().reshape(heads, rank))
@@ -203,19 +215,53 @@ def _spiked_latents(dtype, window, T, query, key, rank, heads, sink):
     return outs, ref
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("rank,heads", [(40, 3), (48, 5), (128, 16), (512, 2)])
-def test_latents_far_away_at_the_edges_of_a_window_and_against_a_sink(dtype, rank, heads):
+@pytest.mark.parametrize("dtype,rank,heads,made", [(d, r, h, None) for d in ("float32", "bfloat16") for r, h in ((40, 3), (48, 5), (128, 16), (512, 2))]
+                         + [("bfloat16", r, 3, how) for r, how in ((64, "roles"), (128, "roles"), (64, "narrow"), (72, "wide"))])
+def test_latents_far_away_at_the_edges_of_a_window_and_against_a_sink(dtype, rank, heads, made):
     T, query = 250, 245
     for window, keys in ((37, ((209, True), (208, False), (245, True), (216, True), (215, True), (0, False), (224, True), (223, True))),
                          (1, ((245, True), (244, False))), (54, ((192, True), (191, False))), (246, ((0, True), (31, True))),
                          (245, ((0, False), (1, True))), (None, ((0, True), (2, True)))):
         for key, seen in keys:
             for sink in (-2.0, 29.0):
-                outs, ref = _spiked_latents(dtype, window, T, query, key, rank, heads, sink)
+                outs, ref = _spiked_latents(dtype, window, T, query, key, rank, heads, sink, made)
                 assert (ref[0, 0] > 3.0) == seen and (not seen or (ref[0, 0] < 4.0) == (sink > 0))      # the sink takes its share
                 for got in outs:
                     assert np.abs(got - ref).max() < (2e-5 if dtype == "float32" else 3e-2) * max(1.0, np.abs(ref).max()), (window, key, sink)
+
+
+@pytest.mark.parametrize("shape,kernel", [
+    (dict(heads=5, dim=32, vdim=48, kv_rank=40, size=200), "window_flash_attention"),
+    (dict(heads=3, dim=64, vdim=64, kv_rank=104, size=37), "window_flash_attention"),       # too few tiles to fill the GPU
+    (dict(heads=150, dim=64, vdim=64, kv_rank=64, scale=0.1, size=130), "flash_attention_rows_masked"),
+    (dict(heads=75, dim=128, vdim=128, kv_rank=96, scale=0.08, size=None), "flash_attention_rows_masked"),
+])
+def test_long_runs_make_their_keys_and_values(shape, kernel):
+    """bfloat16: a run of 512 tokens from position 0, one of 300 that starts inside a page and a window beside two single
+    tokens and a run of 20, and short portions and single tokens that attend to the cached latents; a run that sees
+    too far back for the tokens it brings does not make them."""
+    from kv_cache_optimization_for_llm_b200 import ops
+    rng = np.random.default_rng(7)
+    ctx, H = _ctx("bfloat16", max_positions=2048), 40
+    m = tiny.latent(**shape)
+    wt, w64 = _lat_weights(rng, H, m)
+    mixer = _make("mixer", "latent_attention", _lat_params(H, m), wt, ctx)
+    xs, refs = {}, {}
+    for r, T in enumerate((840, 40, 30, 60)):
+        x, x64 = _w(rng, (T, H), 1.0)
+        xs[r], refs[r] = x.to(torch.bfloat16).cuda(), S.latent_attention_mixer(x64, S.latent(x64, w64, "", 1e-5), w64, "", m)
+    before = dict(ops.choices)
+    used = lambda name: ops.choices[name] - before.get(name, 0)
+    steps = [[(0, 512)], [(1, 39), (2, 29)], [(3, 40)], [(1, 1), (0, 300), (2, 1), (3, 20)], [(0, 1)], [(0, 2)], [(0, 25)]]
+    got = _run_in_steps(mixer, ctx, xs, steps)
+    for r in xs:
+        n = got[r].shape[0]
+        assert _err(got[r], refs[r][:n], "bfloat16") < TOL["bfloat16"]
+    assert used("latent_up_library") == 2 and used(kernel) >= 2
+    # token by token in front of the second run's end: the same numbers up to rounding
+    short = _run_in_steps(mixer, ctx, {0: xs[0][:560]}, [[(0, 250)], [(0, 250)]] + [[(0, 1)]] * 60)
+    assert used("latent_up_library") == 2
+    assert _err(short[0], got[0][:560].double().numpy(), "bfloat16") < TOL["bfloat16"]
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])

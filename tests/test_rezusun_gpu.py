@@ -297,7 +297,7 @@ def test_latent_attention_alone_in_portions_and_beside_another_request(dtype, sh
     whole = _run_in_steps(mixer, ctx, xs, [[(0, 70)], [(1, 33)]])
     cut = _run_in_steps(mixer, ctx, xs, [[(0, 8), (1, 1)], [(0, 9), (1, 1)], [(0, 2), (1, 30)], [(0, 1), (1, 1)],
                                          [(0, 44)], [(0, 1)], [(0, 1)], [(0, 4)]])
-    on_tensor_cores = dtype == "bfloat16" and mx["kv_rank"] % 32 == 0 and (mx["kv_rank"] + mx["rot_dim"]) % 16 == 0
+    on_tensor_cores = dtype == "bfloat16" and mx["kv_rank"] % 16 == 0 and (mx["kv_rank"] + mx["rot_dim"]) % 16 == 0
     assert (ops.choices["latent_attention_tc"] > before) == on_tensor_cores
     for r in xs:
         assert _rel(whole[r], refs[r]) < TOL[dtype]
