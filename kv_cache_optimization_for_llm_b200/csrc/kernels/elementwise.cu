@@ -3,6 +3,7 @@
 // into cache pages.  Each takes float32 or bfloat16 activations; statistics,
 // rotation and the residual sum are float32 in both.
 #include "common.cuh"
+#include "pack4.cuh"
 
 // ---------------------------------------------------------------- embedding
 // residual[t, :] = table[ids[t], :] * scale, the factor applied in float32   (upstream, without a factor:
@@ -60,26 +61,6 @@ KVB_EXPORT int kvb_embed_gather(const void* table, int dtype, const int* ids, co
 // depends on H and the block size only, never on the batch.
 constexpr int kNormThreads = 256;
 constexpr int kNormVec = 8;   // float4 groups per thread: rows up to 256*8*4 = 8192 wide stay in registers
-
-template <typename T> struct Pack4;
-template <> struct Pack4<float> {
-  static __device__ __forceinline__ float4 load(const float* p) { return *reinterpret_cast<const float4*>(p); }
-  static __device__ __forceinline__ void store(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-};
-template <> struct Pack4<__nv_bfloat16> {
-  static __device__ __forceinline__ float4 load(const __nv_bfloat16* p) {
-    const uint2 u = *reinterpret_cast<const uint2*>(p);
-    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u),
-                       __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xffff0000u));
-  }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, float4 v) {
-    __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    uint2 u;
-    u.x = *reinterpret_cast<unsigned*>(&a);
-    u.y = *reinterpret_cast<unsigned*>(&b);
-    *reinterpret_cast<uint2*>(p) = u;
-  }
-};
 
 __device__ __forceinline__ float block_sum(float v, float* warp_part) {
   v = warp_sum(v);

@@ -390,7 +390,7 @@ KVB_EXPORT int kvb_limited_act(const void* p, int ld_p, const float* gate, int l
   if (T_ <= 0) return 0;
   const int width = E * F + S + pad;
   if (E < 0 || F < 1 || S < 0 || pad < 0 || E * F + S < 1 || ld_p < 2 * (E * F + S)) return KVB_ERR_BAD_SIZE;
-  if (dtype == KVB_BF16 && F % 8 == 0 && S % 8 == 0 && pad % 8 == 0 && ld_p % 8 == 0 &&
+  if (dtype == KVB_BF16 && (E == 0 || F % 8 == 0) && S % 8 == 0 && pad % 8 == 0 && ld_p % 8 == 0 &&
       (reinterpret_cast<uintptr_t>(p) & 15) == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0) {
     const size_t groups = (size_t)T_ * (width / 8);
     const size_t want8 = (groups + 255) / 256;

@@ -21,9 +21,27 @@
 // Scores, softmax weights, sums and angles are float32.  Keys are walked in chunks of 32 by
 // absolute position, so a token's result does not depend on how its request was cut into steps,
 // on the rest of the batch or on where its pages lie.
+#include "cluster.cuh"
 #include "common.cuh"
 
 #include <math_constants.h>
+
+__device__ __forceinline__ void ldsm_x4(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
+  const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm_x4_trans(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
+  const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
+                                               unsigned b0, unsigned b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
+               "{%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
 
 // ---------------------------------------------------------------- prep
 // d_in [T, ld]: the query latent at column 0 (q_rank wide), the key/value latent at column
@@ -80,6 +98,83 @@ latent_prep_kernel(const T* __restrict__ d_in, int ld, int q_rank, int kv_off, i
   for (int i = rdims + threadIdx.x; i < rot; i += blockDim.x) dst[rank + i] = kr[i];
 }
 
+// The same for bfloat16 rows whose segments are multiples of 8 wide: a warp per token, 16-byte accesses, no barrier.
+__device__ __forceinline__ float square_sum8(const uint4& u) {
+  const unsigned w[4] = {u.x, u.y, u.z, u.w};
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float a = __uint_as_float(w[i] << 16), b = __uint_as_float(w[i] & 0xffff0000u);
+    s = fmaf(a, a, s);
+    s = fmaf(b, b, s);
+  }
+  return s;
+}
+__device__ __forceinline__ uint4 scaled8(const uint4& u, float f, const float* weight) {
+  const unsigned w[4] = {u.x, u.y, u.z, u.w};
+  const float4 lo = *reinterpret_cast<const float4*>(weight), hi = *reinterpret_cast<const float4*>(weight + 4);
+  const float c[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+  unsigned r[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(w[i] << 16) * f * c[2 * i],
+                                                   __uint_as_float(w[i] & 0xffff0000u) * f * c[2 * i + 1]);
+    r[i] = *reinterpret_cast<const unsigned*>(&v);
+  }
+  return make_uint4(r[0], r[1], r[2], r[3]);
+}
+
+constexpr int kPrepWarps = 4;
+
+__global__ void __launch_bounds__(kPrepWarps * 32)
+latent_prep_bf16x8_kernel(const __nv_bfloat16* __restrict__ d_in, int ld, int q_rank, int kv_off, int rank, int rot, int rdims,
+                          const float* __restrict__ wq, const float* __restrict__ wkv, float eps,
+                          const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len,
+                          const int* __restrict__ positions, const int* __restrict__ token_req,
+                          const int* __restrict__ block_table, int max_pages, int page_size, int num_pages,
+                          __nv_bfloat16* __restrict__ cq, __nv_bfloat16* __restrict__ pages, int write, int T_, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x * kPrepWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= T_) return;
+  const __nv_bfloat16* row = d_in + (size_t)t * ld;
+  const uint4* q4 = reinterpret_cast<const uint4*>(row);
+  const uint4* k4 = reinterpret_cast<const uint4*>(row + kv_off);
+  const int nq = q_rank >> 3, nk = rank >> 3;
+  const int pos = positions[t], req = token_req[t];
+  float sq = 0.f, sk = 0.f;
+  for (int i = lane; i < nq; i += 32) sq += square_sum8(q4[i]);
+  if (write)
+    for (int i = lane; i < nk; i += 32) sk += square_sum8(k4[i]);
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  const float iq = 1.0f / sqrtf(sq / (float)q_rank + eps), ik = 1.0f / sqrtf(sk / (float)rank + eps);
+  uint4* cq4 = reinterpret_cast<uint4*>(cq + (size_t)t * q_rank);
+  for (int i = lane; i < nq; i += 32) cq4[i] = scaled8(q4[i], iq, wq + 8 * i);
+  if (!write) return;
+  if (pos < 0 || (rdims > 0 && pos >= table_len)) {
+    if (lane == 0) atomicCAS(status, 0, KVB_STATUS_BAD_POSITION);
+    return;
+  }
+  const int lp = pos / page_size;
+  const int page = lp < max_pages ? block_table[(size_t)req * max_pages + lp] : -1;
+  if (page < 0 || page >= num_pages) {
+    if (lane == 0) atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE);
+    return;
+  }
+  __nv_bfloat16* dst = pages + ((size_t)page * page_size + (pos % page_size)) * (rank + rot);
+  for (int i = lane; i < nk; i += 32) reinterpret_cast<uint4*>(dst)[i] = scaled8(k4[i], ik, wkv + 8 * i);
+  const int half = rdims >> 1;
+  const __nv_bfloat16* kr = row + kv_off + rank;
+  for (int i = lane; i < half; i += 32) {
+    const float c = cos_t[(size_t)pos * half + i], s = sin_t[(size_t)pos * half + i];
+    const float u = __bfloat162float(kr[2 * i]), v = __bfloat162float(kr[2 * i + 1]);
+    dst[rank + 2 * i] = __float2bfloat16_rn(u * c - v * s);
+    dst[rank + 2 * i + 1] = __float2bfloat16_rn(v * c + u * s);
+  }
+  for (int i = rdims + lane; i < rot; i += 32) dst[rank + i] = kr[i];
+}
+
 KVB_EXPORT int kvb_latent_prep(const void* d_in, int ld, int q_rank, int kv_off, int rank, int rot, int rdims,
                                const float* wq, const float* wkv, float eps, const float* cos_t, const float* sin_t,
                                int table_len, const int* positions, const int* token_req, const int* block_table,
@@ -87,6 +182,14 @@ KVB_EXPORT int kvb_latent_prep(const void* d_in, int ld, int q_rank, int kv_off,
                                int T_, int dtype, int* status, cudaStream_t stream) {
   if (T_ <= 0) return 0;
   if (q_rank < 0 || rank < 1 || rot < 0 || rdims < 0 || (rdims & 1) || rdims > rot) return KVB_ERR_BAD_SIZE;
+  const uintptr_t at = reinterpret_cast<uintptr_t>(d_in) | reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(pages) |
+                       reinterpret_cast<uintptr_t>(wq) | reinterpret_cast<uintptr_t>(wkv);
+  if (dtype == KVB_BF16 && ((ld | q_rank | kv_off | rank | (rank + rot)) & 7) == 0 && (at & 15) == 0) {
+    kvb_launch(latent_prep_bf16x8_kernel, dim3((T_ + kPrepWarps - 1) / kPrepWarps), dim3(kPrepWarps * 32), 0, stream,
+               (const __nv_bfloat16*)d_in, ld, q_rank, kv_off, rank, rot, rdims, wq, wkv, eps, cos_t, sin_t, table_len, positions,
+               token_req, block_table, max_pages, page_size, num_pages, (__nv_bfloat16*)cq, (__nv_bfloat16*)pages, write, T_, status);
+    return kvb_launch_result();
+  }
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(latent_prep_kernel<T>, dim3(T_), dim3(128), 0, stream, (const T*)d_in, ld,
                                             q_rank, kv_off, rank, rot, rdims, wq, wkv, eps, cos_t, sin_t, table_len,
                                             positions, token_req, block_table, max_pages, page_size, num_pages,
@@ -159,12 +262,91 @@ head_gemm_kernel(const T* __restrict__ in, int ld_in, int hs_in, const T* __rest
   }
 }
 
+// The same product on mma.sync m16n8k16 for bfloat16 steps of few rows, which are bound by bringing the weights: a warp
+// takes 8 rows n of W[h] and up to 16 MT rows m; lane (g, t) loads 16 bytes, the elements k0 + 8 t .. + 7, of row n0 + g of
+// W and of rows g and g + 8 of every tile of the input, and hands elements 0 - 3 to one product and 4 - 7 to the next: the
+// order of the k within a product is free as long as both operands have the same.  K a multiple of 8.
+constexpr int HM_WARPS = 4;
+
+template <int MT>
+__global__ void __launch_bounds__(HM_WARPS * 32)
+head_gemm_mma_kernel(const __nv_bfloat16* __restrict__ in, int ld_in, int hs_in, const __nv_bfloat16* __restrict__ W,
+                     __nv_bfloat16* __restrict__ out, int ld_out, int hs_out, int M, int N, int K,
+                     const __nv_bfloat16* __restrict__ gate, int ld_gate) {
+  pdl_trigger();
+  const int h = blockIdx.z, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int n0 = (blockIdx.x * HM_WARPS + (threadIdx.x >> 5)) * 8, m0 = blockIdx.y * 16 * MT;
+  if (n0 >= N) return;
+  const __nv_bfloat16* w = W + ((size_t)h * N + min(n0 + g, N - 1)) * K + 8 * t;
+  const __nv_bfloat16* a[2 * MT];
+#pragma unroll
+  for (int i = 0; i < 2 * MT; ++i) a[i] = in + (size_t)min(m0 + 8 * i + g, M - 1) * ld_in + (size_t)h * hs_in + 8 * t;
+  float acc[MT][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  // the weights do not depend on what runs before: the first pieces are on their way while the kernel waits
+  constexpr int AHEAD = 4;
+  uint4 b[AHEAD];
+#pragma unroll
+  for (int s = 0; s < AHEAD; ++s)
+    b[s] = 32 * s + 8 * t < K ? *reinterpret_cast<const uint4*>(w + 32 * s) : make_uint4(0u, 0u, 0u, 0u);
+  pdl_wait();
+  for (int k0 = 0; k0 < K; k0 += 32 * AHEAD) {
+    uint4 next[AHEAD];
+#pragma unroll
+    for (int s = 0; s < AHEAD; ++s) {
+      const int k = k0 + 32 * (AHEAD + s);
+      next[s] = k + 8 * t < K ? *reinterpret_cast<const uint4*>(w + k) : make_uint4(0u, 0u, 0u, 0u);
+    }
+#pragma unroll
+    for (int s = 0; s < AHEAD; ++s) {
+      const int k = k0 + 32 * s;
+      if (k >= K) break;
+      const bool in_row = k + 8 * t < K;
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        const uint4 lo = in_row ? *reinterpret_cast<const uint4*>(a[2 * i] + k) : make_uint4(0u, 0u, 0u, 0u);
+        const uint4 hi = in_row ? *reinterpret_cast<const uint4*>(a[2 * i + 1] + k) : make_uint4(0u, 0u, 0u, 0u);
+        mma_bf16_16816(acc[i], lo.x, hi.x, lo.y, hi.y, b[s].x, b[s].y);
+        mma_bf16_16816(acc[i], lo.z, hi.z, lo.w, hi.w, b[s].z, b[s].w);
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < AHEAD; ++s) b[s] = next[s];
+  }
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int m = m0 + 16 * i + g + 8 * (e >> 1), n = n0 + 2 * t + (e & 1);
+      if (m < M && n < N) {
+        float v = acc[i][e];
+        if (gate != nullptr) v *= 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)m * ld_gate + (size_t)h * hs_out + n])));
+        out[(size_t)m * ld_out + (size_t)h * hs_out + n] = __float2bfloat16_rn(v);
+      }
+    }
+}
+
 KVB_EXPORT int kvb_head_gemm(const void* in, int ld_in, int hs_in, const void* W, void* out, int ld_out, int hs_out,
-                             int M, int N, int K, int H, const void* gate, int ld_gate, int dtype, cudaStream_t stream) {
+                             int M, int N, int K, int H, const void* gate, int ld_gate, int tensor_cores, int dtype,
+                             cudaStream_t stream) {
   if (M <= 0 || N <= 0 || H <= 0) return 0;
   if (K <= 0 || H > 65535) return KVB_ERR_BAD_SIZE;
   dim3 grid((N + HG_BN - 1) / HG_BN, (M + HG_BM - 1) / HG_BM, H);
   if (grid.y > 65535) return KVB_ERR_BAD_SIZE;
+  if (tensor_cores && dtype == KVB_BF16 && ((K | ld_in | hs_in) & 7) == 0 &&
+      ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(W)) & 15) == 0) {
+    using B = __nv_bfloat16;
+    const int nb = (N + 8 * HM_WARPS - 1) / (8 * HM_WARPS);
+#define KVB_HEAD_MMA(MT)                                                                                               \
+    kvb_launch(head_gemm_mma_kernel<MT>, dim3(nb, (M + 16 * MT - 1) / (16 * MT), H), dim3(HM_WARPS * 32), 0, stream,   \
+               (const B*)in, ld_in, hs_in, (const B*)W, (B*)out, ld_out, hs_out, M, N, K, (const B*)gate, ld_gate)
+    if (M <= 16) KVB_HEAD_MMA(1);
+    else if (M <= 32) KVB_HEAD_MMA(2);
+    else KVB_HEAD_MMA(4);
+#undef KVB_HEAD_MMA
+    return kvb_launch_result();
+  }
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(head_gemm_kernel<T>, grid, dim3(256), 0, stream, (const T*)in, ld_in, hs_in,
                                             (const T*)W, (T*)out, ld_out, hs_out, M, N, K, (const T*)gate, ld_gate)));
   return kvb_launch_result();
@@ -457,23 +639,6 @@ KVB_EXPORT int kvb_latent_attention(const void* q_abs, int ld_qa, int hs_qa, con
 // depends on its own query and on the chunks only, not on what else shares its tile.
 constexpr int TC_ROWS = 64, TC_KEYS = 32, TC_THREADS = 256, TC_SPAD = 33, TC_PPAD = 40;
 
-__device__ __forceinline__ void ldsm_x4(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
-  const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_trans(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
-  const unsigned addr = (unsigned)__cvta_generic_to_shared(p);
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16_16816(float (&c)[4], unsigned a0, unsigned a1, unsigned a2, unsigned a3,
-                                               unsigned b0, unsigned b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, "
-               "{%0, %1, %2, %3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-
 // NT: tiles of 8 value columns per warp at most (a warp owns half of the value columns): rank <= 16 NT.
 template <int NT>
 __global__ void __launch_bounds__(TC_THREADS, 1)
@@ -760,4 +925,306 @@ KVB_EXPORT int kvb_latent_attention_tc(const void* q_abs, int ld_qa, int hs_qa, 
   if (rank <= 256) { KVB_LATENT_TC(16); }
   KVB_LATENT_TC(32);
 #undef KVB_LATENT_TC
+}
+
+// ---------------------------------------------------------------- single tokens: a request's keys dealt over a cluster
+// A step of single tokens has few rows per request (its heads) and many cached rows: a cluster of S blocks takes one
+// request and up to 16 heads, block s the chunks of 64 keys s, s + S, ... (chunks by absolute position, the first one that
+// the window reaches first).  Per chunk: S = Q K^T by mma.sync (each of the eight warps 16 heads x 8 keys over all of
+// Dc), a softmax step of two heads per warp (running maximum and sum), O += P V (each warp 16 heads x its pairs of
+// 8 value columns).  Rows are requested (cp.async) one chunk ahead.  Then the blocks tell each other their maxima and
+// sums, every block scales its sums and hands each other block the columns that one writes out; the sink joins there.
+constexpr int LD_KEYS = 64, LD_THREADS = 256, LD_SPAD = 68, LD_PPAD = 72;
+
+struct LatentDecodeArgs {
+  const __nv_bfloat16* q_abs; int ld_qa, hs_qa;
+  const __nv_bfloat16* q_raw; int ld_q, hs_q;
+  const float* cos_t; const float* sin_t; int table_len, rdims;
+  const __nv_bfloat16* pages; const int* block_table; int max_pages, page_size, num_pages;
+  const int* positions; const int* q_start;
+  const float* sink; float scale; int window;
+  __nv_bfloat16* out; int ld_out, hs_out, H, rank, rot;
+  int* status;
+};
+
+// NP: pairs of 8 value columns per warp at most: rank <= 128 NP.
+template <int NP>
+__global__ void __launch_bounds__(LD_THREADS, 1)
+latent_decode_kernel(LatentDecodeArgs p) {
+  extern __shared__ uint4 ld_smem4[];
+  const int Dc = p.rank + p.rot, DcP = Dc + 8;
+  __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ld_smem4);              // [16][DcP]
+  __nv_bfloat16* Ks0 = Qs + 16 * DcP;                                           // two buffers of [64][DcP]
+  __nv_bfloat16* Ps = Ks0 + 2 * LD_KEYS * DcP;                                  // [16][LD_PPAD]
+  float* Ss = reinterpret_cast<float*>(Ps + 16 * LD_PPAD);                      // [16][LD_SPAD]
+  float* merged = reinterpret_cast<float*>(Ks0);                                // [S][own pairs][16][16], once the keys are done with
+  __shared__ float m_s[16], l_s[16], corr_s[16];
+  __shared__ float all_m[8 * 16], all_l[8 * 16];                                // of every block of the cluster
+  __shared__ int row_ok[2][LD_KEYS];
+  const int S = gridDim.z, part = blockIdx.z;                                   // the cluster lies along z
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  pdl_trigger();
+  if (S > 1) cluster_meet();                       // every block of the cluster runs before another writes into it
+  pdl_wait();
+  const int req = blockIdx.x, h0 = blockIdx.y * 16, HB = min(16, p.H - h0);
+  const int tr = p.q_start[req], pos = p.positions[tr];
+  const int* table = p.block_table + (size_t)req * p.max_pages;
+  const int lowest = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int first = lowest / LD_KEYS + part, last = pos >= 0 ? pos / LD_KEYS : -1;      // this block's chunks: first, first + S, ...
+  const int half = p.rdims >> 1;
+
+  auto request_chunk = [&](int c, int buf) {
+    __nv_bfloat16* Kb = Ks0 + (size_t)buf * LD_KEYS * DcP;
+    // a warp brings eight rows; its lanes 0 - 7 look their pages up
+    const int key_l = c * LD_KEYS + warp * 8 + (lane & 7);
+    int page_l = -1;
+    if (lane < 8 && key_l >= lowest && key_l <= pos) {
+      const int lp = key_l / p.page_size;
+      page_l = lp < p.max_pages ? table[lp] : -1;
+      if (page_l < 0 || page_l >= p.num_pages) { atomicCAS(p.status, 0, KVB_STATUS_UNMAPPED_PAGE); page_l = -1; }
+    }
+    if (lane < 8) row_ok[buf][warp * 8 + lane] = page_l >= 0;
+    const int vecs = Dc >> 3;
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      const int page = __shfl_sync(0xffffffffu, page_l, r), key = c * LD_KEYS + warp * 8 + r;
+      __nv_bfloat16* dst = Kb + (size_t)(warp * 8 + r) * DcP;
+      if (page >= 0) {
+        const __nv_bfloat16* src = p.pages + ((long long)page * p.page_size + key % p.page_size) * Dc;
+        for (int v = lane; v < vecs; v += 32) {
+          const unsigned d = (unsigned)__cvta_generic_to_shared(dst + 8 * v);
+          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"(d), "l"(src + 8 * v) : "memory");
+        }
+      } else {
+        for (int v = lane; v < vecs; v += 32) reinterpret_cast<uint4*>(dst)[v] = make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (first <= last) request_chunk(first, 0);
+
+  // the heads' queries: absorbed plain part as it is, the rotated part turned here; two rows a warp
+  const bool bad_pos = p.rdims > 0 && (pos < 0 || pos >= p.table_len);
+  if (bad_pos && tid == 0) atomicCAS(p.status, 0, KVB_STATUS_BAD_POSITION);
+#pragma unroll
+  for (int rr = 0; rr < 2; ++rr) {
+    const int r = 2 * warp + rr;
+    __nv_bfloat16* q = Qs + (size_t)r * DcP;
+    if (r >= HB) {
+      for (int i = lane; i < DcP; i += 32) q[i] = __float2bfloat16_rn(0.f);
+    } else {
+      const __nv_bfloat16* qa = p.q_abs + (size_t)tr * p.ld_qa + (size_t)(h0 + r) * p.hs_qa;
+      for (int i = lane; i < p.rank / 8; i += 32) reinterpret_cast<uint4*>(q)[i] = reinterpret_cast<const uint4*>(qa)[i];
+      const __nv_bfloat16* qr = p.q_raw + (size_t)tr * p.ld_q + (size_t)(h0 + r) * p.hs_q;
+      for (int i = lane; i < half; i += 32) {
+        float c = 1.f, sn = 0.f;
+        if (!bad_pos) { c = p.cos_t[(size_t)pos * half + i]; sn = p.sin_t[(size_t)pos * half + i]; }
+        const float u = __bfloat162float(qr[2 * i]), v = __bfloat162float(qr[2 * i + 1]);
+        q[p.rank + 2 * i] = __float2bfloat16_rn(u * c - v * sn);
+        q[p.rank + 2 * i + 1] = __float2bfloat16_rn(v * c + u * sn);
+      }
+      for (int i = p.rdims + lane; i < p.rot; i += 32) q[p.rank + i] = qr[i];
+    }
+    if (lane == 0) { m_s[r] = -CUDART_INF_F; l_s[r] = 0.f; }
+  }
+  const int g = lane >> 2, t4 = lane & 3, n_pairs = p.rank / 16;
+  float acc[NP][2][4];
+#pragma unroll
+  for (int i = 0; i < NP; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][0][e] = acc[i][1][e] = 0.f;
+
+  int it = 0;
+  for (int c = first; c <= last; c += S, ++it) {
+    const __nv_bfloat16* Ks = Ks0 + (size_t)(it & 1) * LD_KEYS * DcP;
+    const int* ok = row_ok[it & 1];
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                               // this chunk has arrived; the chunk before is used up (first round: Qs and the row state are written)
+    if (c + S <= last) request_chunk(c + S, (it + 1) & 1);
+    {
+      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+      const __nv_bfloat16* a_ptr = Qs + (size_t)(lane & 15) * DcP + (lane >> 4) * 8;
+      const __nv_bfloat16* b_row = Ks + (size_t)(warp * 8 + (lane & 7)) * DcP;
+      int ks = 0;
+      for (; ks + 32 <= Dc; ks += 32) {
+        unsigned a0, a1, a2, a3, e0, e1, e2, e3, b0, b1, b2, b3;
+        ldsm_x4(a0, a1, a2, a3, a_ptr + ks);
+        ldsm_x4(e0, e1, e2, e3, a_ptr + ks + 16);
+        ldsm_x4(b0, b1, b2, b3, b_row + ks + (lane >> 3) * 8);
+        mma_bf16_16816(s0, a0, a1, a2, a3, b0, b1);
+        mma_bf16_16816(s1, e0, e1, e2, e3, b2, b3);
+      }
+      if (ks < Dc) {
+        unsigned a0, a1, a2, a3, b0, b1, b2, b3;
+        ldsm_x4(a0, a1, a2, a3, a_ptr + ks);
+        ldsm_x4(b0, b1, b2, b3, b_row + ks + ((lane >> 3) & 1) * 8);
+        mma_bf16_16816(s0, a0, a1, a2, a3, b0, b1);
+      }
+      float* srow = Ss + g * LD_SPAD + warp * 8 + 2 * t4;
+      srow[0] = (s0[0] + s1[0]) * p.scale;
+      srow[1] = (s0[1] + s1[1]) * p.scale;
+      srow[8 * LD_SPAD] = (s0[2] + s1[2]) * p.scale;
+      srow[8 * LD_SPAD + 1] = (s0[3] + s1[3]) * p.scale;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int rr = 0; rr < 2; ++rr) {
+      const int r = 2 * warp + rr;
+      const float a = ok[lane] ? Ss[r * LD_SPAD + lane] : -CUDART_INF_F;
+      const float b = ok[lane + 32] ? Ss[r * LD_SPAD + lane + 32] : -CUDART_INF_F;
+      const float m_old = m_s[r], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
+      const float pa = a == -CUDART_INF_F ? 0.f : expf(a - m_new), pb = b == -CUDART_INF_F ? 0.f : expf(b - m_new);
+      Ps[r * LD_PPAD + lane] = __float2bfloat16_rn(pa);
+      Ps[r * LD_PPAD + lane + 32] = __float2bfloat16_rn(pb);
+      const float sum = warp_sum(pa + pb);
+      if (lane == 0) {
+        const float corr = m_old == m_new ? 1.f : expf(m_old - m_new);
+        m_s[r] = m_new;
+        l_s[r] = l_s[r] * corr + sum;
+        corr_s[r] = corr;
+      }
+    }
+    __syncthreads();
+    const float c_lo = corr_s[g], c_hi = corr_s[g + 8];
+#pragma unroll
+    for (int i = 0; i < NP; ++i)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        acc[i][u][0] *= c_lo; acc[i][u][1] *= c_lo; acc[i][u][2] *= c_hi; acc[i][u][3] *= c_hi;
+      }
+#pragma unroll
+    for (int kk = 0; kk < LD_KEYS; kk += 16) {
+      unsigned a0, a1, a2, a3;
+      ldsm_x4(a0, a1, a2, a3, Ps + (size_t)(lane & 15) * LD_PPAD + (lane >> 4) * 8 + kk);
+      const __nv_bfloat16* b_row = Ks + (size_t)(kk + ((lane >> 3) & 1) * 8 + (lane & 7)) * DcP + (lane >> 4) * 8;
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        const int pair = warp + 8 * i;
+        if (pair < n_pairs) {
+          unsigned b0, b1, b2, b3;
+          ldsm_x4_trans(b0, b1, b2, b3, b_row + pair * 16);
+          mma_bf16_16816(acc[i][0], a0, a1, a2, a3, b0, b1);
+          mma_bf16_16816(acc[i][1], a0, a1, a2, a3, b2, b3);
+        }
+      }
+    }
+  }
+  __syncthreads();
+  // ---- the blocks' maxima and sums
+  if (S > 1) {
+    if (tid < 16 * S) {
+      const int to = tid >> 4, r = tid & 15;
+      store_in_block(all_m + part * 16 + r, to, m_s[r]);
+      store_in_block(all_l + part * 16 + r, to, l_s[r]);
+    }
+    cluster_meet();                                // and every block is done with its keys
+  } else {
+    if (tid < 16) { all_m[tid] = m_s[tid]; all_l[tid] = l_s[tid]; }
+    __syncthreads();
+  }
+  float f[2];                                      // what this block's sums of heads g and g + 8 are multiplied by
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const int r = g + 8 * u;
+    const float sink = p.sink != nullptr && r < HB ? p.sink[h0 + r] : -CUDART_INF_F;
+    float m = sink;
+    for (int s = 0; s < S; ++s) m = fmaxf(m, all_m[s * 16 + r]);
+    float l = 0.f;
+    if (m != -CUDART_INF_F) {
+      l = sink == -CUDART_INF_F ? 0.f : expf(sink - m);
+      for (int s = 0; s < S; ++s)
+        if (all_m[s * 16 + r] != -CUDART_INF_F) l += all_l[s * 16 + r] * expf(all_m[s * 16 + r] - m);
+    }
+    const float own = all_m[part * 16 + r];
+    f[u] = own != -CUDART_INF_F && l > 0.f ? expf(own - m) / l : 0.f;
+  }
+  __nv_bfloat16* out = p.out + (size_t)tr * p.ld_out + (size_t)h0 * p.hs_out;
+  if (S == 1) {
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int pair = warp + 8 * i;
+      if (pair >= n_pairs) continue;
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int hi = 0; hi < 2; ++hi) {
+          const int r = g + 8 * hi;
+          if (r < HB)
+            *reinterpret_cast<__nv_bfloat162*>(out + (size_t)r * p.hs_out + pair * 16 + u * 8 + 2 * t4) =
+                __floats2bfloat162_rn(acc[i][u][2 * hi] * f[hi], acc[i][u][2 * hi + 1] * f[hi]);
+        }
+    }
+    return;
+  }
+  // ---- pair q of the columns is written out by block q mod S: everybody hands it the (scaled) sums
+  const int own_pairs = (n_pairs + S - 1) / S;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int pair = warp + 8 * i;
+    if (pair >= n_pairs) continue;
+    float* to = merged + ((size_t)part * own_pairs + pair / S) * 256 + 2 * t4;
+#pragma unroll
+    for (int u = 0; u < 2; ++u)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        store_in_block(to + (g + 8 * (e >> 1)) * 16 + u * 8 + (e & 1), pair % S, acc[i][u][e] * f[e >> 1]);
+  }
+  cluster_meet();                                  // the last time anything is written into another block
+  for (int i = tid; i < own_pairs * 128; i += LD_THREADS) {
+    const int lp = i >> 7, r = (i >> 3) & 15, col = (i & 7) * 2, pair = lp * S + part;
+    if (pair >= n_pairs || r >= HB) continue;
+    float a = 0.f, b = 0.f;
+    for (int s = 0; s < S; ++s) {
+      const float* v = merged + ((size_t)s * own_pairs + lp) * 256 + r * 16 + col;
+      a += v[0];
+      b += v[1];
+    }
+    *reinterpret_cast<__nv_bfloat162*>(out + (size_t)r * p.hs_out + pair * 16 + col) = __floats2bfloat162_rn(a, b);
+  }
+}
+
+static size_t latent_decode_smem(int Dc) {
+  return (size_t)(16 + 2 * LD_KEYS) * (Dc + 8) * 2 + 16 * LD_PPAD * 2 + 16 * LD_SPAD * 4;
+}
+
+// Whether the form for single tokens takes these sizes: those of the tensor-core form whose chunks fit shared memory.
+KVB_EXPORT int kvb_latent_decode_supported(int rank, int rot) {
+  return kvb_latent_attention_tc_supported(rank, rot) && latent_decode_smem(rank + rot) <= 220 * 1024 ? 1 : 0;
+}
+
+// n_reqs requests, each with one token: row q_start[r] of the queries, the positions and the result.  max_keys: the most keys
+// that one of them may see (what the launch is sized by; any number is right).  The rest as for kvb_latent_attention_tc.
+KVB_EXPORT int kvb_latent_decode(const void* q_abs, int ld_qa, int hs_qa, const void* q_raw, int ld_q, int hs_q,
+                                 const float* cos_t, const float* sin_t, int table_len, int rdims, const void* pages,
+                                 const int* block_table, int max_pages, int page_size, int num_pages, const int* positions,
+                                 const int* q_start, int n_reqs, int max_keys, const float* sink, float scale, int window,
+                                 void* out, int ld_out, int hs_out, int H, int rank, int rot, int* status,
+                                 cudaStream_t stream) {
+  if (n_reqs <= 0) return 0;
+  if (!kvb_latent_decode_supported(rank, rot) || H < 1 || (rdims & 1) || rdims > rot || window < 0 || (H + 15) / 16 > 65535)
+    return KVB_ERR_BAD_SIZE;
+  if (((reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(q_abs)) & 15) || ((ld_qa | hs_qa) & 7) ||
+      (reinterpret_cast<uintptr_t>(out) & 3) || (ld_out & 1) || (hs_out & 1))
+    return KVB_ERR_ALIGN;
+  using B = __nv_bfloat16;
+  const LatentDecodeArgs a{(const B*)q_abs, ld_qa, hs_qa, (const B*)q_raw, ld_q, hs_q, cos_t, sin_t, table_len, rdims,
+                           (const B*)pages, block_table, max_pages, page_size, num_pages, positions, q_start, sink, scale,
+                           window, (B*)out, ld_out, hs_out, H, rank, rot, status};
+  const size_t smem = latent_decode_smem(rank + rot);
+  const int tiles = (H + 15) / 16, chunks = (max_keys + LD_KEYS - 1) / LD_KEYS;
+  int S = 1;                          // blocks per request: as many as find an SM of their own and a chunk to take
+  while (S < 8 && n_reqs * tiles * 2 * S <= kvb_sm_count() && 2 * S <= chunks) S *= 2;
+  const dim3 grid(n_reqs, tiles, S);
+#define KVB_LATENT_DECODE(NP)                                                                                           \
+  do {                                                                                                                  \
+    cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    if (e != cudaSuccess) return (int)e;                                                                                \
+    if (S > 1) e = kvb_launch_cluster(latent_decode_kernel<NP>, grid, dim3(LD_THREADS), dim3(1, 1, S), smem, stream, a); \
+    else e = kvb_launch(latent_decode_kernel<NP>, grid, dim3(LD_THREADS), smem, stream, a);                             \
+    return e != cudaSuccess ? (int)e : kvb_launch_result();                                                             \
+  } while (0)
+  if (rank <= 128) KVB_LATENT_DECODE(1);
+  if (rank <= 256) KVB_LATENT_DECODE(2);
+  KVB_LATENT_DECODE(4);
+#undef KVB_LATENT_DECODE
 }

@@ -4,6 +4,7 @@
 // gated feed-forward with biases.  Statistics, the residual and the activation's
 // arithmetic are float32 whatever the activations' type.
 #include "common.cuh"
+#include "pack4.cuh"
 
 enum NormKind { NORM_NONE = 0, NORM_LAYER = 1, NORM_RMS = 2 };
 
@@ -90,11 +91,106 @@ add_norm_kernel(float* __restrict__ resid, const T* __restrict__ delta, const fl
     o[i] = from_f32<T>((row[i] - mean) * rstd * (pre_w ? pre_w[i] : 1.f));
 }
 
+// The same for rows whose width is a multiple of 4, up to 256 * 4 * G elements: every thread keeps its G groups of four in
+// registers from the loads to the last store.
+template <typename T, int G>
+__global__ void __launch_bounds__(kRowThreads)
+add_norm_vec_kernel(float* __restrict__ resid, const T* __restrict__ delta, const float* __restrict__ delta_bias,
+                    const float* __restrict__ post_w, int post_kind, float post_eps, const float* __restrict__ pre_w, int pre_kind,
+                    float pre_eps, T* __restrict__ out, const int* __restrict__ rows, int H) {
+  __shared__ float part[32];
+  pdl_trigger();
+  pdl_wait();
+  const int b = blockIdx.x, n = H >> 2;
+  const size_t src = (size_t)(rows ? rows[b] : b) * H;
+  float4 v[G];
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const int i = g * kRowThreads + threadIdx.x;
+    v[g] = i < n ? *reinterpret_cast<const float4*>(resid + src + 4 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  // mean and 1 / sqrt(mean square of the deviations + eps) of the row that x holds
+  auto stats = [&](const float4 (&x)[G], int kind, float eps, float& mean, float& rstd) {
+    mean = 0.f;
+    if (kind == NORM_LAYER) {
+      float s = 0.f;
+#pragma unroll
+      for (int g = 0; g < G; ++g) s += (x[g].x + x[g].y) + (x[g].z + x[g].w);       // groups behind the row are zero
+      mean = row_block_sum(s, part) / (float)H;
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      if (g * kRowThreads + threadIdx.x < n) {
+        const float p = x[g].x - mean, q = x[g].y - mean, r = x[g].z - mean, s = x[g].w - mean;
+        ss += (p * p + q * q) + (r * r + s * s);
+      }
+    }
+    rstd = 1.0f / sqrtf(row_block_sum(ss, part) / (float)H + eps);
+  };
+  float mean = 0.f, rstd = 1.f;
+  if (delta != nullptr) {
+    float4 d[G];
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      const int i = g * kRowThreads + threadIdx.x;
+      d[g] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < n) {
+        d[g] = Pack4<T>::load(delta + src + 4 * i);
+        if (delta_bias) {
+          const float4 c = *reinterpret_cast<const float4*>(delta_bias + 4 * i);
+          d[g].x += c.x; d[g].y += c.y; d[g].z += c.z; d[g].w += c.w;
+        }
+      }
+    }
+    if (post_kind != NORM_NONE) stats(d, post_kind, post_eps, mean, rstd);
+#pragma unroll
+    for (int g = 0; g < G; ++g) {
+      const int i = g * kRowThreads + threadIdx.x;
+      if (i < n) {
+        float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (post_w) w = *reinterpret_cast<const float4*>(post_w + 4 * i);
+        v[g].x += (d[g].x - mean) * rstd * w.x; v[g].y += (d[g].y - mean) * rstd * w.y;
+        v[g].z += (d[g].z - mean) * rstd * w.z; v[g].w += (d[g].w - mean) * rstd * w.w;
+        if (!rows) *reinterpret_cast<float4*>(resid + src + 4 * i) = v[g];
+      }
+    }
+  }
+  if (out == nullptr) return;
+  mean = 0.f; rstd = 1.f;
+  if (pre_kind != NORM_NONE) stats(v, pre_kind, pre_eps, mean, rstd);
+  T* o = out + (size_t)b * H;
+#pragma unroll
+  for (int g = 0; g < G; ++g) {
+    const int i = g * kRowThreads + threadIdx.x;
+    if (i < n) {
+      float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (pre_kind != NORM_NONE && pre_w) w = *reinterpret_cast<const float4*>(pre_w + 4 * i);
+      Pack4<T>::store(o + 4 * i, make_float4((v[g].x - mean) * rstd * w.x, (v[g].y - mean) * rstd * w.y,
+                                             (v[g].z - mean) * rstd * w.z, (v[g].w - mean) * rstd * w.w));
+    }
+  }
+}
+
 KVB_EXPORT int kvb_add_norm(float* resid, const void* delta, const float* delta_bias, const float* post_w,
                             int post_kind, float post_eps, const float* pre_w, int pre_kind, float pre_eps,
                             void* out, const int* rows, int n_out_rows, int H, int dtype, cudaStream_t stream) {
   if (n_out_rows <= 0) return 0;
   if (post_kind < 0 || post_kind > 2 || pre_kind < 0 || pre_kind > 2) return KVB_ERR_BAD_SIZE;
+  const uintptr_t at = reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(delta) | reinterpret_cast<uintptr_t>(delta_bias) |
+                       reinterpret_cast<uintptr_t>(post_w) | reinterpret_cast<uintptr_t>(pre_w) | reinterpret_cast<uintptr_t>(out);
+  if (H % 4 == 0 && H <= 4 * kRowThreads * 8 && (at & 15) == 0) {
+#define KVB_ADD_NORM(G)                                                                                                 \
+    KVB_DISPATCH_DTYPE(dtype, T, kvb_launch(add_norm_vec_kernel<T, G>, dim3(n_out_rows), dim3(kRowThreads), 0, stream, resid, \
+                                            (const T*)delta, delta_bias, post_w, post_kind, post_eps, pre_w, pre_kind,  \
+                                            pre_eps, (T*)out, rows, H))
+    if (H <= 4 * kRowThreads) { KVB_ADD_NORM(1); }
+    else if (H <= 4 * kRowThreads * 2) { KVB_ADD_NORM(2); }
+    else if (H <= 4 * kRowThreads * 4) { KVB_ADD_NORM(4); }
+    else { KVB_ADD_NORM(8); }
+#undef KVB_ADD_NORM
+    return kvb_launch_result();
+  }
   const size_t smem = (size_t)H * sizeof(float);
   if (smem > 200 * 1024) return KVB_ERR_BAD_SIZE;
   KVB_DISPATCH_DTYPE(dtype, T, {

@@ -6,6 +6,7 @@
 //     a[t, j] = gelu_tanh(p[t, j]) * table[token, first + j].
 //   * token_input_step_kernel: for steps of few tokens: all of it in one launch, the norm and the addition of the
 //     branch that is still pending in front of it included.
+#include "cluster.cuh"
 #include "common.cuh"
 
 __device__ __forceinline__ float gelu_tanh(float z) {
@@ -61,21 +62,11 @@ KVB_EXPORT int kvb_token_gate(const void* p, int ld_p, const void* table, int ld
 // A cluster of kStepBlocks blocks takes NT tokens.  Block r owns columns [c0, c1) of the stream, for the rows of x, for
 // the columns of W_g and for the rows of W_p alike, so the stream itself never leaves its block; what crosses the
 // cluster (written into every block's shared memory, then one hardware barrier) is three sets of partial sums: the
-// squares of the pending branch output, the products W_g x, and the squares of y.  Both products run on plain FMAs:
-// the weights are read once per cluster, and a step of few tokens is bound by bringing them.  Their lines are requested
-// into L2 before the kernel waits for its predecessor.
+// squares of the pending branch output, the products W_g x, and the squares of y.  A step of few tokens is bound by
+// bringing the weights, which are read once per cluster; their lines are requested into L2 before the kernel waits for
+// its predecessor.  This form, for float32, does both products with plain FMAs.
 // Every sum is taken in an order that depends on the sizes only.
 constexpr int kStepBlocks = 8, kStepThreads = 256, kStepWarps = kStepThreads / 32;
-
-__device__ __forceinline__ void cluster_meet() {
-  asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
-}
-// v into the same place of block `rank`'s shared memory
-__device__ __forceinline__ void store_in_block(float* p, int rank, float v) {
-  unsigned local = (unsigned)__cvta_generic_to_shared(p), remote;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
-  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
-}
 
 template <typename T> struct Piece;      // 16 bytes of a row
 template <> struct Piece<float> {
@@ -283,6 +274,208 @@ token_input_step_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
   }
 }
 
+// ---------------------------------------------------------------- the same in bfloat16 on mma.sync
+// A cluster takes 8 tokens, the upper half of the products' 16 rows staying empty.  A lane (g, t) loads 16 bytes of a row of
+// weights, columns k0 + 8 t .. + 7, and the same columns of token g, and hands elements 0 - 3 to one m16n8k16 product
+// and 4 - 7 to the next: the order of the columns within a product is free as long as both operands have the same.
+// W_g x: warps take (tile of 8 rows, part of the block's columns) in turn; every part's sums go to every block.
+constexpr int kStepTokens = 8;
+
+__device__ __forceinline__ void mma_tokens(float (&c)[4], const uint4& a, const uint4& b) {
+  const unsigned z = 0u;
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a.x), "r"(z), "r"(a.y), "r"(z), "r"(b.x), "r"(b.y));
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a.z), "r"(z), "r"(a.w), "r"(z), "r"(b.z), "r"(b.w));
+}
+__device__ __forceinline__ void store2_in_block(float* p, int rank, float a, float b) {
+  unsigned local = (unsigned)__cvta_generic_to_shared(p), remote;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
+  asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(remote), "f"(a), "f"(b) : "memory");
+}
+
+// row . x over n_cols columns for 8 rows of weights (this lane's: `row`, valid when live) and 8 tokens (`x`: this lane's
+// token's columns in shared memory): c[0], c[1] of lane (g, t) are token g's sums for rows 2 t and 2 t + 1.
+__device__ __forceinline__ void tile_dots(const __nv_bfloat16* row, bool live, const __nv_bfloat16* x, int n_cols, int t, float (&c)[4]) {
+  c[0] = c[1] = c[2] = c[3] = 0.f;
+#pragma unroll 8
+  for (int k = 0; k < n_cols; k += 32) {
+    uint4 a = make_uint4(0u, 0u, 0u, 0u), b = a;
+    if (k + 8 * t < n_cols) {
+      a = *reinterpret_cast<const uint4*>(x + k + 8 * t);
+      if (live) b = *reinterpret_cast<const uint4*>(row + k + 8 * t);
+    }
+    mma_tokens(c, a, b);
+  }
+}
+
+// parts: into how many parts of `part_cols` columns (a multiple of 32) a block's columns are dealt for W_g x; dim_s: dim rounded up to
+// a multiple of 8.
+__global__ void __launch_bounds__(kStepThreads)
+token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __restrict__ delta, const float* __restrict__ post_w,
+                            float post_eps, const __nv_bfloat16* __restrict__ w_gate, const __nv_bfloat16* __restrict__ w_proj,
+                            const float* __restrict__ norm_w, float eps, const __nv_bfloat16* __restrict__ table, int ld_table,
+                            int first, int V, const int* __restrict__ ids, const int* __restrict__ sampled, int n_sampled,
+                            __nv_bfloat16* __restrict__ out, int T_, int W, int dim, int dim_p, int slice, int parts,
+                            int part_cols, int* status) {
+  constexpr int NT = kStepTokens;
+  extern __shared__ uint4 step_mma_smem[];
+  const int xs_ld = slice + 8, act_ld = dim_p + 8, dim_s = (dim + 7) / 8 * 8;
+  __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(step_mma_smem);      // [NT][xs_ld] the stream, as the product reads it
+  __nv_bfloat16* act = xs + NT * xs_ld;                                      // [NT][act_ld]
+  float* rs = reinterpret_cast<float*>(act + NT * act_ld);                   // [NT][slice] the float32 stream
+  float* sums = rs + NT * slice;                                             // [kStepBlocks * parts][NT][dim_s] shares of W_g x
+  float* ys = sums;                                                          // [NT][slice], once those are used up
+  __shared__ float part_sq[kStepWarps * NT];
+  __shared__ float sq_pending[kStepBlocks * NT], sq_y[kStepBlocks * NT];
+  __shared__ int token[NT];
+  pdl_trigger();
+  const int rank = blockIdx.x % kStepBlocks, t0 = blockIdx.x / kStepBlocks * NT;      // the cluster is kStepBlocks neighbours along x
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const int n_tok = min(NT, T_ - t0);
+  const int c0 = min(W, rank * slice), c1 = min(W, c0 + slice), nc = c1 - c0;
+  if (t0 == 0) {       // the weights do not depend on what runs before: the first cluster asks for their lines
+    const int per = (nc + 63) / 64;
+    for (int i = tid; i < dim * per; i += kStepThreads) {
+      const int j = i / per;
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(w_gate + (size_t)j * W + c0 + (i - j * per) * 64));
+    }
+    for (int i = tid * 64; i < nc * dim_p; i += kStepThreads * 64)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(w_proj + (size_t)c0 * dim_p + i));
+  }
+  cluster_meet();                                         // every block of the cluster runs before another writes into it
+  pdl_wait();
+  // ---- the stream, brought up to date; a warp takes a token
+  const bool live_tok = warp < n_tok;
+  const size_t row_at = (size_t)(t0 + (live_tok ? warp : 0)) * W + c0;
+  const bool normed = delta != nullptr && post_w != nullptr;
+  if (normed) {
+    float sq = 0.f;
+    if (live_tok)
+      for (int i = lane * 8; i < nc; i += 256) {
+        float d[8];
+        Piece<__nv_bfloat16>::open(*reinterpret_cast<const uint4*>(delta + row_at + i), d);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) sq = fmaf(d[e], d[e], sq);
+      }
+    sq = warp_sum(sq);
+    if (lane < kStepBlocks) store_in_block(sq_pending + rank * NT + warp, lane, sq);
+  }
+  if (tid < NT) {
+    int id = -1;
+    if (tid < n_tok) {
+      id = token_of(ids, sampled, n_sampled, t0 + tid, V);
+      if (id < 0 && rank == 0) atomicCAS(status, 0, KVB_STATUS_BAD_TOKEN);
+    }
+    token[tid] = id;
+  }
+  if (normed) cluster_meet();
+  else __syncthreads();
+  {
+    float f = 1.f;
+    if (normed) {
+      float s = 0.f;
+#pragma unroll
+      for (int b = 0; b < kStepBlocks; ++b) s += sq_pending[b * NT + warp];
+      f = 1.0f / sqrtf(s / (float)W + post_eps);
+    }
+    for (int i = lane * 8; i < slice; i += 256) {
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+      if (live_tok && i < nc) {
+        const float4 lo = *reinterpret_cast<const float4*>(resid + row_at + i), hi = *reinterpret_cast<const float4*>(resid + row_at + i + 4);
+        x[0] = lo.x; x[1] = lo.y; x[2] = lo.z; x[3] = lo.w; x[4] = hi.x; x[5] = hi.y; x[6] = hi.z; x[7] = hi.w;
+        if (delta != nullptr) {
+          float d[8];
+          Piece<__nv_bfloat16>::open(*reinterpret_cast<const uint4*>(delta + row_at + i), d);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) x[e] += d[e] * f * (normed ? post_w[c0 + i + e] : 1.f);
+        }
+      }
+      *reinterpret_cast<float4*>(rs + warp * slice + i) = make_float4(x[0], x[1], x[2], x[3]);
+      *reinterpret_cast<float4*>(rs + warp * slice + i + 4) = make_float4(x[4], x[5], x[6], x[7]);
+      __nv_bfloat162 h[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) h[e] = __floats2bfloat162_rn(x[2 * e], x[2 * e + 1]);
+      *reinterpret_cast<uint4*>(xs + warp * xs_ld + i) = *reinterpret_cast<const uint4*>(h);
+    }
+  }
+  __syncthreads();
+  // ---- this block's columns of W_g x, for all of its rows, to every block of the cluster
+  const int tiles = dim_s / 8;
+  for (int u = warp; u < tiles * parts; u += kStepWarps) {
+    const int tile = u % tiles, part = u / tiles, k0 = part * part_cols;
+    const int j = tile * 8 + g;
+    float c[4];
+    tile_dots(w_gate + (size_t)j * W + c0 + k0, j < dim, xs + g * xs_ld + k0, max(0, min(part_cols, nc - k0)), t, c);
+    if (g < n_tok) {
+      float* to = sums + ((size_t)(rank * parts + part) * NT + g) * dim_s + tile * 8 + 2 * t;
+#pragma unroll
+      for (int b = 0; b < kStepBlocks; ++b) store2_in_block(to, b, c[0], c[1]);
+    }
+  }
+  cluster_meet();
+  for (int i = tid; i < NT * act_ld; i += kStepThreads) {
+    const int n = i / act_ld, j = i - n * act_ld;
+    float a = 0.f;
+    if (j < dim && n < n_tok && token[n] >= 0) {
+      float z = 0.f;
+      for (int b = 0; b < kStepBlocks * parts; ++b) z += sums[((size_t)b * NT + n) * dim_s + j];
+      a = gelu_tanh(__bfloat162float(__float2bfloat16_rn(z))) * __bfloat162float(table[(size_t)token[n] * ld_table + first + j]);
+    }
+    act[i] = __float2bfloat16_rn(a);
+  }
+  __syncthreads();                                        // the shares are used up: their room is y's from here on
+  // ---- this block's rows of y = W_p a
+  float sq = 0.f;                                         // of token g, over this lane's rows
+  for (int r0 = warp * 8; r0 < nc; r0 += kStepWarps * 8) {
+    float c[4];
+    tile_dots(w_proj + (size_t)(c0 + r0 + g) * dim_p, true, act + g * act_ld, dim_p, t, c);     // nc is a multiple of 8
+    ys[g * slice + r0 + 2 * t] = c[0];
+    ys[g * slice + r0 + 2 * t + 1] = c[1];
+    sq = fmaf(c[0], c[0], fmaf(c[1], c[1], sq));
+  }
+  sq += __shfl_xor_sync(0xffffffffu, sq, 1);
+  sq += __shfl_xor_sync(0xffffffffu, sq, 2);
+  if (t == 0) part_sq[warp * NT + g] = sq;
+  __syncthreads();
+  if (tid < NT * kStepBlocks) {
+    const int n = tid % NT, to = tid / NT;
+    float s = 0.f;
+    for (int w = 0; w < kStepWarps; ++w) s += part_sq[w * NT + n];
+    store_in_block(sq_y + rank * NT + n, to, s);
+  }
+  cluster_meet();                                         // the last time anything is written into another block
+  if (!live_tok) return;
+  float s = 0.f;
+#pragma unroll
+  for (int b = 0; b < kStepBlocks; ++b) s += sq_y[b * NT + warp];
+  const float f = 1.0f / sqrtf(s / (float)W + eps);
+  for (int i = lane * 4; i < nc; i += 128) {
+    const float4 x = *reinterpret_cast<const float4*>(rs + warp * slice + i), y = *reinterpret_cast<const float4*>(ys + warp * slice + i);
+    const float4 w = *reinterpret_cast<const float4*>(norm_w + c0 + i);
+    const float4 v = make_float4(x.x + y.x * f * w.x, x.y + y.y * f * w.y, x.z + y.z * f * w.z, x.w + y.w * f * w.w);
+    *reinterpret_cast<float4*>(resid + row_at + i) = v;
+    __nv_bfloat162 h[2] = {__floats2bfloat162_rn(v.x, v.y), __floats2bfloat162_rn(v.z, v.w)};
+    *reinterpret_cast<uint2*>(out + row_at + i) = *reinterpret_cast<const uint2*>(h);
+  }
+}
+
+// How a block's columns are dealt over warps that would be idle otherwise.
+static void step_parts(int slice, int dim, int* parts, int* part_cols) {
+  const int tiles = (dim + 7) / 8, chunks = (slice + 31) / 32;
+  int n = tiles >= kStepWarps ? 1 : kStepWarps / tiles;
+  if (n > chunks) n = chunks;
+  *part_cols = (chunks + n - 1) / n * 32;
+  *parts = (slice + *part_cols - 1) / *part_cols;
+}
+
+static size_t step_mma_smem_bytes(int slice, int dim, int dim_p) {
+  int parts, cols;
+  step_parts(slice, dim, &parts, &cols);
+  const size_t shares = (size_t)kStepBlocks * parts * kStepTokens * ((dim + 7) / 8 * 8), y = (size_t)kStepTokens * slice;
+  return (size_t)kStepTokens * (slice + 8 + dim_p + 8) * 2 + (size_t)kStepTokens * slice * 4 + (shares > y ? shares : y) * 4;
+}
+
 template <typename T, int NT>
 static int launch_step(float* resid, const void* delta, const float* post_w, float post_eps, const void* w_gate,
                        const void* w_proj, const float* norm_w, float eps, const void* table, int ld_table, int first, int V,
@@ -292,22 +485,10 @@ static int launch_step(float* resid, const void* delta, const float* post_w, flo
     cudaError_t e = cudaFuncSetAttribute(token_input_step_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3((T_ + NT - 1) / NT * kStepBlocks);
-  cfg.blockDim = dim3(kStepThreads);
-  cfg.dynamicSmemBytes = smem;
-  cfg.stream = stream;
-  cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = kStepBlocks;
-  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[1].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = kvb_pdl_enabled() ? 2 : 1;
-  cudaError_t e = cudaLaunchKernelEx(&cfg, token_input_step_kernel<T, NT>, resid, (const T*)delta, post_w, post_eps,
-                                     (const T*)w_gate, (const T*)w_proj, norm_w, eps, (const T*)table, ld_table, first, V, ids,
-                                     sampled, n_sampled, (T*)out, T_, W, dim, dim_p, slice, status);
+  const cudaError_t e = kvb_launch_cluster(
+      token_input_step_kernel<T, NT>, dim3((T_ + NT - 1) / NT * kStepBlocks), dim3(kStepThreads), dim3(kStepBlocks), smem, stream, resid,
+      (const T*)delta, post_w, post_eps, (const T*)w_gate, (const T*)w_proj, norm_w, eps, (const T*)table, ld_table, first, V, ids,
+      sampled, n_sampled, (T*)out, T_, W, dim, dim_p, slice, status);
   return e != cudaSuccess ? (int)e : kvb_launch_result();
 }
 
@@ -319,10 +500,11 @@ static size_t step_smem_bytes(int nt, int slice, int dim, int dim_p) {
 static int step_tokens(int T_) { return T_ <= 16 ? 1 : (T_ <= 32 ? 2 : 4); }
 
 // Whether one launch can do the branch for steps of up to T_ tokens: W a multiple of 8, the shared memory at hand.
-KVB_EXPORT int kvb_token_input_step_supported(int T_, int W, int dim, int dim_p) {
+KVB_EXPORT int kvb_token_input_step_supported(int T_, int W, int dim, int dim_p, int dtype) {
   if (W < 8 || W % 8 != 0 || dim < 1 || dim_p < dim || dim_p % 8 != 0) return 0;
   const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
-  return step_smem_bytes(step_tokens(T_), slice, dim, dim_p) <= 200 * 1024 ? 1 : 0;
+  const size_t smem = dtype == KVB_BF16 ? step_mma_smem_bytes(slice, dim, dim_p) : step_smem_bytes(step_tokens(T_), slice, dim, dim_p);
+  return smem <= 200 * 1024 ? 1 : 0;
 }
 
 // resid [T, W] float32, in place; delta [T, W] or null, post_w null or the weight of the RMS norm it passes first;
@@ -333,18 +515,32 @@ KVB_EXPORT int kvb_token_input_step(float* resid, const void* delta, const float
                                     int first, int V, const int* ids, const int* sampled, int n_sampled, void* out, int T_,
                                     int W, int dim, int dim_p, int dtype, int* status, cudaStream_t stream) {
   if (T_ <= 0) return 0;
-  if (!kvb_token_input_step_supported(T_, W, dim, dim_p) || first < 0 || first + dim > ld_table) return KVB_ERR_BAD_SIZE;
-  if ((reinterpret_cast<uintptr_t>(w_gate) | reinterpret_cast<uintptr_t>(w_proj)) & 15) return KVB_ERR_ALIGN;
+  if (!kvb_token_input_step_supported(T_, W, dim, dim_p, dtype) || first < 0 || first + dim > ld_table) return KVB_ERR_BAD_SIZE;
+  if ((reinterpret_cast<uintptr_t>(resid) | reinterpret_cast<uintptr_t>(delta) | reinterpret_cast<uintptr_t>(w_gate) |
+       reinterpret_cast<uintptr_t>(w_proj) | reinterpret_cast<uintptr_t>(norm_w) | reinterpret_cast<uintptr_t>(out)) & 15)
+    return KVB_ERR_ALIGN;
   const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
+  if (dtype == KVB_BF16) {
+    using B = __nv_bfloat16;
+    const size_t smem = step_mma_smem_bytes(slice, dim, dim_p);
+    int parts, cols;
+    step_parts(slice, dim, &parts, &cols);
+    cudaError_t e = cudaFuncSetAttribute(token_input_step_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    e = kvb_launch_cluster(token_input_step_mma_kernel, dim3((T_ + kStepTokens - 1) / kStepTokens * kStepBlocks), dim3(kStepThreads),
+                           dim3(kStepBlocks), smem, stream, resid, (const B*)delta, post_w, post_eps, (const B*)w_gate,
+                           (const B*)w_proj, norm_w, eps, (const B*)table, ld_table, first, V, ids, sampled, n_sampled, (B*)out, T_,
+                           W, dim, dim_p, slice, parts, cols, status);
+    return e != cudaSuccess ? (int)e : kvb_launch_result();
+  }
+  if (dtype != KVB_F32) return KVB_ERR_BAD_DTYPE;
   const int nt = step_tokens(T_);
   const size_t smem = step_smem_bytes(nt, slice, dim, dim_p);
-#define KVB_STEP(NT)                                                                                                      \
-  KVB_DISPATCH_DTYPE(dtype, T, return (launch_step<T, NT>(resid, delta, post_w, post_eps, w_gate, w_proj, norm_w, eps, table, \
-                                                          ld_table, first, V, ids, sampled, n_sampled, out, T_, W, dim,   \
-                                                          dim_p, slice, smem, status, stream)))
-  if (nt == 1) { KVB_STEP(1); }
-  if (nt == 2) { KVB_STEP(2); }
+#define KVB_STEP(NT)                                                                                                     \
+  return launch_step<float, NT>(resid, delta, post_w, post_eps, w_gate, w_proj, norm_w, eps, table, ld_table, first, V, ids, \
+                                sampled, n_sampled, out, T_, W, dim, dim_p, slice, smem, status, stream)
+  if (nt == 1) KVB_STEP(1);
+  if (nt == 2) KVB_STEP(2);
   KVB_STEP(4);
 #undef KVB_STEP
-  return KVB_ERR_BAD_DTYPE;
 }

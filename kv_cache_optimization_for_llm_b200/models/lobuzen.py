@@ -29,7 +29,7 @@ def _mixer(cfg: LobuzenConfig, i: int, layer: LobuzenLayerConfig) -> PartSpec:
         return PartSpec("latent_attention", {
             "hidden_size": W, "heads": int(m["heads"]), "dim": int(m["dim"]), "rot_dim": 0, "vdim": int(m["vdim"]),
             "q_rank": None, "kv_rank": int(m["kv_rank"]), "scale": float(m["scale"]), "window": layer.window, "sink": True,
-            "borrows_latent": borrows, "eps": cfg.norm_eps,
+            "borrows_latent": borrows, "split_decode": True, "eps": cfg.norm_eps,
         }, names)
     return PartSpec("shaped_window_attention", {
         "hidden_size": W, "heads": int(m["heads"]), "kv_heads": int(m["kv_heads"]), "dim": int(m["dim"]),

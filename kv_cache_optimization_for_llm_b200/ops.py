@@ -555,10 +555,10 @@ def latent_prep(d_in: torch.Tensor, q_rank: int, kv_off: int, rank: int, rot: in
 HEAD_GEMM_LIBRARY_MIN_ROWS = int(os.environ.get('KVB200_HEAD_GEMM_LIBRARY_MIN_ROWS', '128'))
 
 
-def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, gate=None) -> torch.Tensor:
+def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, gate=None, tensor_cores: bool = False) -> torch.Tensor:
     """A product per head: ``out[t, h, :] = w[h] @ x[t, first + h * head_stride : ... + K]`` with
     ``w`` [H, N, K].  ``gate``: (tensor, first column) of rows [T, H * N] by whose sigmoid the result is multiplied.  float32, and bfloat16 steps of fewer than 128 rows: this package's FMA kernel, float32
-    sums in ascending k; bfloat16 with more rows: the library's batched product.  Returns [T, H * N]."""
+    sums in ascending k, or with ``tensor_cores`` (bfloat16, K a multiple of 8, aligned) its mma.sync kernel; bfloat16 with more rows: the library's batched product.  Returns [T, H * N]."""
     _need_cuda(x, w)
     H, N, K = w.shape
     assert w.is_contiguous() and w.dtype == x.dtype and x.stride(1) == 1
@@ -584,13 +584,15 @@ def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, ga
     rc = lib("latent_attention").kvb_head_gemm(c_void_p(_at(x, first)), c_int(x.stride(0)), c_int(head_stride), _p(w),
                                                _p(out), c_int(out.stride(0)), c_int(N), c_int(x.shape[0]), c_int(N),
                                                c_int(K), c_int(H), c_void_p(gate_at), c_int(gate_ld),
-                                               c_int(dtype_code(x.dtype)), _stream())
+                                               c_int(1 if tensor_cores else 0), c_int(dtype_code(x.dtype)), _stream())
     _check(rc, "head_gemm")
     return out
 
 
 LATENT_TC = os.environ.get('KVB200_LATENT_TC', '1') != '0'
+LATENT_DECODE = os.environ.get('KVB200_LATENT_DECODE', '1') != '0'
 _latent_tc_ok: Dict[tuple, bool] = {}
+_latent_decode_ok: Dict[tuple, bool] = {}
 _latent_tpt: Dict[int, int] = {}
 
 
@@ -600,6 +602,14 @@ def latent_attention_tc_supported(rank: int, rot: int) -> bool:
     if key not in _latent_tc_ok:
         _latent_tc_ok[key] = bool(lib("latent_attention").kvb_latent_attention_tc_supported(c_int(key[0]), c_int(key[1])))
     return _latent_tc_ok[key]
+
+
+def latent_decode_supported(rank: int, rot: int) -> bool:
+    """Whether the form for steps of single tokens takes these sizes (bfloat16 only)."""
+    key = (int(rank), int(rot))
+    if key not in _latent_decode_ok:
+        _latent_decode_ok[key] = bool(lib("latent_attention").kvb_latent_decode_supported(c_int(key[0]), c_int(key[1])))
+    return _latent_decode_ok[key]
 
 
 def latent_tokens_per_tile(heads: int) -> int:
@@ -635,17 +645,33 @@ def _query_tiles(batch, nt: int) -> torch.Tensor:
 
 def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, rot_first: int, q_head_stride: int, cos, sin, rdims: int,
                      pages: torch.Tensor, block_table, batch, sink: Optional[torch.Tensor], scale: float, heads: int,
-                     rank: int, rot: int, window: int = 0, singles: bool = False) -> torch.Tensor:
+                     rank: int, rot: int, window: int = 0, singles: bool = False, split: bool = False) -> torch.Tensor:
     """Causal attention of every token over its request's cached rows [latent | rotated part],
     all heads sharing the rows; query i sees key j when ``0 <= i - j < window`` (``window`` 0: every key up to i); softmax with a sink per head (``sink`` None: without).  ``q_abs`` [T, heads * rank]: the
     queries' plain parts moved into the latent's space; with ``singles`` only the step's leading single tokens' rows
-    (``batch.num_single``) are given and answered.  ``q`` holds head h's part to be rotated at
+    (``batch.num_single``) are given and answered.  ``split``: in bfloat16 steps of single tokens a request's keys may be dealt
+    over a cluster of blocks, whose sums are then taken in another order than a long portion's.  ``q`` holds head h's part to be rotated at
     ``rot_first + h * q_head_stride``.  Returns the attended latents [T, heads * rank]."""
     _need_cuda(q_abs, pages)
     assert q_abs.is_contiguous() and q.stride(1) == 1 and pages.is_contiguous()
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == heads)
     T = q_abs.shape[0]
     out = new((T, heads * rank), q_abs.dtype, q_abs.device)
+    if (split and q_abs.dtype == torch.bfloat16 and LATENT_TC and LATENT_DECODE and (batch.decode_only or singles)
+            and latent_decode_supported(rank, rot)):
+        # single tokens: a request's keys are dealt over a cluster of blocks
+        max_keys = decode_launch_context(batch)
+        rc = lib("latent_attention").kvb_latent_decode(
+            _p(q_abs), c_int(q_abs.stride(0)), c_int(rank), c_void_p(_at(q, rot_first)), c_int(q.stride(0)),
+            c_int(q_head_stride), _p(cos), _p(sin), c_int(0 if cos is None else cos.shape[0]), c_int(rdims), _p(pages),
+            _p(block_table), c_int(block_table.shape[1]), c_int(pages.shape[2]), c_int(pages.shape[0]),
+            _p(batch.positions), _p(batch.q_start), c_int(batch.num_single if singles else batch.num_reqs),
+            c_int(min(max_keys, window) if window else max_keys), _p(sink), c_float(scale), c_int(int(window or 0)), _p(out),
+            c_int(out.stride(0)), c_int(rank), c_int(heads), c_int(rank), c_int(rot), _p(batch.status), _stream())
+        _check(rc, "latent_decode")
+        choices["latent_attention_tc"] += 1
+        choices["latent_decode"] += 1
+        return out
     if q_abs.dtype == torch.bfloat16 and LATENT_TC and latent_attention_tc_supported(rank, rot):
         nt = latent_tokens_per_tile(heads)
         if batch.decode_only or singles:
@@ -1636,17 +1662,17 @@ TOKEN_STEP_MAX_ROWS = int(os.environ.get('KVB200_TOKEN_STEP_MAX_ROWS', '64'))
 _token_step_ok: Dict[tuple, bool] = {}
 
 
-def token_input_step_wanted(rows: int, width: int, dim: int, dim_padded: int, pending) -> bool:
+def token_input_step_wanted(rows: int, width: int, dim: int, dim_padded: int, pending, dtype: torch.dtype) -> bool:
     """Whether :func:`token_input_step` takes a step of ``rows`` tokens: few of them, and on the stream nothing pending but a
     branch output, as it is or in front of an RMS norm without a bias."""
     if rows > TOKEN_STEP_MAX_ROWS or not (pending is None or isinstance(pending, torch.Tensor)
                                           or (isinstance(pending, PostNormed) and pending.kind == "rms" and pending.bias is None
                                               and pending.weight is not None)):
         return False
-    key = (rows, width, dim, dim_padded)
+    key = (rows, width, dim, dim_padded, dtype)
     if key not in _token_step_ok:
         _token_step_ok[key] = bool(lib("token_input").kvb_token_input_step_supported(c_int(rows), c_int(width), c_int(dim),
-                                                                                     c_int(dim_padded)))
+                                                                                     c_int(dim_padded), c_int(dtype_code(dtype))))
     return _token_step_ok[key]
 
 

@@ -31,9 +31,11 @@ class LatentAttention(Part):
     to the attended latents; the output projection follows.  Long runs of tokens in bfloat16 (no rotated part, no gate,
     sizes that the prompt kernels for [key | value] rows take) go the other way: the keys and values of all positions that
     the runs see are made once (``ops.latent_step_rows``), and every head attends to rows of its own, which is a multiple
-    fewer operations per query and key (dim + vdim against twice the latent) on a faster kernel.
-    params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, window, sink, gate, borrows_latent, eps,
-    position (PartSpec)."""
+    fewer operations per query and key (dim + vdim against twice the latent) on a faster kernel.  With ``split_decode``
+    bfloat16 steps of single tokens deal a request's keys over several blocks and make the products per head on tensor cores:
+    faster, but a token's result then differs by rounding between a short portion and a step of its own.
+    params: hidden_size, heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, window, sink, gate, borrows_latent, split_decode,
+    eps, position (PartSpec)."""
 
     @classmethod
     def weight_specs(cls, params):
@@ -77,6 +79,7 @@ class LatentAttention(Part):
         self.q_rank, self.rank = int(params["q_rank"] or 0), int(params["kv_rank"])
         self.window = int(params["window"]) if params.get("window") else None
         self.borrows = bool(params.get("borrows_latent"))
+        self.split = bool(params.get("split_decode"))
         self.scale, self.eps = float(params["scale"]), float(params["eps"])
         if self.rank > 512:
             raise ValueError(f"latent_attention: a latent of {self.rank} is refused (up to 512)")
@@ -144,10 +147,10 @@ class LatentAttention(Part):
                                            self.window or 0, 0, False, sinks=self.sink, rows=rows)
         n = batch.num_single
         if n:
-            q_abs = ops.head_gemm(q[:n], 0, self.dim, self.uk_t)
+            q_abs = ops.head_gemm(q[:n], 0, self.dim, self.uk_t, tensor_cores=self.split)
             lat = ops.latent_attention(q_abs, q[:n], 0, self.dim, None, None, 0, cache.k, table, batch, self.sink, self.scale,
-                                       self.heads, self.rank, self.behind, self.window or 0, singles=True)
-            a[:n].copy_(ops.head_gemm(lat, 0, self.rank, self.uv))
+                                       self.heads, self.rank, self.behind, self.window or 0, singles=True, split=self.split)
+            a[:n].copy_(ops.head_gemm(lat, 0, self.rank, self.uv, tensor_cores=self.split))
         return a
 
     def forward(self, x, batch, cache):
@@ -163,8 +166,8 @@ class LatentAttention(Part):
         per_head = self.dim + self.rot
         if self.ukv is not None and ops.latent_up_wanted(batch, self.window or 0):
             return ops.linear(self._over_made_rows(q, table, batch, cache), self.o)
-        q_abs = ops.head_gemm(q, 0, per_head, self.uk_t)
+        q_abs = ops.head_gemm(q, 0, per_head, self.uk_t, tensor_cores=self.split)
         lat = ops.latent_attention(q_abs, q, self.dim if self.rot else 0, per_head, cos, sin, rdims, cache.k, table, batch, self.sink,
-                                   self.scale, self.heads, self.rank, self.behind, self.window or 0)
+                                   self.scale, self.heads, self.rank, self.behind, self.window or 0, split=self.split)
         gate = (d, self.at_g) if self.at_g is not None else None
-        return ops.linear(ops.head_gemm(lat, 0, self.rank, self.uv, gate), self.o)
+        return ops.linear(ops.head_gemm(lat, 0, self.rank, self.uv, gate, tensor_cores=self.split), self.o)

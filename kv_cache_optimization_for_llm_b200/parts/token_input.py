@@ -46,7 +46,7 @@ class GatedTokenRows(Part):
         branch reads it, passes the RMS norm ``norm`` and joins it too.  Returns an :class:`ops.Folded`, or None where the step
         or the sizes want the products' own kernels (:meth:`forward`)."""
         if norm.kind != "rmsnorm" or not ops.token_input_step_wanted(residual.shape[0], residual.shape[1], self.dim, self.padded,
-                                                                     pending):
+                                                                     pending, self.ctx.dtype):
             return None
         return ops.Folded(ops.token_input_step(residual, pending, self.gate, self.proj, norm.weight, norm.eps, self.table, self.first,
                                                batch))

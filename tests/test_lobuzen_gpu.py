@@ -131,7 +131,7 @@ def test_keys_far_away_and_at_the_edges_of_a_window(dtype, kernel):
 
 def _lat_params(H, m, eps=1e-5, borrows=False):
     return {"hidden_size": H, **{k: m[k] for k in ("heads", "dim", "vdim", "kv_rank", "scale")}, "rot_dim": 0, "q_rank": None,
-            "window": S.window_size(m), "sink": True, "borrows_latent": borrows, "eps": eps}
+            "window": S.window_size(m), "sink": True, "borrows_latent": borrows, "split_decode": True, "eps": eps}
 
 
 def _lat_weights(rng, H, m, borrows=False):
@@ -163,7 +163,11 @@ def test_latent_attention_alone_in_portions_and_beside_another_request(dtype, sh
     eps = 0.2
     mixer = _make("mixer", "latent_attention", _lat_params(H, m, eps), wt, ctx)
     plain = lambda x: S.latent_attention_mixer(x, S.latent(x, w64, "", eps), w64, "", m)
-    _mixer_against_plain(mixer, ctx, dtype, rng, H, plain, {"latent_attention_tc": dtype == "bfloat16" and m["kv_rank"] % 16 == 0})
+    from kv_cache_optimization_for_llm_b200 import ops
+    on_tensor_cores = dtype == "bfloat16" and m["kv_rank"] % 16 == 0
+    before = ops.choices["latent_decode"]
+    _mixer_against_plain(mixer, ctx, dtype, rng, H, plain, {"latent_attention_tc": on_tensor_cores})
+    assert (ops.choices["latent_decode"] > before) == on_tensor_cores
     # the sinks show: without them the plain answer is another one
     x = rng.normal(size=(40, H))
     bare = S.latent_attention_mixer(x, S.latent(x, w64, "", eps), dict(w64, sink=w64["sink"] - 1e9), "", m)
@@ -209,7 +213,7 @@ def _spiked_latents(dtype, window, T, query, key, rank, heads, sink, made=None):
             outs.append(got[query - at].float().cpu().numpy().reshape(heads, rank))
             continue
         got = ops.latent_attention(qt[at:at + n].contiguous(), qt, 0, 0, None, None, 0, pages, batch.block_tables[0], batch, _f32(sinks),
-                                   1.0, heads, rank, 0, window or 0)
+                                   1.0, heads, rank, 0, window or 0, split=True)
         outs.append(got[query - at].float().cpu().numpy().reshape(heads, rank))
     assert int(ctx.status.item()) == 0
     return outs, ref
@@ -228,6 +232,58 @@ def test_latents_far_away_at_the_edges_of_a_window_and_against_a_sink(dtype, ran
                 assert (ref[0, 0] > 3.0) == seen and (not seen or (ref[0, 0] < 4.0) == (sink > 0))      # the sink takes its share
                 for got in outs:
                     assert np.abs(got - ref).max() < (2e-5 if dtype == "float32" else 3e-2) * max(1.0, np.abs(ref).max()), (window, key, sink)
+
+
+@pytest.mark.parametrize("T,H,N,K", [(8, 16, 512, 128), (64, 5, 24, 40), (1, 3, 7, 8), (33, 2, 100, 72), (127, 4, 16, 96), (20, 3, 9, 10)])
+def test_per_head_products_of_few_rows_on_tensor_cores(T, H, N, K):
+    from kv_cache_optimization_for_llm_b200 import ops
+    rng = np.random.default_rng(6)
+    (x, x64), (w, w64), (g, g64) = _w(rng, (T, H * K + 8), 1.0), _w(rng, (H, N, K), 0.3), _w(rng, (T, 16 + H * N), 1.0)
+    ref = np.einsum("hnk,thk->thn", w64, x64[:, 8:].reshape(T, H, K)).reshape(T, H * N)
+    xc, wc, gc = (t.to(torch.bfloat16).cuda() for t in (x, w, g))
+    assert _err(ops.head_gemm(xc, 8, K, wc, tensor_cores=True), ref, "bfloat16") < 6e-3
+    assert _err(ops.head_gemm(xc, 8, K, wc, (gc, 16), tensor_cores=True), ref / (1.0 + np.exp(-g64[:, 16:])), "bfloat16") < 6e-3
+
+
+@pytest.mark.parametrize("R,H,rank,window,ctx_len", [(1, 16, 512, 700, 1000), (3, 5, 48, None, 900), (40, 20, 64, 100, 300), (8, 16, 512, None, 129),
+                                                     (150, 3, 16, 37, 90), (2, 33, 80, 1024, 1500)])
+def test_single_tokens_deal_their_keys_over_a_cluster(R, H, rank, window, ctx_len):
+    """Requests of unequal length whose last tokens attend in one step, against the plain answer: from one block a request to
+    eight, some of which find no keys; pages behind the windows are gone."""
+    from kv_cache_optimization_for_llm_b200 import ops
+    from kv_cache_optimization_for_llm_b200.engine.batch import BatchBuilder, StepEntry
+    rng = np.random.default_rng(R)
+    ctx, page = _ctx("bfloat16"), 16
+    lens = [ctx_len] + [int(n) for n in rng.integers(1, ctx_len, R - 1)]
+    each = -(-ctx_len // page)
+    order = rng.permutation(R * each)
+    pages = torch.full((R * each + 1, 1, page, rank), 100.0, dtype=torch.bfloat16, device="cuda")
+    c64, tables = [], {}
+    for r, n in enumerate(lens):
+        c, c_ = _w(rng, (n, rank), 1.0)
+        c64.append(c_)
+        table = order[r * each:(r + 1) * each].tolist()
+        padded = torch.full((each * page, rank), 100.0, dtype=torch.bfloat16)
+        padded[:n] = c
+        pages[table, 0] = padded.view(each, page, rank).cuda()
+        first = max(0, n - 1 - window + 1) // page if window else 0
+        tables[r] = [-1] * first + table[first:]
+    q, q64 = _w(rng, (R, H * rank), 3.0 * rank ** -0.5)
+    sinks = rng.normal(size=H) + 2.0
+    builder = BatchBuilder(256, 160, [each], ctx.device, ctx.status)
+    batch = builder.build([StepEntry(r, [0], n - 1, ()) for r, n in enumerate(lens)], _Manager(tables, {r: 0 for r in range(R)}))
+    before = ops.choices["latent_decode"]
+    qc = q.cuda()
+    got = ops.latent_attention(qc, qc, 0, 0, None, None, 0, pages, batch.block_tables[0], batch, _f32(sinks), 0.7, H, rank, 0, window or 0,
+                               split=True)
+    assert ops.choices["latent_decode"] == before + 1 and int(ctx.status.item()) == 0
+    ref = np.zeros((R, H, rank))
+    for r, n in enumerate(lens):
+        low = max(0, n - window) if window else 0
+        s = q64[r].reshape(H, rank) @ c64[r][low:].T * 0.7
+        for h in range(H):
+            ref[r, h] = S.softmax_rows(s[h:h + 1], np.ones((1, n - low), bool), sinks[h])[0] @ c64[r][low:]
+    assert _err(got, ref.reshape(R, -1), "bfloat16") < 1e-2
 
 
 @pytest.mark.parametrize("shape,kernel", [
