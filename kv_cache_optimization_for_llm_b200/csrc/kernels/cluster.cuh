@@ -15,6 +15,13 @@ __device__ __forceinline__ void store_in_block(float* p, int rank, float v) {
   asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(remote), "f"(v) : "memory");
 }
 
+// The same for two neighbours (8-byte aligned).
+__device__ __forceinline__ void store2_in_block(float* p, int rank, float a, float b) {
+  unsigned local = (unsigned)__cvta_generic_to_shared(p), remote;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
+  asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(remote), "f"(a), "f"(b) : "memory");
+}
+
 // kvb_launch in clusters of `cx` x `cy` x `cz` blocks.
 template <typename... KArgs, typename... Args>
 static inline cudaError_t kvb_launch_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 block, dim3 cluster, size_t smem,

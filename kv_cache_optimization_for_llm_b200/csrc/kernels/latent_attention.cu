@@ -930,24 +930,37 @@ KVB_EXPORT int kvb_latent_attention_tc(const void* q_abs, int ld_qa, int hs_qa, 
 // ---------------------------------------------------------------- single tokens: a request's keys dealt over a cluster
 // A step of single tokens has few rows per request (its heads) and many cached rows: a cluster of S blocks takes one
 // request and up to 16 heads, block s the chunks of 64 keys s, s + S, ... (chunks by absolute position, the first one that
-// the window reaches first).  Per chunk: S = Q K^T by mma.sync (each of the eight warps 16 heads x 8 keys over all of
-// Dc), a softmax step of two heads per warp (running maximum and sum), O += P V (each warp 16 heads x its pairs of
-// 8 value columns).  Rows are requested (cp.async) one chunk ahead.  Then the blocks tell each other their maxima and
-// sums, every block scales its sums and hands each other block the columns that one writes out; the sink joins there.
-constexpr int LD_KEYS = 64, LD_THREADS = 256, LD_SPAD = 68, LD_PPAD = 72;
+// the window reaches first).  Per chunk: S = Q K^T by mma.sync (each of the sixteen warps 16 heads x 8 keys over half of
+// Dc), a softmax step of one head per warp (running maximum and sum), O += P V (each warp 16 heads x its pairs of
+// 8 value columns).  A row is one bulk copy (cp.async.bulk) that counts its bytes on the buffer's barrier, requested one
+// chunk ahead.  Then the blocks tell each other their maxima and sums, every block scales its sums and hands each other
+// block the columns that one writes out; the sink joins there.
+constexpr int LD_KEYS = 64, LD_WARPS = 16, LD_THREADS = LD_WARPS * 32, LD_SPAD = 68, LD_PPAD = 72;
+constexpr unsigned LD_SPINS = 1u << 20;      // polls of a barrier before a block gives up
+
+__device__ __forceinline__ bool ld_wait(unsigned long long* bar, unsigned parity) {
+  const unsigned addr = (unsigned)__cvta_generic_to_shared(bar);
+  for (unsigned i = 0; i < LD_SPINS; ++i) {
+    unsigned ok;
+    asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.b32 %0, 1, 0, p;\n\t}"
+                 : "=r"(ok) : "r"(addr), "r"(parity) : "memory");
+    if (ok) return true;
+  }
+  return false;
+}
 
 struct LatentDecodeArgs {
   const __nv_bfloat16* q_abs; int ld_qa, hs_qa;
   const __nv_bfloat16* q_raw; int ld_q, hs_q;
   const float* cos_t; const float* sin_t; int table_len, rdims;
-  const __nv_bfloat16* pages; const int* block_table; int max_pages, page_size, num_pages;
+  const __nv_bfloat16* pages; const int* block_table; int max_pages, page_size, page_shift, num_pages;      // page_shift: -1 where the size is no power of two
   const int* positions; const int* q_start;
   const float* sink; float scale; int window;
   __nv_bfloat16* out; int ld_out, hs_out, H, rank, rot;
   int* status;
 };
 
-// NP: pairs of 8 value columns per warp at most: rank <= 128 NP.
+// NP: pairs of 8 value columns per warp at most: rank <= 256 NP.
 template <int NP>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(LatentDecodeArgs p) {
@@ -956,15 +969,21 @@ latent_decode_kernel(LatentDecodeArgs p) {
   __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(ld_smem4);              // [16][DcP]
   __nv_bfloat16* Ks0 = Qs + 16 * DcP;                                           // two buffers of [64][DcP]
   __nv_bfloat16* Ps = Ks0 + 2 * LD_KEYS * DcP;                                  // [16][LD_PPAD]
-  float* Ss = reinterpret_cast<float*>(Ps + 16 * LD_PPAD);                      // [16][LD_SPAD]
+  float* Ss = reinterpret_cast<float*>(Ps + 16 * LD_PPAD);                      // [2][16][LD_SPAD]: the halves of Dc
   float* merged = reinterpret_cast<float*>(Ks0);                                // [S][own pairs][16][16], once the keys are done with
   __shared__ float m_s[16], l_s[16], corr_s[16];
   __shared__ float all_m[8 * 16], all_l[8 * 16];                                // of every block of the cluster
   __shared__ int row_ok[2][LD_KEYS];
+  __shared__ __align__(8) unsigned long long full[2];                           // a buffer's rows have arrived
   const int S = gridDim.z, part = blockIdx.z;                                   // the cluster lies along z
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   pdl_trigger();
+  if (tid < 2) {
+    asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" :: "r"((unsigned)__cvta_generic_to_shared(full + tid)), "r"(LD_WARPS));
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+  }
   if (S > 1) cluster_meet();                       // every block of the cluster runs before another writes into it
+  else __syncthreads();
   pdl_wait();
   const int req = blockIdx.x, h0 = blockIdx.y * 16, HB = min(16, p.H - h0);
   const int tr = p.q_start[req], pos = p.positions[tr];
@@ -972,50 +991,48 @@ latent_decode_kernel(LatentDecodeArgs p) {
   const int lowest = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   const int first = lowest / LD_KEYS + part, last = pos >= 0 ? pos / LD_KEYS : -1;      // this block's chunks: first, first + S, ...
   const int half = p.rdims >> 1;
+  const unsigned row_bytes = (unsigned)Dc * 2u;
 
+  // a warp brings four rows, a lane each
   auto request_chunk = [&](int c, int buf) {
+    const int slot = warp * 4 + (lane & 3), key = c * LD_KEYS + slot;
+    long long row = -1;
+    if (lane < 4 && key >= lowest && key <= pos) {
+      const int lp = p.page_shift >= 0 ? key >> p.page_shift : key / p.page_size;
+      const int page = lp < p.max_pages ? table[lp] : -1;
+      if (page < 0 || page >= p.num_pages) atomicCAS(p.status, 0, KVB_STATUS_UNMAPPED_PAGE);
+      else row = (long long)page * p.page_size + (key - lp * p.page_size);
+    }
+    const unsigned here = __ballot_sync(0xffffffffu, row >= 0);
     __nv_bfloat16* Kb = Ks0 + (size_t)buf * LD_KEYS * DcP;
-    // a warp brings eight rows; its lanes 0 - 7 look their pages up
-    const int key_l = c * LD_KEYS + warp * 8 + (lane & 7);
-    int page_l = -1;
-    if (lane < 8 && key_l >= lowest && key_l <= pos) {
-      const int lp = key_l / p.page_size;
-      page_l = lp < p.max_pages ? table[lp] : -1;
-      if (page_l < 0 || page_l >= p.num_pages) { atomicCAS(p.status, 0, KVB_STATUS_UNMAPPED_PAGE); page_l = -1; }
+    const unsigned bar = (unsigned)__cvta_generic_to_shared(full + buf);
+    if (lane < 4) row_ok[buf][slot] = row >= 0;
+    if (lane == 0)
+      asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" :: "r"(bar), "r"(__popc(here) * row_bytes) : "memory");
+    __syncwarp();
+    if (row >= 0)
+      asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+                   :: "r"((unsigned)__cvta_generic_to_shared(Kb + (size_t)slot * DcP)), "l"(p.pages + row * Dc), "r"(row_bytes), "r"(bar)
+                   : "memory");
+    if (here != 0xfu) {                            // keys that are not there: zeros (at the ends of the window only)
+      for (int r = 0; r < 4; ++r)
+        if (!((here >> r) & 1u))
+          for (int v = lane; v < Dc / 8; v += 32) reinterpret_cast<uint4*>(Kb + (size_t)(warp * 4 + r) * DcP)[v] = make_uint4(0u, 0u, 0u, 0u);
     }
-    if (lane < 8) row_ok[buf][warp * 8 + lane] = page_l >= 0;
-    const int vecs = Dc >> 3;
-#pragma unroll
-    for (int r = 0; r < 8; ++r) {
-      const int page = __shfl_sync(0xffffffffu, page_l, r), key = c * LD_KEYS + warp * 8 + r;
-      __nv_bfloat16* dst = Kb + (size_t)(warp * 8 + r) * DcP;
-      if (page >= 0) {
-        const __nv_bfloat16* src = p.pages + ((long long)page * p.page_size + key % p.page_size) * Dc;
-        for (int v = lane; v < vecs; v += 32) {
-          const unsigned d = (unsigned)__cvta_generic_to_shared(dst + 8 * v);
-          asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"(d), "l"(src + 8 * v) : "memory");
-        }
-      } else {
-        for (int v = lane; v < vecs; v += 32) reinterpret_cast<uint4*>(dst)[v] = make_uint4(0u, 0u, 0u, 0u);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (first <= last) request_chunk(first, 0);
 
-  // the heads' queries: absorbed plain part as it is, the rotated part turned here; two rows a warp
+  // the heads' queries: absorbed plain part as it is, the rotated part turned here; a row a warp
   const bool bad_pos = p.rdims > 0 && (pos < 0 || pos >= p.table_len);
   if (bad_pos && tid == 0) atomicCAS(p.status, 0, KVB_STATUS_BAD_POSITION);
-#pragma unroll
-  for (int rr = 0; rr < 2; ++rr) {
-    const int r = 2 * warp + rr;
-    __nv_bfloat16* q = Qs + (size_t)r * DcP;
-    if (r >= HB) {
+  {
+    __nv_bfloat16* q = Qs + (size_t)warp * DcP;
+    if (warp >= HB) {
       for (int i = lane; i < DcP; i += 32) q[i] = __float2bfloat16_rn(0.f);
     } else {
-      const __nv_bfloat16* qa = p.q_abs + (size_t)tr * p.ld_qa + (size_t)(h0 + r) * p.hs_qa;
+      const __nv_bfloat16* qa = p.q_abs + (size_t)tr * p.ld_qa + (size_t)(h0 + warp) * p.hs_qa;
       for (int i = lane; i < p.rank / 8; i += 32) reinterpret_cast<uint4*>(q)[i] = reinterpret_cast<const uint4*>(qa)[i];
-      const __nv_bfloat16* qr = p.q_raw + (size_t)tr * p.ld_q + (size_t)(h0 + r) * p.hs_q;
+      const __nv_bfloat16* qr = p.q_raw + (size_t)tr * p.ld_q + (size_t)(h0 + warp) * p.hs_q;
       for (int i = lane; i < half; i += 32) {
         float c = 1.f, sn = 0.f;
         if (!bad_pos) { c = p.cos_t[(size_t)pos * half + i]; sn = p.sin_t[(size_t)pos * half + i]; }
@@ -1025,28 +1042,31 @@ latent_decode_kernel(LatentDecodeArgs p) {
       }
       for (int i = p.rdims + lane; i < p.rot; i += 32) q[p.rank + i] = qr[i];
     }
-    if (lane == 0) { m_s[r] = -CUDART_INF_F; l_s[r] = 0.f; }
+    if (lane == 0) { m_s[warp] = -CUDART_INF_F; l_s[warp] = 0.f; }
   }
   const int g = lane >> 2, t4 = lane & 3, n_pairs = p.rank / 16;
+  const int steps = Dc / 16, k_from = (warp >> 3) ? (steps + 1) / 2 * 16 : 0, k_to = (warp >> 3) ? Dc : (steps + 1) / 2 * 16;
   float acc[NP][2][4];
 #pragma unroll
   for (int i = 0; i < NP; ++i)
 #pragma unroll
     for (int e = 0; e < 4; ++e) acc[i][0][e] = acc[i][1][e] = 0.f;
 
+  bool arrived = true;
   int it = 0;
   for (int c = first; c <= last; c += S, ++it) {
-    const __nv_bfloat16* Ks = Ks0 + (size_t)(it & 1) * LD_KEYS * DcP;
-    const int* ok = row_ok[it & 1];
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                               // this chunk has arrived; the chunk before is used up (first round: Qs and the row state are written)
-    if (c + S <= last) request_chunk(c + S, (it + 1) & 1);
+    const int buf = it & 1;
+    const __nv_bfloat16* Ks = Ks0 + (size_t)buf * LD_KEYS * DcP;
+    __syncthreads();                               // the chunk before is used up (first round: Qs and the row state are written)
+    if (c + S <= last) request_chunk(c + S, buf ^ 1);
+    arrived = ld_wait(full + buf, (unsigned)(it >> 1) & 1u) && arrived;
     {
       float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
       const __nv_bfloat16* a_ptr = Qs + (size_t)(lane & 15) * DcP + (lane >> 4) * 8;
-      const __nv_bfloat16* b_row = Ks + (size_t)(warp * 8 + (lane & 7)) * DcP;
-      int ks = 0;
-      for (; ks + 32 <= Dc; ks += 32) {
+      const __nv_bfloat16* b_row = Ks + (size_t)((warp & 7) * 8 + (lane & 7)) * DcP;
+      int ks = k_from;
+#pragma unroll 4
+      for (; ks + 32 <= k_to; ks += 32) {
         unsigned a0, a1, a2, a3, e0, e1, e2, e3, b0, b1, b2, b3;
         ldsm_x4(a0, a1, a2, a3, a_ptr + ks);
         ldsm_x4(e0, e1, e2, e3, a_ptr + ks + 16);
@@ -1054,34 +1074,31 @@ latent_decode_kernel(LatentDecodeArgs p) {
         mma_bf16_16816(s0, a0, a1, a2, a3, b0, b1);
         mma_bf16_16816(s1, e0, e1, e2, e3, b2, b3);
       }
-      if (ks < Dc) {
+      if (ks < k_to) {
         unsigned a0, a1, a2, a3, b0, b1, b2, b3;
         ldsm_x4(a0, a1, a2, a3, a_ptr + ks);
         ldsm_x4(b0, b1, b2, b3, b_row + ks + ((lane >> 3) & 1) * 8);
         mma_bf16_16816(s0, a0, a1, a2, a3, b0, b1);
       }
-      float* srow = Ss + g * LD_SPAD + warp * 8 + 2 * t4;
-      srow[0] = (s0[0] + s1[0]) * p.scale;
-      srow[1] = (s0[1] + s1[1]) * p.scale;
-      srow[8 * LD_SPAD] = (s0[2] + s1[2]) * p.scale;
-      srow[8 * LD_SPAD + 1] = (s0[3] + s1[3]) * p.scale;
+      float* srow = Ss + ((warp >> 3) * 16 + g) * LD_SPAD + (warp & 7) * 8 + 2 * t4;
+      *reinterpret_cast<float2*>(srow) = make_float2(s0[0] + s1[0], s0[1] + s1[1]);
+      *reinterpret_cast<float2*>(srow + 8 * LD_SPAD) = make_float2(s0[2] + s1[2], s0[3] + s1[3]);
     }
     __syncthreads();
-#pragma unroll
-    for (int rr = 0; rr < 2; ++rr) {
-      const int r = 2 * warp + rr;
-      const float a = ok[lane] ? Ss[r * LD_SPAD + lane] : -CUDART_INF_F;
-      const float b = ok[lane + 32] ? Ss[r * LD_SPAD + lane + 32] : -CUDART_INF_F;
-      const float m_old = m_s[r], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
+    {
+      const float* s = Ss + warp * LD_SPAD + lane;
+      const float a = row_ok[buf][lane] ? (s[0] + s[16 * LD_SPAD]) * p.scale : -CUDART_INF_F;
+      const float b = row_ok[buf][lane + 32] ? (s[32] + s[16 * LD_SPAD + 32]) * p.scale : -CUDART_INF_F;
+      const float m_old = m_s[warp], m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
       const float pa = a == -CUDART_INF_F ? 0.f : expf(a - m_new), pb = b == -CUDART_INF_F ? 0.f : expf(b - m_new);
-      Ps[r * LD_PPAD + lane] = __float2bfloat16_rn(pa);
-      Ps[r * LD_PPAD + lane + 32] = __float2bfloat16_rn(pb);
+      Ps[warp * LD_PPAD + lane] = __float2bfloat16_rn(pa);
+      Ps[warp * LD_PPAD + lane + 32] = __float2bfloat16_rn(pb);
       const float sum = warp_sum(pa + pb);
       if (lane == 0) {
         const float corr = m_old == m_new ? 1.f : expf(m_old - m_new);
-        m_s[r] = m_new;
-        l_s[r] = l_s[r] * corr + sum;
-        corr_s[r] = corr;
+        m_s[warp] = m_new;
+        l_s[warp] = l_s[warp] * corr + sum;
+        corr_s[warp] = corr;
       }
     }
     __syncthreads();
@@ -1099,7 +1116,7 @@ latent_decode_kernel(LatentDecodeArgs p) {
       const __nv_bfloat16* b_row = Ks + (size_t)(kk + ((lane >> 3) & 1) * 8 + (lane & 7)) * DcP + (lane >> 4) * 8;
 #pragma unroll
       for (int i = 0; i < NP; ++i) {
-        const int pair = warp + 8 * i;
+        const int pair = warp + LD_WARPS * i;
         if (pair < n_pairs) {
           unsigned b0, b1, b2, b3;
           ldsm_x4_trans(b0, b1, b2, b3, b_row + pair * 16);
@@ -1108,6 +1125,10 @@ latent_decode_kernel(LatentDecodeArgs p) {
         }
       }
     }
+  }
+  if (!arrived) {                                  // copies that may still run must not meet the block's end
+    if (lane == 0) atomicCAS(p.status, 0, KVB_STATUS_WAIT_TIMEOUT);
+    for (int i = 0; i < 2000; ++i) __nanosleep(1000);
   }
   __syncthreads();
   // ---- the blocks' maxima and sums
@@ -1142,7 +1163,7 @@ latent_decode_kernel(LatentDecodeArgs p) {
   if (S == 1) {
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
-      const int pair = warp + 8 * i;
+      const int pair = warp + LD_WARPS * i;
       if (pair >= n_pairs) continue;
 #pragma unroll
       for (int u = 0; u < 2; ++u)
@@ -1160,14 +1181,14 @@ latent_decode_kernel(LatentDecodeArgs p) {
   const int own_pairs = (n_pairs + S - 1) / S;
 #pragma unroll
   for (int i = 0; i < NP; ++i) {
-    const int pair = warp + 8 * i;
+    const int pair = warp + LD_WARPS * i;
     if (pair >= n_pairs) continue;
-    float* to = merged + ((size_t)part * own_pairs + pair / S) * 256 + 2 * t4;
+    float* to = merged + ((size_t)part * own_pairs + pair / S) * 256 + g * 16 + 2 * t4;
 #pragma unroll
-    for (int u = 0; u < 2; ++u)
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        store_in_block(to + (g + 8 * (e >> 1)) * 16 + u * 8 + (e & 1), pair % S, acc[i][u][e] * f[e >> 1]);
+    for (int u = 0; u < 2; ++u) {
+      store2_in_block(to + u * 8, pair % S, acc[i][u][0] * f[0], acc[i][u][1] * f[0]);
+      store2_in_block(to + 128 + u * 8, pair % S, acc[i][u][2] * f[1], acc[i][u][3] * f[1]);
+    }
   }
   cluster_meet();                                  // the last time anything is written into another block
   for (int i = tid; i < own_pairs * 128; i += LD_THREADS) {
@@ -1175,16 +1196,16 @@ latent_decode_kernel(LatentDecodeArgs p) {
     if (pair >= n_pairs || r >= HB) continue;
     float a = 0.f, b = 0.f;
     for (int s = 0; s < S; ++s) {
-      const float* v = merged + ((size_t)s * own_pairs + lp) * 256 + r * 16 + col;
-      a += v[0];
-      b += v[1];
+      const float2 v = *reinterpret_cast<const float2*>(merged + ((size_t)s * own_pairs + lp) * 256 + r * 16 + col);
+      a += v.x;
+      b += v.y;
     }
     *reinterpret_cast<__nv_bfloat162*>(out + (size_t)r * p.hs_out + pair * 16 + col) = __floats2bfloat162_rn(a, b);
   }
 }
 
 static size_t latent_decode_smem(int Dc) {
-  return (size_t)(16 + 2 * LD_KEYS) * (Dc + 8) * 2 + 16 * LD_PPAD * 2 + 16 * LD_SPAD * 4;
+  return (size_t)(16 + 2 * LD_KEYS) * (Dc + 8) * 2 + 16 * LD_PPAD * 2 + 32 * LD_SPAD * 4;
 }
 
 // Whether the form for single tokens takes these sizes: those of the tensor-core form whose chunks fit shared memory.
@@ -1207,8 +1228,11 @@ KVB_EXPORT int kvb_latent_decode(const void* q_abs, int ld_qa, int hs_qa, const 
       (reinterpret_cast<uintptr_t>(out) & 3) || (ld_out & 1) || (hs_out & 1))
     return KVB_ERR_ALIGN;
   using B = __nv_bfloat16;
+  int page_shift = 0;
+  while ((1 << page_shift) < page_size) ++page_shift;
+  if ((1 << page_shift) != page_size) page_shift = -1;
   const LatentDecodeArgs a{(const B*)q_abs, ld_qa, hs_qa, (const B*)q_raw, ld_q, hs_q, cos_t, sin_t, table_len, rdims,
-                           (const B*)pages, block_table, max_pages, page_size, num_pages, positions, q_start, sink, scale,
+                           (const B*)pages, block_table, max_pages, page_size, page_shift, num_pages, positions, q_start, sink, scale,
                            window, (B*)out, ld_out, hs_out, H, rank, rot, status};
   const size_t smem = latent_decode_smem(rank + rot);
   const int tiles = (H + 15) / 16, chunks = (max_keys + LD_KEYS - 1) / LD_KEYS;
@@ -1223,8 +1247,7 @@ KVB_EXPORT int kvb_latent_decode(const void* q_abs, int ld_qa, int hs_qa, const 
     else e = kvb_launch(latent_decode_kernel<NP>, grid, dim3(LD_THREADS), smem, stream, a);                             \
     return e != cudaSuccess ? (int)e : kvb_launch_result();                                                             \
   } while (0)
-  if (rank <= 128) KVB_LATENT_DECODE(1);
-  if (rank <= 256) KVB_LATENT_DECODE(2);
-  KVB_LATENT_DECODE(4);
+  if (rank <= 256) KVB_LATENT_DECODE(1);
+  KVB_LATENT_DECODE(2);
 #undef KVB_LATENT_DECODE
 }

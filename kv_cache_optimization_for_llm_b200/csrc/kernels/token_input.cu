@@ -279,6 +279,8 @@ token_input_step_kernel(float* __restrict__ resid, const T* __restrict__ delta, 
 // weights, columns k0 + 8 t .. + 7, and the same columns of token g, and hands elements 0 - 3 to one m16n8k16 product
 // and 4 - 7 to the next: the order of the columns within a product is free as long as both operands have the same.
 // W_g x: warps take (tile of 8 rows, part of the block's columns) in turn; every part's sums go to every block.
+// STAGED: the block's share of both matrices fits shared memory and is brought there before the kernel waits for its
+// predecessor, so that nothing behind the wait but the rows themselves comes from further away.
 constexpr int kStepTokens = 8;
 
 __device__ __forceinline__ void mma_tokens(float (&c)[4], const uint4& a, const uint4& b) {
@@ -288,12 +290,6 @@ __device__ __forceinline__ void mma_tokens(float (&c)[4], const uint4& a, const 
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a.z), "r"(z), "r"(a.w), "r"(z), "r"(b.z), "r"(b.w));
 }
-__device__ __forceinline__ void store2_in_block(float* p, int rank, float a, float b) {
-  unsigned local = (unsigned)__cvta_generic_to_shared(p), remote;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(local), "r"(rank));
-  asm volatile("st.shared::cluster.v2.f32 [%0], {%1, %2};" ::"r"(remote), "f"(a), "f"(b) : "memory");
-}
-
 // row . x over n_cols columns for 8 rows of weights (this lane's: `row`, valid when live) and 8 tokens (`x`: this lane's
 // token's columns in shared memory): c[0], c[1] of lane (g, t) are token g's sums for rows 2 t and 2 t + 1.
 __device__ __forceinline__ void tile_dots(const __nv_bfloat16* row, bool live, const __nv_bfloat16* x, int n_cols, int t, float (&c)[4]) {
@@ -311,6 +307,9 @@ __device__ __forceinline__ void tile_dots(const __nv_bfloat16* row, bool live, c
 
 // parts: into how many parts of `part_cols` columns (a multiple of 32) a block's columns are dealt for W_g x; dim_s: dim rounded up to
 // a multiple of 8.
+constexpr int kStepPad = 32;      // elements behind a row of shared memory: two rows of a product's operand, side by side, in different banks
+
+template <bool STAGED>
 __global__ void __launch_bounds__(kStepThreads)
 token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __restrict__ delta, const float* __restrict__ post_w,
                             float post_eps, const __nv_bfloat16* __restrict__ w_gate, const __nv_bfloat16* __restrict__ w_proj,
@@ -320,12 +319,15 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
                             int part_cols, int* status) {
   constexpr int NT = kStepTokens;
   extern __shared__ uint4 step_mma_smem[];
-  const int xs_ld = slice + 8, act_ld = dim_p + 8, dim_s = (dim + 7) / 8 * 8;
+  const int xs_ld = slice + kStepPad, act_ld = dim_p + kStepPad, dim_s = (dim + 7) / 8 * 8;
   __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(step_mma_smem);      // [NT][xs_ld] the stream, as the product reads it
   __nv_bfloat16* act = xs + NT * xs_ld;                                      // [NT][act_ld]
   float* rs = reinterpret_cast<float*>(act + NT * act_ld);                   // [NT][slice] the float32 stream
   float* sums = rs + NT * slice;                                             // [kStepBlocks * parts][NT][dim_s] shares of W_g x
   float* ys = sums;                                                          // [NT][slice], once those are used up
+  const int shares = kStepBlocks * parts * NT * dim_s;
+  __nv_bfloat16* wg_s = reinterpret_cast<__nv_bfloat16*>(sums + max(shares, NT * slice));      // STAGED: [dim][xs_ld]
+  __nv_bfloat16* wp_s = wg_s + dim * xs_ld;                                  // STAGED: [slice][act_ld]
   __shared__ float part_sq[kStepWarps * NT];
   __shared__ float sq_pending[kStepBlocks * NT], sq_y[kStepBlocks * NT];
   __shared__ int token[NT];
@@ -334,7 +336,24 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const int n_tok = min(NT, T_ - t0);
   const int c0 = min(W, rank * slice), c1 = min(W, c0 + slice), nc = c1 - c0;
-  if (t0 == 0) {       // the weights do not depend on what runs before: the first cluster asks for their lines
+  // the weights do not depend on what runs before
+  if (STAGED) {
+    const int per = nc / 8, per_p = dim_p / 8;
+    auto bring = [](__nv_bfloat16* dst, const __nv_bfloat16* src) {
+      const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" :: "r"(d), "l"(src) : "memory");
+    };
+    for (int i = tid; i < dim * per; i += kStepThreads) {
+      const int j = i / per, k = (i - j * per) * 8;
+      bring(wg_s + (size_t)j * xs_ld + k, w_gate + (size_t)j * W + c0 + k);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    for (int i = tid; i < nc * per_p; i += kStepThreads) {
+      const int r = i / per_p, k = (i - r * per_p) * 8;
+      bring(wp_s + (size_t)r * act_ld + k, w_proj + (size_t)(c0 + r) * dim_p + k);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  } else if (t0 == 0) {       // the first cluster asks for their lines
     const int per = (nc + 63) / 64;
     for (int i = tid; i < dim * per; i += kStepThreads) {
       const int j = i / per;
@@ -349,6 +368,16 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
   const bool live_tok = warp < n_tok;
   const size_t row_at = (size_t)(t0 + (live_tok ? warp : 0)) * W + c0;
   const bool normed = delta != nullptr && post_w != nullptr;
+  // the rows of the table the tokens name, and the stream: asked for before anything is waited for
+  int id_w = -1;
+  if (live_tok) {
+    id_w = token_of(ids, sampled, n_sampled, t0 + warp, V);
+    if (id_w < 0 && rank == 0 && lane == 0) atomicCAS(status, 0, KVB_STATUS_BAD_TOKEN);
+    for (int i = lane * 64; i < dim + 64; i += 2048)
+      if (id_w >= 0) asm volatile("prefetch.global.L2 [%0];" ::"l"(table + (size_t)id_w * ld_table + first + min(i, dim - 1)));
+    for (int i = lane * 32; i < nc; i += 1024) asm volatile("prefetch.global.L2 [%0];" ::"l"(resid + row_at + i));
+  }
+  if (lane == 0) token[warp] = id_w;
   if (normed) {
     float sq = 0.f;
     if (live_tok)
@@ -360,14 +389,6 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
       }
     sq = warp_sum(sq);
     if (lane < kStepBlocks) store_in_block(sq_pending + rank * NT + warp, lane, sq);
-  }
-  if (tid < NT) {
-    int id = -1;
-    if (tid < n_tok) {
-      id = token_of(ids, sampled, n_sampled, t0 + tid, V);
-      if (id < 0 && rank == 0) atomicCAS(status, 0, KVB_STATUS_BAD_TOKEN);
-    }
-    token[tid] = id;
   }
   if (normed) cluster_meet();
   else __syncthreads();
@@ -399,6 +420,7 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
       *reinterpret_cast<uint4*>(xs + warp * xs_ld + i) = *reinterpret_cast<const uint4*>(h);
     }
   }
+  if (STAGED) asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
   // ---- this block's columns of W_g x, for all of its rows, to every block of the cluster
   const int tiles = dim_s / 8;
@@ -406,7 +428,8 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
     const int tile = u % tiles, part = u / tiles, k0 = part * part_cols;
     const int j = tile * 8 + g;
     float c[4];
-    tile_dots(w_gate + (size_t)j * W + c0 + k0, j < dim, xs + g * xs_ld + k0, max(0, min(part_cols, nc - k0)), t, c);
+    const __nv_bfloat16* w_row = STAGED ? wg_s + (size_t)min(j, dim - 1) * xs_ld + k0 : w_gate + (size_t)j * W + c0 + k0;
+    tile_dots(w_row, j < dim, xs + g * xs_ld + k0, max(0, min(part_cols, nc - k0)), t, c);
     if (g < n_tok) {
       float* to = sums + ((size_t)(rank * parts + part) * NT + g) * dim_s + tile * 8 + 2 * t;
 #pragma unroll
@@ -424,12 +447,13 @@ token_input_step_mma_kernel(float* __restrict__ resid, const __nv_bfloat16* __re
     }
     act[i] = __float2bfloat16_rn(a);
   }
+  if (STAGED) asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();                                        // the shares are used up: their room is y's from here on
   // ---- this block's rows of y = W_p a
   float sq = 0.f;                                         // of token g, over this lane's rows
   for (int r0 = warp * 8; r0 < nc; r0 += kStepWarps * 8) {
     float c[4];
-    tile_dots(w_proj + (size_t)(c0 + r0 + g) * dim_p, true, act + g * act_ld, dim_p, t, c);     // nc is a multiple of 8
+    tile_dots(STAGED ? wp_s + (size_t)(r0 + g) * act_ld : w_proj + (size_t)(c0 + r0 + g) * dim_p, true, act + g * act_ld, dim_p, t, c);     // nc is a multiple of 8
     ys[g * slice + r0 + 2 * t] = c[0];
     ys[g * slice + r0 + 2 * t + 1] = c[1];
     sq = fmaf(c[0], c[0], fmaf(c[1], c[1], sq));
@@ -469,11 +493,13 @@ static void step_parts(int slice, int dim, int* parts, int* part_cols) {
   *parts = (slice + *part_cols - 1) / *part_cols;
 }
 
-static size_t step_mma_smem_bytes(int slice, int dim, int dim_p) {
+static size_t step_mma_smem_bytes(int slice, int dim, int dim_p, bool staged) {
   int parts, cols;
   step_parts(slice, dim, &parts, &cols);
   const size_t shares = (size_t)kStepBlocks * parts * kStepTokens * ((dim + 7) / 8 * 8), y = (size_t)kStepTokens * slice;
-  return (size_t)kStepTokens * (slice + 8 + dim_p + 8) * 2 + (size_t)kStepTokens * slice * 4 + (shares > y ? shares : y) * 4;
+  const size_t weights = staged ? (size_t)dim * (slice + kStepPad) + (size_t)slice * (dim_p + kStepPad) : 0;
+  return (size_t)kStepTokens * (slice + dim_p + 2 * kStepPad) * 2 + (size_t)kStepTokens * slice * 4 + (shares > y ? shares : y) * 4 +
+         weights * 2;
 }
 
 template <typename T, int NT>
@@ -503,7 +529,7 @@ static int step_tokens(int T_) { return T_ <= 16 ? 1 : (T_ <= 32 ? 2 : 4); }
 KVB_EXPORT int kvb_token_input_step_supported(int T_, int W, int dim, int dim_p, int dtype) {
   if (W < 8 || W % 8 != 0 || dim < 1 || dim_p < dim || dim_p % 8 != 0) return 0;
   const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
-  const size_t smem = dtype == KVB_BF16 ? step_mma_smem_bytes(slice, dim, dim_p) : step_smem_bytes(step_tokens(T_), slice, dim, dim_p);
+  const size_t smem = dtype == KVB_BF16 ? step_mma_smem_bytes(slice, dim, dim_p, false) : step_smem_bytes(step_tokens(T_), slice, dim, dim_p);
   return smem <= 200 * 1024 ? 1 : 0;
 }
 
@@ -522,12 +548,14 @@ KVB_EXPORT int kvb_token_input_step(float* resid, const void* delta, const float
   const int slice = (W / 8 + kStepBlocks - 1) / kStepBlocks * 8;
   if (dtype == KVB_BF16) {
     using B = __nv_bfloat16;
-    const size_t smem = step_mma_smem_bytes(slice, dim, dim_p);
+    const bool staged = step_mma_smem_bytes(slice, dim, dim_p, true) <= 220 * 1024;
+    const size_t smem = step_mma_smem_bytes(slice, dim, dim_p, staged);
+    auto kernel = staged ? token_input_step_mma_kernel<true> : token_input_step_mma_kernel<false>;
     int parts, cols;
     step_parts(slice, dim, &parts, &cols);
-    cudaError_t e = cudaFuncSetAttribute(token_input_step_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    e = kvb_launch_cluster(token_input_step_mma_kernel, dim3((T_ + kStepTokens - 1) / kStepTokens * kStepBlocks), dim3(kStepThreads),
+    e = kvb_launch_cluster(kernel, dim3((T_ + kStepTokens - 1) / kStepTokens * kStepBlocks), dim3(kStepThreads),
                            dim3(kStepBlocks), smem, stream, resid, (const B*)delta, post_w, post_eps, (const B*)w_gate,
                            (const B*)w_proj, norm_w, eps, (const B*)table, ld_table, first, V, ids, sampled, n_sampled, (B*)out, T_,
                            W, dim, dim_p, slice, parts, cols, status);

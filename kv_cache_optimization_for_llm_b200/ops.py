@@ -558,7 +558,8 @@ HEAD_GEMM_LIBRARY_MIN_ROWS = int(os.environ.get('KVB200_HEAD_GEMM_LIBRARY_MIN_RO
 def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, gate=None, tensor_cores: bool = False) -> torch.Tensor:
     """A product per head: ``out[t, h, :] = w[h] @ x[t, first + h * head_stride : ... + K]`` with
     ``w`` [H, N, K].  ``gate``: (tensor, first column) of rows [T, H * N] by whose sigmoid the result is multiplied.  float32, and bfloat16 steps of fewer than 128 rows: this package's FMA kernel, float32
-    sums in ascending k, or with ``tensor_cores`` (bfloat16, K a multiple of 8, aligned) its mma.sync kernel; bfloat16 with more rows: the library's batched product.  Returns [T, H * N]."""
+    sums in ascending k, or, for fewer than 16 rows with ``tensor_cores`` (bfloat16, K a multiple of 8, aligned), its
+    mma.sync kernel; bfloat16 with more rows: the library's batched product.  Returns [T, H * N]."""
     _need_cuda(x, w)
     H, N, K = w.shape
     assert w.is_contiguous() and w.dtype == x.dtype and x.stride(1) == 1
@@ -569,7 +570,7 @@ def head_gemm(x: torch.Tensor, first: int, head_stride: int, w: torch.Tensor, ga
         gt, gcol = gate
         assert gt.dtype == x.dtype and gt.stride(1) == 1 and gt.shape[0] == T and gt.shape[1] >= gcol + H * N
         gate_at, gate_ld = _at(gt, gcol), gt.stride(0)
-    if x.dtype == torch.bfloat16 and T >= HEAD_GEMM_LIBRARY_MIN_ROWS:
+    if x.dtype == torch.bfloat16 and T >= (16 if tensor_cores else HEAD_GEMM_LIBRARY_MIN_ROWS):
         # many rows: the library's batched product (tensor cores, float32 sums), as the other products of such steps
         xv = torch.as_strided(x, (H, T, K), (head_stride, x.stride(0), 1), x.storage_offset() + first)
         tmp = new((H, T, N), x.dtype, x.device)
