@@ -973,23 +973,28 @@ def run_compare_lobuzen(size):
     pre, dec = ("prefill_2048", "operators"), ("decode_b64", "operators_launched")
     lat_names = ("latent_attention_tc", "latent_attention")
     att_names = ("flash_attention_rows", "window_flash_attention", "window_attention")
+    # a long run of Lobuzen's latent layers attends to keys and values that were made for it, on the kernels of its other
+    # attention: all layers together
+    lob_att_ms = sum(lob["prefill_2048"]["operators"].get(k, (0, 0.0))[1] for k in att_names)
+    lat_up = 2 * z["lat_heads"] * (z["lat_dim"] + z["lat_vdim"]) * kr * T
     kernels = {
         "zatusun latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
             pairs * z["lat_heads"] * 2 * (dc + kr), per_launch(zat, *pre, *lat_names), tensor),
-        "lobuzen latent_attention, 2048 tokens (of the measured bf16 peak)": frac(
-            seen * z["lat_heads"] * 2 * (kr + kr), per_launch(lob, *pre, *lat_names), tensor),
+        "lobuzen attention of all layers, 2048 tokens (of the measured bf16 peak)": frac(
+            seen * 2 * ((n - n // 3) * z["lat_heads"] * (z["lat_dim"] + z["lat_vdim"]) + n // 3 * H * 128), lob_att_ms, tensor),
+        "lobuzen latent_rows, 2048 tokens (of the measured copy peak)": frac(T * kr * 4, per_launch(lob, *pre, "latent_rows"), hbm),
+        "lobuzen keys and values of a latent, 2048 tokens (of the measured bf16 peak)": frac(
+            lat_up, per_launch(lob, *pre, "latent_up_library"), tensor),
         "zatusun latent_attention, batch 64 (of the measured copy peak)": frac(
             R * ctx * dc * 2, per_launch(zat, *dec, *lat_names), hbm),
         "lobuzen latent_attention, batch 64 (of the measured copy peak)": frac(
-            R * min(ctx, window) * kr * 2, per_launch(lob, *dec, *lat_names), hbm),
+            R * min(ctx, window) * kr * 2, per_launch(lob, *dec, "latent_decode", *lat_names), hbm),
         "zatusun latent_prep, 2048 tokens (of the measured copy peak)": frac(
             T * 2 * (z["q_rank"] + dc) * 2, per_launch(zat, *pre, "latent_prep"), hbm),
         "lobuzen latent_prep, 2048 tokens (of the measured copy peak)": frac(
             T * 2 * kr * 2, per_launch(lob, *pre, "latent_prep"), hbm),
         "tevanex attention, 2048 tokens (of the measured bf16 peak)": frac(
             in_block * 4 * H * 64, per_launch(tev, *pre, *att_names), tensor),
-        "lobuzen attention, 2048 tokens (of the measured bf16 peak)": frac(
-            seen * 4 * H * 64, per_launch(lob, *pre, *att_names), tensor),
         "tevanex window_attention, batch 64 (of the measured copy peak)": frac(
             R * min(ctx, window) * 2 * G * 64 * 2, per_launch(tev, *dec, "window_attention"), hbm),
         "lobuzen window_attention, batch 64 (of the measured copy peak)": frac(

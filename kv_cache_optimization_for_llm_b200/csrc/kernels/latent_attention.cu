@@ -412,7 +412,7 @@ KVB_EXPORT int kvb_head_rows(const void* in, void* out, int ld_out, const void* 
 }
 
 // ---------------------------------------------------------------- the rows that long runs see
-// A block fills one page of `rows_per_page` rows of out [n_pages * rows_per_page, rank]: info [n_pages, 4] int32 holds the
+// A block fills eight rows, one per warp, of a page of `rows_per_page` rows of out [n_pages * rows_per_page, rank]: info [n_pages, 4] int32 holds the
 // request's row in the batch, the position of the page's first row, and the first position that the run sees; rows
 // in front of that or behind the request's last token are zero.  16-byte pieces.
 __global__ void __launch_bounds__(256)
@@ -426,7 +426,8 @@ latent_rows_kernel(const __nv_bfloat16* __restrict__ pages, const int* __restric
   const int end = ctx_len[req];
   const int* table = block_table + (size_t)req * max_pages;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int r = warp; r < rows_per_page; r += 8) {
+  const int r = blockIdx.y * 8 + warp;
+  if (r < rows_per_page) {
     const int pos = first + r;
     const uint4* src = nullptr;
     if (pos >= lowest && pos < end) {
@@ -448,7 +449,7 @@ KVB_EXPORT int kvb_latent_rows(const void* pages, const int* block_table, int ma
   if (rank < 8 || rank % 8 != 0 || rows_per_page < 1) return KVB_ERR_BAD_SIZE;
   if ((reinterpret_cast<uintptr_t>(pages) | reinterpret_cast<uintptr_t>(info) | reinterpret_cast<uintptr_t>(out)) & 15)
     return KVB_ERR_ALIGN;
-  kvb_launch(latent_rows_kernel, dim3(n_pages), dim3(256), 0, stream, (const __nv_bfloat16*)pages, block_table, max_pages,
+  kvb_launch(latent_rows_kernel, dim3(n_pages, (rows_per_page + 7) / 8), dim3(256), 0, stream, (const __nv_bfloat16*)pages, block_table, max_pages,
              page_size, num_pages, ctx_len, (const int4*)info, rows_per_page, rank / 8, (__nv_bfloat16*)out, status);
   return kvb_launch_result();
 }

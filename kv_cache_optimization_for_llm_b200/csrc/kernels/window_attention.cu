@@ -804,6 +804,69 @@ qk_norm_append_kernel(const T* __restrict__ src, int ld, int k_off, int v_off, c
   }
 }
 
+// The same for bfloat16 heads that are multiples of 8 wide: `lanes` neighbouring lanes (a power of two) take a head, eight
+// channels each, so that a head is one 16-byte access per lane and its norm a few shuffles.
+__global__ void __launch_bounds__(256)
+qk_norm_append_bf16x8_kernel(const __nv_bfloat16* __restrict__ src, int ld, int k_off, int v_off, const float* __restrict__ bq,
+                             const float* __restrict__ bk, const float* __restrict__ bv, const float* __restrict__ qw,
+                             const float* __restrict__ kw, float eps, __nv_bfloat16* __restrict__ q_out,
+                             __nv_bfloat16* __restrict__ pages, const int* __restrict__ block_table, int max_pages, int page_size,
+                             int num_pages, const int* __restrict__ positions, const int* __restrict__ token_req, int T_, int nq,
+                             int nkv, int Dk, int Dv, int write, int lanes, int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int units = nq + 2 * nkv, lane = threadIdx.x & (lanes - 1);
+  const int item = (blockIdx.x * 256 + threadIdx.x) / lanes;
+  const int t = item / units, unit = item - t * units;
+  const bool live = t < T_;
+  const bool is_q = unit < nq, is_k = !is_q && unit < nq + nkv;
+  const int head = is_q ? unit : (is_k ? unit - nq : unit - nq - nkv);
+  const int D = is_q || is_k ? Dk : Dv, c = lane * 8;
+  const bool mine = live && c < D;
+  float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  float sq = 0.f;
+  const float* w = is_q ? qw : (is_k ? kw : nullptr);
+  if (mine) {
+    const float* bias = is_q ? bq : (is_k ? bk : bv);
+    const uint4 u = *reinterpret_cast<const uint4*>(src + (size_t)t * ld + (is_q ? 0 : (is_k ? k_off : v_off)) + head * D + c);
+    const unsigned x[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { v[2 * i] = __uint_as_float(x[i] << 16); v[2 * i + 1] = __uint_as_float(x[i] & 0xffff0000u); }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      if (bias != nullptr) v[i] += bias[head * D + c + i];
+      sq = fmaf(v[i], v[i], sq);
+    }
+  }
+  for (int o = lanes >> 1; o > 0; o >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+  if (!mine) return;
+  __nv_bfloat16* dst;
+  if (is_q) {
+    dst = q_out + ((size_t)t * nq + head) * Dk;
+  } else {
+    if (!write) return;
+    const int pos = positions[t], lp = pos / page_size;
+    const int page = pos >= 0 && lp < max_pages ? block_table[(size_t)token_req[t] * max_pages + lp] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (lane == 0) atomicCAS(status, 0, KVB_STATUS_UNMAPPED_PAGE);
+      return;
+    }
+    dst = pages + (((size_t)page * nkv + head) * page_size + (pos - lp * page_size)) * (Dk + Dv) + (is_k ? 0 : Dk);
+  }
+  if (w != nullptr) {
+    const float f = 1.0f / sqrtf(sq / (float)D + eps);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] *= f * w[c + i];
+  }
+  unsigned r[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+    r[i] = *reinterpret_cast<const unsigned*>(&h);
+  }
+  *reinterpret_cast<uint4*>(dst + c) = make_uint4(r[0], r[1], r[2], r[3]);
+}
+
 KVB_EXPORT int kvb_qk_norm_append(const void* src, int ld, int k_off, int v_off, const float* bq, const float* bk,
                                   const float* bv, const float* qw, const float* kw, float eps, void* q_out, void* pages,
                                   const int* block_table, int max_pages, int page_size, int num_pages,
@@ -812,6 +875,16 @@ KVB_EXPORT int kvb_qk_norm_append(const void* src, int ld, int k_off, int v_off,
   if (T_ <= 0) return 0;
   if (Dk > kMaxDim || Dv > kMaxDim || Dk < 1 || Dv < 1 || nkv < 1 || nq < 1) return KVB_ERR_BAD_SIZE;
   const int units = nq + 2 * nkv;
+  if (dtype == KVB_BF16 && ((Dk | Dv | ld | k_off | v_off) & 7) == 0 && (long long)T_ * units < (1ll << 25) &&
+      ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(q_out) | reinterpret_cast<uintptr_t>(pages)) & 15) == 0) {
+    int lanes = 1;
+    while (lanes * 8 < Dk || lanes * 8 < Dv) lanes <<= 1;
+    using B = __nv_bfloat16;
+    kvb_launch(qk_norm_append_bf16x8_kernel, dim3((int)(((long long)T_ * units * lanes + 255) / 256)), dim3(256), 0, stream,
+               (const B*)src, ld, k_off, v_off, bq, bk, bv, qw, kw, eps, (B*)q_out, (B*)pages, block_table, max_pages, page_size,
+               num_pages, positions, token_req, T_, nq, nkv, Dk, Dv, write, lanes, status);
+    return kvb_launch_result();
+  }
   const int threads = units >= 8 ? 256 : 32 * units;
   KVB_DISPATCH_DTYPE(dtype, T, (kvb_launch(qk_norm_append_kernel<T>, dim3(T_), dim3(threads), 0, stream, (const T*)src, ld,
                                             k_off, v_off, bq, bk, bv, qw, kw, eps, (T*)q_out, (T*)pages, block_table,
