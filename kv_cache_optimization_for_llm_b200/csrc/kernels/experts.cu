@@ -125,7 +125,7 @@ route_kernel(const T* __restrict__ h, int ld_h, const float* __restrict__ w_rout
     }
     __syncwarp();
     if (groups > 0) {
-      // a group's score is the sum of its two best choice scores; the experts of all but the `keep` best groups are out
+      // a group stands or falls with its two best experts, added up; those of all but the `keep` best groups are out
       float* gs = g_all + (size_t)tt * groups;
       const int per = n_all / groups;
       for (int g = lane; g < groups; g += 32) {

@@ -1582,7 +1582,7 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
     chooses.  ``score`` "softmax": the scores are the logits' softmax over all experts; "sigmoid": each logit's sigmoid.
     ``renormalize`` False: a chosen expert's weight is its score times ``scale``, not divided by the chosen scores' sum.
     ``correction`` None: the choice goes by the scores alone.  ``groups`` > 0: the experts form that many equal groups of
-    neighbours; a group is judged by the sum of its two largest choice scores, and only experts of the ``keep_groups``
+    neighbours, each judged by its two best experts' scores (correction included) added up; only experts of the ``keep_groups``
     best groups can be chosen."""
     _need_cuda(h, w_router)
     T, K = h.shape

@@ -104,7 +104,7 @@ class LimitedExperts(Part):
     The router's logits ``W_r h`` are float32.  ``score`` "sigmoid" (the default): the scores are their sigmoids, each by
     itself; the ``top`` experts with the largest scores are chosen and weighted with their scores as they are.  With
     ``correction`` a learned number per expert joins the score for the choice only.  With ``groups`` the experts form that
-    many equal groups of neighbours, a group is judged by the sum of its two largest choice scores, and only experts of
+    many equal groups of neighbours, each judged by its two best experts' scores (correction included) added up; only experts of
     the ``keep_groups`` best groups can be chosen.
     "softmax_chosen": the ``top`` experts of the highest logits, each weighing its share of a softmax that leaves out all others.
     ``weigh`` "input" (the default): the weight multiplies the expert's *input*, the layer's output is the sum of
